@@ -126,12 +126,14 @@ class CacheManager:
 
     @property
     def free_pages(self) -> int:
-        return min((g.pool.free_pages for g in self.groups), default=0)
+        return min((g.pool.free_pages for g in self.groups), default=1 << 30)      # (no pages: nothing runs out)
 
     def pages_needed(self, req: RequestCache | None, n_new: int, length: int = 0) -> int:
         """Most pages any group must take so that `n_new` more tokens fit.  (A block table has
         an entry for every page of positions, given back or not, so a group with a window asks
         for as many new pages as one without.)"""
+        if not self.groups:                           # a model without pages (recurrent layers alone)
+            return 0
         cur = length if req is None else req.length + req.reserved
         total = -(-(cur + n_new) // self.page_size)
         if req is None or not req.tables:

@@ -1,9 +1,10 @@
 from .base import ConfigError, ModelConfig, parse_config_json, read_config_json
+from .bonerax import BoneraxConfig
 from .gekavik import GekavikConfig
 from .kafepel import KafepelConfig
-from .llama import LlamaConfig, RopeScaling
+from .llama import LlamaConfig, RopeScaling, YarnScaling
 from .medirax import MediraxConfig
 from .sorupel import SorupelConfig
 
-__all__ = ["ConfigError", "ModelConfig", "LlamaConfig", "MediraxConfig", "GekavikConfig", "SorupelConfig", "KafepelConfig", "RopeScaling",
+__all__ = ["ConfigError", "ModelConfig", "LlamaConfig", "MediraxConfig", "GekavikConfig", "SorupelConfig", "KafepelConfig", "BoneraxConfig", "RopeScaling", "YarnScaling",
            "parse_config_json", "read_config_json"]

@@ -19,6 +19,20 @@ from .base import ConfigError, ModelConfig
 
 
 @dataclass(frozen=True)
+class YarnScaling:
+    """YaRN's rescaling of rotary frequencies (`parts.rope.inverse_frequencies`) for contexts `factor` times as long as
+    `original` positions; cosines and sines are multiplied by `amplitude`."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    @property
+    def amplitude(self) -> float:
+        return 0.1 * math.log(self.factor) + 1.0
+
+
+@dataclass(frozen=True)
 class RopeScaling:
     """The `rope_scaling` block.  Only the llama3 frequency-band rescaling is known."""
     rope_type: str

@@ -1,5 +1,7 @@
 // Paged grouped-query attention in bfloat16 on the tensor cores, for one head size
-// (compile with -DFMX_HD=<head size>, a multiple of 16 up to 256).
+// (compile with -DFMX_HD=<head size>, a multiple of 16 up to 256; with -DFMX_VD=<head size of the values>, another
+// multiple of 16, the library holds the prefill kernel's form with 32-bit queries only, over pages of
+// [nkv, page_size, hd] keys followed by [nkv, page_size, vd] values).
 //
 // Two kernels over the same paged cache [page, 2 (k|v), nkv, page_size, hd]:
 //
@@ -36,24 +38,31 @@
 #ifndef FMX_HD
 #error "compile with -DFMX_HD=<head size>"
 #endif
+#ifndef FMX_VD
+#define FMX_VD FMX_HD              // the values' head size; another one than the keys' builds the form with 32-bit queries alone
+#endif
 
 namespace {
 constexpr int HD = FMX_HD;
+constexpr int VD = FMX_VD;               // head size of the values and of the output
 static_assert(HD % 16 == 0 && HD >= 16 && HD <= 256, "head size must be a multiple of 16, at most 256");
+static_assert(VD % 16 == 0 && VD >= 16 && VD <= 256, "the values' head size must be a multiple of 16, at most 256");
 constexpr int KSTEPS = HD / 16;          // k-steps of Q.K^T
-constexpr int NT_O = HD / 8;             // 8-wide column tiles of the output
+constexpr int NT_O = VD / 8;             // 8-wide column tiles of the output
 constexpr int BN = 64;                   // keys per tile
 constexpr int BM = 64;                   // packed query rows per prefill block
 constexpr int ROW = HD + 8;              // padded shared-memory row (elements): conflict-free ldmatrix
 constexpr int CHUNKS = HD / 8;           // 16-byte chunks per row
-constexpr int TILE = BN * ROW;           // elements of one K (or V) tile
+constexpr int TILE = BN * ROW;           // elements of one K tile (and of a V tile as wide)
+constexpr int VROW = VD + 8;
+constexpr int VTILE = BN * VROW;         // elements of one V tile
 constexpr int THREADS = 128;
-constexpr int PREFILL_STAGES = HD <= 128 ? 3 : 2;
+constexpr int PREFILL_STAGES = (HD > VD ? HD : VD) <= 128 ? 3 : 2;
 constexpr int DECODE_STAGES = HD <= 128 ? 3 : 2;
 // The form with 32-bit queries holds 2 x KSTEPS x 4 registers of query fragments beside NT_O x 4 of output: past a
 // head size of 128 that is more than a thread has, so the fragments live in shared memory behind the tiles.
-constexpr bool Q_SHARED = HD > 128;
-constexpr size_t prefill_smem() { return (size_t)PREFILL_STAGES * 2 * TILE * 2; }
+constexpr bool Q_SHARED = HD + VD > 256;
+constexpr size_t prefill_smem() { return (size_t)PREFILL_STAGES * (TILE + VTILE) * 2; }
 constexpr size_t wide_smem() { return prefill_smem() + (Q_SHARED ? (size_t)(THREADS / 32) * 2 * KSTEPS * 32 * 16 : 0); }
 constexpr int MO_ROW = HD + 4;           // floats in a row of a warp's partial output: heads 2t and 2t + 2 on other banks
 // Groups of 16 keys in a warp's decode tile.  Grids of few blocks (batch 1 to 4 with 8 kv heads) are bound by the
@@ -110,12 +119,71 @@ __device__ __forceinline__ int page_shift_of(int page_size) {
   return (page_size >= 4 && (page_size & (page_size - 1)) == 0) ? 31 - __clz(page_size) : -1;
 }
 
+#if FMX_VD != FMX_HD
+// One plane (keys or values, W wide) of keys [k0, k0 + BN) into a shared tile, for pages whose keys and values differ in
+// width: `plane` is where this kv head's rows start in a page, `page_stride` a page's elements.  As load_tiles below.
+template <int W>
+__device__ __forceinline__ void load_plane(bf16* dst, const Cache& c, long long plane, long long page_stride, int k0, int kbeg,
+                                           int kend, int* status, int where) {
+  constexpr int CH = W / 8, RW = W + 8;
+  const bf16* base = c.kv + plane;
+  if (c.page_shift >= 0) {
+    for (int item = threadIdx.x; item < (BN / 4) * CH; item += THREADS) {
+      const int rg = item / CH, ch = item - rg * CH;
+      const int key0 = k0 + 4 * rg;
+      const bf16* src = c.kv;
+      bool have = false;
+      if (key0 + 3 >= kbeg && key0 < kend) {
+        const int blk = key0 >> c.page_shift;
+        const int page = blk < c.bt_len ? c.bt[blk] : -1;
+        if (page < 0 || page >= c.num_pages) {
+          fmx_set_status(status, FMX_BAD_PAGE, page, where);
+        } else {
+          have = true;
+          src = base + page * page_stride + (long long)(key0 & (c.page_size - 1)) * W + ch * 8;
+        }
+      }
+      bf16* d = dst + (4 * rg) * RW + ch * 8;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const bool valid = have && key0 + i >= kbeg && key0 + i < kend;
+        cp_async16(d + i * RW, valid ? src + i * W : c.kv, valid);
+      }
+    }
+    return;
+  }
+  for (int idx = threadIdx.x; idx < BN * CH; idx += THREADS) {
+    const int r = idx / CH, ch = idx - r * CH;
+    const int key = k0 + r;
+    bool valid = key >= kbeg && key < kend;
+    const bf16* src = c.kv;
+    if (valid) {
+      const int blk = key / c.page_size;
+      const int page = blk < c.bt_len ? c.bt[blk] : -1;
+      if (page < 0 || page >= c.num_pages) {
+        fmx_set_status(status, FMX_BAD_PAGE, page, where);
+        valid = false;
+      } else {
+        src = base + page * page_stride + (long long)(key - blk * c.page_size) * W + ch * 8;
+      }
+    }
+    cp_async16(dst + r * RW + ch * 8, src, valid);
+  }
+}
+#endif
+
 // Bring keys [k0, k0 + BN) of kv head g into a shared K tile and a shared V tile; keys
 // outside [kbeg, kend) or without a page become zeros.  k0 is a multiple of 4.  When the
 // page size is a power of two (>= 4), four consecutive keys share a page: one block-table
 // read serves eight 16-byte copies.
 __device__ __forceinline__ void load_tiles(bf16* kdst, bf16* vdst, const Cache& c, int g, int k0, int kbeg, int kend,
                                            int* status, int where) {
+#if FMX_VD != FMX_HD
+  const long long keys = (long long)c.nkv * c.page_size * HD;
+  const long long both = keys + (long long)c.nkv * c.page_size * VD;
+  load_plane<HD>(kdst, c, (long long)g * c.page_size * HD, both, k0, kbeg, kend, status, where);
+  load_plane<VD>(vdst, c, keys + (long long)g * c.page_size * VD, both, k0, kbeg, kend, status, where);
+#else
   const long long plane_k = (long long)c.nkv * c.page_size * HD;
   const long long plane = c.keys_only ? 0 : plane_k;                    // k plane -> v plane
   const long long page_stride = c.keys_only ? plane_k : 2 * plane_k;
@@ -191,6 +259,7 @@ __device__ __forceinline__ void load_tiles(bf16* kdst, bf16* vdst, const Cache& 
     cp_async16(kdst + r * ROW + ch * 8, src, valid);
     cp_async16(vdst + r * ROW + ch * 8, valid ? src + plane : c.kv, valid);
   }
+#endif
 }
 
 // S[16 x 8*NT] += Q[16 x HD] . K^T for the key rows [key_row0, key_row0 + 8*NT) of a shared tile.
@@ -283,7 +352,7 @@ __device__ __forceinline__ void pv_tile(float (&o)[NT_O][4], const float (&p)[2 
         const int np = np0 + u;
         if (np >= PAIRS) break;
         // matrices: (keys 16kk.., hd 16np), (keys 16kk+8.., hd 16np), (keys 16kk.., hd 16np+8), (keys 16kk+8.., hd 16np+8)
-        const bf16* ptr = vs + (key_row0 + 16 * kk + (mi & 1) * 8 + ri) * ROW + 16 * np + (mi >> 1) * 8;
+        const bf16* ptr = vs + (key_row0 + 16 * kk + (mi & 1) * 8 + ri) * VROW + 16 * np + (mi >> 1) * 8;
         ldmatrix_x4_trans(b[u][0], b[u][1], b[u][2], b[u][3], ptr);
         mma_bf16(o[2 * np], a, b[u][0], b[u][1]);
         mma_bf16(o[2 * np + 1], a, b[u][2], b[u][3]);
@@ -345,6 +414,7 @@ __device__ __forceinline__ void softmax_step(float (&s)[NT][4], float (&m)[2], f
   }
 }
 
+#if FMX_VD == FMX_HD
 // ---- decode: keys on the rows ----
 // A decode row brings the few query heads of one kv head (4 with Llama's grouping).  With the heads on the 16 rows
 // of the MMA three quarters of every product were padding; here the keys are the rows and up to 8 heads the
@@ -536,6 +606,8 @@ __device__ __forceinline__ void warp_tile_any(bf16* kdst, bf16* vdst, const Cach
   }
 }
 
+#endif  // FMX_VD == FMX_HD
+
 // ------------------------------------------------------------------------------------ prefill
 // WIDE: 32-bit queries, two-term products, an optional cap and an output row stride (see the head of the file).
 template <bool WIDE>
@@ -664,8 +736,8 @@ attn_prefill_kernel(const void* __restrict__ q_any, long long q_stride, const bf
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
 
-  auto stage_k = [&](int s) { return smem + (size_t)s * 2 * TILE; };
-  auto stage_v = [&](int s) { return smem + (size_t)s * 2 * TILE + TILE; };
+  auto stage_k = [&](int s) { return smem + (size_t)s * (TILE + VTILE); };
+  auto stage_v = [&](int s) { return smem + (size_t)s * (TILE + VTILE) + TILE; };
   // tile i of the block: its first key, and the keys it may hold
   auto tile_key = [&](int i) { return i < kept_tiles ? i * BN : kstart + (i - kept_tiles) * BN; };
   auto fetch = [&](int stage, int i) {
@@ -754,28 +826,28 @@ attn_prefill_kernel(const void* __restrict__ q_any, long long q_stride, const bf
   if (one_token) {
     // the warps' parts of the same rows, added up in warp order through the tiles' shared memory
     __syncthreads();
-    float* red = reinterpret_cast<float*>(smem_raw);           // [4][16][HD + 2]
+    float* red = reinterpret_cast<float*>(smem_raw);           // [4][16][VD + 2]
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
       l[x] += __shfl_xor_sync(0xffffffffu, l[x], 1);
       l[x] += __shfl_xor_sync(0xffffffffu, l[x], 2);
-      float* mine = red + (warp * 16 + gq + 8 * x) * (HD + 2);
+      float* mine = red + (warp * 16 + gq + 8 * x) * (VD + 2);
 #pragma unroll
       for (int n = 0; n < NT_O; ++n) *reinterpret_cast<float2*>(mine + 8 * n + 2 * tq) = make_float2(o[n][2 * x], o[n][2 * x + 1]);
-      if (tq == 0) *reinterpret_cast<float2*>(mine + HD) = make_float2(m[x], l[x]);
+      if (tq == 0) *reinterpret_cast<float2*>(mine + VD) = make_float2(m[x], l[x]);
     }
     __syncthreads();
-    for (int idx = threadIdx.x; idx < rep * HD; idx += THREADS) {
-      const int row = idx / HD, e = idx - row * HD;
+    for (int idx = threadIdx.x; idx < rep * VD; idx += THREADS) {
+      const int row = idx / VD, e = idx - row * VD;
       const int w0 = (row >> 4) * kparts, wr = row & 15;     // the warps that hold this row, and its place in theirs
       float M = -INFINITY;
-      for (int w = w0; w < w0 + kparts; ++w) M = fmaxf(M, red[(w * 16 + wr) * (HD + 2) + HD]);
+      for (int w = w0; w < w0 + kparts; ++w) M = fmaxf(M, red[(w * 16 + wr) * (VD + 2) + VD]);
       float L = 0.f, O = 0.f;
       if (M != -INFINITY) {
         for (int w = w0; w < w0 + kparts; ++w) {
-          const float* pw = red + (w * 16 + wr) * (HD + 2);
-          const float f = fast_exp2(pw[HD] - M);
-          L = fmaf(pw[HD + 1], f, L);
+          const float* pw = red + (w * 16 + wr) * (VD + 2);
+          const float f = fast_exp2(pw[VD] - M);
+          L = fmaf(pw[VD + 1], f, L);
           O = fmaf(pw[e], f, O);
         }
       }
@@ -788,11 +860,11 @@ attn_prefill_kernel(const void* __restrict__ q_any, long long q_stride, const bf
         O *= a;
       }
       if (shared_keys) {
-        float* part = split_out + (((long long)t0 * nh + hq) * n_splits + split) * (HD + 2);
+        float* part = split_out + (((long long)t0 * nh + hq) * n_splits + split) * (VD + 2);
         part[e] = O;
-        if (e == 0) { part[HD] = M; part[HD + 1] = L; }
+        if (e == 0) { part[VD] = M; part[VD + 1] = L; }
       } else {
-        out[(long long)t0 * out_stride + (long long)hq * HD + e] = __float2bfloat16_rn(L > 0.f ? O / L : 0.f);
+        out[(long long)t0 * out_stride + (long long)hq * VD + e] = __float2bfloat16_rn(L > 0.f ? O / L : 0.f);
       }
     }
     return;
@@ -804,10 +876,10 @@ attn_prefill_kernel(const void* __restrict__ q_any, long long q_stride, const bf
     if (!rvalid[x]) continue;
     if (shared_keys) {
       // this share's output as it stands (not yet divided), with its maximum (scaled, base 2) and its sum
-      float* part = split_out + (((long long)(t0 + tok[x]) * nh + head[x]) * n_splits + split) * (HD + 2);
+      float* part = split_out + (((long long)(t0 + tok[x]) * nh + head[x]) * n_splits + split) * (VD + 2);
 #pragma unroll
       for (int n = 0; n < NT_O; ++n) *reinterpret_cast<float2*>(part + 8 * n + 2 * tq) = make_float2(o[n][2 * x], o[n][2 * x + 1]);
-      if (tq == 0) *reinterpret_cast<float2*>(part + HD) = make_float2(m[x], l[x]);
+      if (tq == 0) *reinterpret_cast<float2*>(part + VD) = make_float2(m[x], l[x]);
       continue;
     }
     if (WIDE && sinks != nullptr) {                        // the term without a value
@@ -819,7 +891,7 @@ attn_prefill_kernel(const void* __restrict__ q_any, long long q_stride, const bf
       for (int n = 0; n < NT_O; ++n) { o[n][2 * x] *= a; o[n][2 * x + 1] *= a; }
     }
     const float inv = l[x] > 0.f ? 1.0f / l[x] : 0.f;
-    bf16* op = out + (long long)(t0 + tok[x]) * out_stride + (long long)head[x] * HD + 2 * tq;
+    bf16* op = out + (long long)(t0 + tok[x]) * out_stride + (long long)head[x] * VD + 2 * tq;
 #pragma unroll
     for (int n = 0; n < NT_O; ++n)
       *reinterpret_cast<unsigned*>(op + 8 * n) = pack_bf16(o[n][2 * x] * inv, o[n][2 * x + 1] * inv);
@@ -836,9 +908,9 @@ attn_wide_combine_kernel(const float* part, bf16* out, long long out_stride, lon
   if (item >= n_items) return;
   const long long t = item / nh;
   const int h = (int)(item - t * nh);
-  const float* p = part + item * n_splits * (HD + 2);
+  const float* p = part + item * n_splits * (VD + 2);
   float M = -INFINITY;
-  for (int s = 0; s < n_splits; ++s) M = fmaxf(M, p[s * (HD + 2) + HD]);
+  for (int s = 0; s < n_splits; ++s) M = fmaxf(M, p[s * (VD + 2) + VD]);
   float L = 0.f;
   if (sinks != nullptr) {                                  // one more term in the denominator, with no value
     const float sk2 = sinks[h] * LOG2E;
@@ -847,30 +919,31 @@ attn_wide_combine_kernel(const float* part, bf16* out, long long out_stride, lon
     L = fast_exp2(sk2 - M);
     if (none) M = -INFINITY;                               // a row that saw no key: zeros
   }
-  float acc[(HD + 31) / 32];
+  float acc[(VD + 31) / 32];
 #pragma unroll
-  for (int i = 0; i < (HD + 31) / 32; ++i) acc[i] = 0.f;
+  for (int i = 0; i < (VD + 31) / 32; ++i) acc[i] = 0.f;
   if (M != -INFINITY) {
     for (int s = 0; s < n_splits; ++s) {
-      const float* ps = p + s * (HD + 2);
-      const float w = fast_exp2(ps[HD] - M);
-      L += ps[HD + 1] * w;
+      const float* ps = p + s * (VD + 2);
+      const float w = fast_exp2(ps[VD] - M);
+      L += ps[VD + 1] * w;
 #pragma unroll
-      for (int i = 0; i < (HD + 31) / 32; ++i) {
+      for (int i = 0; i < (VD + 31) / 32; ++i) {
         const int e = lane + 32 * i;
-        if (e < HD) acc[i] = fmaf(ps[e], w, acc[i]);
+        if (e < VD) acc[i] = fmaf(ps[e], w, acc[i]);
       }
     }
   }
   const float inv = L > 0.f ? 1.0f / L : 0.f;
-  bf16* op = out + t * out_stride + (long long)h * HD;
+  bf16* op = out + t * out_stride + (long long)h * VD;
 #pragma unroll
-  for (int i = 0; i < (HD + 31) / 32; ++i) {
+  for (int i = 0; i < (VD + 31) / 32; ++i) {
     const int e = lane + 32 * i;
-    if (e < HD) op[e] = __float2bfloat16_rn(acc[i] * inv);
+    if (e < VD) op[e] = __float2bfloat16_rn(acc[i] * inv);
   }
 }
 
+#if FMX_VD == FMX_HD
 // ---- the splits of a row as one thread-block cluster ----
 __device__ __forceinline__ void cluster_sync_all() {
   asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -1321,9 +1394,12 @@ cudaError_t configure_decode() {
       if ((rep) <= 8) { LAUNCH(1, 1); } else { LAUNCH(2, 1); }            \
     }                                                     \
   } while (0)
+#endif  // FMX_VD == FMX_HD
 }  // namespace
 
 FMX_EXPORT int fmx_attn_head_dim() { return HD; }
+
+#if FMX_VD == FMX_HD
 
 // 0: the splits of a row always combine through L2 and tickets, as they do where a cluster does not fit (for tests
 // and timings of that path); 1, the default: through a cluster's shared memory where one fits.  -> the old setting
@@ -1388,6 +1464,8 @@ FMX_EXPORT int fmx_attn_prefill(const void* q, long long q_stride, const void* k
   return 0;
 }
 
+#endif  // FMX_VD == FMX_HD
+
 // The form with 32-bit queries q[T, nh*hd] (row stride in floats), two-term products, capped scores (softcap > 0)
 // and an output whose rows are `out_stride` elements apart.  Takes every kind of row, single tokens included.
 // positions (or null): the step's token positions; a row whose first token stands at -1 is padding and gets zeros.
@@ -1408,8 +1486,9 @@ FMX_EXPORT int fmx_attn_prefill_wide_masked(const float* q, long long q_stride, 
   if (rows < 0 || nh <= 0 || nkv <= 0 || nh % nkv || page_size <= 0)
     return fmx_fail("fmx_attn_prefill_wide: bad sizes rows=%d nh=%d nkv=%d page=%d", rows, nh, nkv, page_size);
   if (rows > 65535 || nkv > 65535) return fmx_fail("fmx_attn_prefill_wide: too many rows or kv heads for one launch");
-  if (q_stride % 2 || ((uintptr_t)q & 7) || out_stride % 2 || ((uintptr_t)out & 3) || out_stride < (long long)nh * HD)
-    return fmx_fail("fmx_attn_prefill_wide: queries in 8-byte pairs and outputs in 4-byte pairs, rows at least nh*hd wide");
+  if (VD != HD && keys_only) return fmx_fail("fmx_attn_prefill_wide: values that are the keys have the keys' width");
+  if (q_stride % 2 || ((uintptr_t)q & 7) || out_stride % 2 || ((uintptr_t)out & 3) || out_stride < (long long)nh * VD)
+    return fmx_fail("fmx_attn_prefill_wide: queries in 8-byte pairs and outputs in 4-byte pairs, rows at least nh*vd wide");
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -1425,7 +1504,7 @@ FMX_EXPORT int fmx_attn_prefill_wide_masked(const float* q, long long q_stride, 
     // rows of one token each (their tokens are [first token of the first row, + rows)): the keys of a row are shared
     // out over n_splits blocks, which leave their parts in `scratch` for the combining kernel
     if (max_q_len != 1) return fmx_fail("fmx_attn_prefill_wide: only rows of one token share their keys out over blocks");
-    if (scratch == nullptr || (long long)n_tokens * nh * n_splits * (HD + 2) > scratch_floats)
+    if (scratch == nullptr || (long long)n_tokens * nh * n_splits * (VD + 2) > scratch_floats)
       return fmx_fail("fmx_attn_prefill_wide: the workspace is too small for %d shares of %d tokens", n_splits, n_tokens);
     dim3 grid(nkv, rows, (unsigned)n_splits);
     attn_prefill_kernel<true><<<grid, THREADS, wide_smem(), stream>>>(
@@ -1470,7 +1549,7 @@ FMX_EXPORT int fmx_attn_wide_combine_sinks(const float* scratch, void* out, long
   if (n_tokens <= 0) return 0;
   const long long items = (long long)n_tokens * nh;
   attn_wide_combine_kernel<<<(unsigned)((items + 3) / 4), 128, 0, stream>>>(
-      scratch + (long long)first_token * nh * n_splits * (HD + 2), (bf16*)out + (long long)first_token * out_stride, out_stride,
+      scratch + (long long)first_token * nh * n_splits * (VD + 2), (bf16*)out + (long long)first_token * out_stride, out_stride,
       items, nh, n_splits, sinks);
   FMX_LAUNCH_CHECK();
   return 0;
@@ -1481,6 +1560,7 @@ FMX_EXPORT int fmx_attn_wide_combine(const float* scratch, void* out, long long 
   return fmx_attn_wide_combine_sinks(scratch, out, out_stride, first_token, n_tokens, nh, n_splits, nullptr, stream);
 }
 
+#if FMX_VD == FMX_HD
 // tickets: rows * nkv ints, zero before the first call (every call leaves them zero); with
 // tickets the last block of each (row, kv head) combines the splits itself, without them a
 // second kernel does.  Calls that share scratch or tickets must not overlap on the GPU.
@@ -1619,3 +1699,4 @@ FMX_EXPORT int fmx_attn_decode_noalloc(const void* q, long long q_stride, const 
   }
   return 0;
 }
+#endif  // FMX_VD == FMX_HD

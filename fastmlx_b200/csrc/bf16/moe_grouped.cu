@@ -9,7 +9,8 @@
 //
 // fmx_moe_grouped_gate_up: tile (m, n) = 128 sorted rows x 64 hidden columns of the tile's expert: G = X W_gate^T and
 // U = X W_up^T side by side (mma.sync m16n8k16, bf16 in, 32-bit sums, a three-stage cp.async ring of tiles of 32 along K),
-// and in the epilogue y = w * g' sigmoid(1.702 g') (u' + 1), g' = min(G, limit), u' = clamp(U, -limit, limit), w the
+// and in the epilogue y = w * g' sigmoid(1.702 g') (u' + 1), g' = min(G, limit), u' = clamp(U, -limit, limit) (with limit < 0:
+// y = w silu(G) U), w the
 // pair's weight; rows are gathered from the step's activations by token.  fmx_moe_grouped_down: pair outputs
 // Y W_down^T in 32-bit, 128 x 128 per tile.  fmx_moe_combine: a token's pair outputs added in the order of its choices, plus the shared
 // expert's output, rounded once.
@@ -213,9 +214,14 @@ moe_grouped_kernel(const bf16* a, long long lda, const int* sorted_token, const 
         for (int c = 0; c < 2; ++c) {
           if (n + c >= N) continue;
           if (GATED) {
-            const float g = fminf(acc0[i][j][2 * x + c], limit);
-            const float u = fminf(fmaxf(acc1[i][j][2 * x + c], -limit), limit);
-            const float y = w * (g / (1.0f + expf(-1.702f * g))) * (u + 1.0f);
+            float g = acc0[i][j][2 * x + c], u = acc1[i][j][2 * x + c], y;
+            if (limit < 0.f) {
+              y = w * (g / (1.0f + expf(-g))) * u;
+            } else {
+              g = fminf(g, limit);
+              u = fminf(fmaxf(u, -limit), limit);
+              y = w * (g / (1.0f + expf(-1.702f * g))) * (u + 1.0f);
+            }
             reinterpret_cast<bf16*>(out)[row * ldo + n + c] = __float2bfloat16_rn(y);
           } else {
             reinterpret_cast<float*>(out)[row * ldo + n + c] = acc0[i][j][2 * x + c];

@@ -22,6 +22,7 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 GROUPS = {
     # name: directory of its sources.  A name like "attn_hd64" is the group "attn" compiled
     # with -DFMX_HD=64: one library per head size, built when a model of that size is met.
+    # "attn_hd64_vd128": values of another width than the keys (the kernel with 32-bit queries alone).
     "common": "common",
     "bf16": "bf16",
     "attn": "attn",
@@ -29,6 +30,8 @@ GROUPS = {
     # (values per lane, query heads per key head), built when a model of those sizes is met
     "mixattn": "mixattn",
     "tc": "tc",
+    # linear attention with a decay per key channel (gated linear attention, the delta rule's form)
+    "chan": "chan",
     # host code: the native step executor (no kernel of its own)
     "host": "host",
     # the tensor-core product built for one test: a wait limit of 100,000 clocks and a producer that
@@ -43,10 +46,10 @@ MIXATTN_SIZES = (1, 2, 4, 8)          # values per lane (value heads up to 32 ti
 def _split(group: str) -> tuple[str, list[str]]:
     """'attn_hd64' -> ('attn', ['-DFMX_HD=64']); other names stand for themselves."""
     if group.startswith("attn_hd"):
-        hd = int(group[len("attn_hd"):])
-        if hd not in HEAD_DIMS:
-            raise BuildError(f"the tiled attention kernels take head sizes in steps of 16 up to 256, not {hd}")
-        return "attn", [f"-DFMX_HD={hd}"]
+        hd, _, vd = group[len("attn_hd"):].partition("_vd")
+        if int(hd) not in HEAD_DIMS or (vd and int(vd) not in HEAD_DIMS):
+            raise BuildError(f"the tiled attention kernels take head sizes in steps of 16 up to 256, not {hd} {vd}")
+        return "attn", [f"-DFMX_HD={hd}"] + ([f"-DFMX_VD={vd}"] if vd else [])
     if group.startswith("mixattn_v"):
         try:
             vpl, per = (int(x) for x in group[len("mixattn_v"):].split("_p"))
@@ -84,6 +87,8 @@ def sources(group: str) -> list[str]:
     if not os.path.isdir(d):
         return []
     srcs = sorted(os.path.join(d, f) for f in os.listdir(d) if f.endswith(".cu"))
+    if group.startswith("attn_hd") and "_vd" in group:
+        srcs = [os.path.join(d, "attention_bf16.cu")]             # the other kernels read values as wide as keys
     if srcs and _split(group)[0] != "common":
         srcs.append(os.path.join(HERE, "common", "error.cu"))     # every library carries its own error text
     return srcs

@@ -413,6 +413,32 @@ FMX_EXPORT int fmx_activation(const void* x, long long x_stride, void* out, long
   return 0;
 }
 
+// Output logits scaled and capped in place: x <- cap tanh(x scale / cap) (cap <= 0: x <- x scale), in 32-bit.
+namespace {
+__global__ void logit_cap_kernel(float* x, long long stride, long long rows, int cols, float scale, float cap) {
+  pdl_wait();
+  pdl_trigger();
+  const long long n = rows * cols;
+  for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < n; idx += (long long)gridDim.x * blockDim.x) {
+    const long long r = idx / cols;
+    float* p = x + r * stride + (idx - r * cols);
+    const float v = *p * scale;
+    *p = cap > 0.f ? cap * tanhf(v / cap) : v;
+  }
+}
+}  // namespace
+
+FMX_EXPORT int fmx_logit_cap(float* x, long long stride, int rows, int cols, float scale, float cap, cudaStream_t stream) {
+  if (rows == 0 || cols == 0) return 0;
+  if (rows < 0 || cols < 0 || stride < cols) return fmx_fail("fmx_logit_cap: bad sizes rows=%d cols=%d", rows, cols);
+  const long long n = (long long)rows * cols, most = (long long)fmx_num_sms() * 16;
+  const int block = 256;
+  const int grid = (int)((n + block - 1) / block < most ? (n + block - 1) / block : most);
+  fmx_launch(logit_cap_kernel, dim3(grid), dim3(block), 0, stream, x, stride, (long long)rows, cols, scale, cap);
+  FMX_LAUNCH_CHECK();
+  return 0;
+}
+
 // The scaled embedding: rows of a table of type `dtype`, times `scale`, out in 32-bit.
 FMX_EXPORT int fmx_embed_scaled(const void* table, int dtype, const int* ids, float* out, int n, int d, long long nrows,
                                 float scale, int* status, int code, cudaStream_t stream) {

@@ -9,7 +9,7 @@
 // moe_expert_act: the hidden layer of all experts side by side.  gu[t] holds F gate values and then F up values,
 // F = E * ff (+ ff_shared for an expert that every token uses); y = w * g' sigmoid(1.702 g') (u' + 1) with
 // g' = min(g, limit), u' = clamp(u, -limit, limit), and w the token's weight for the column's expert (1 for the
-// shared one).  A column whose expert the token did not choose is zero, so that one product with all the experts'
+// shared one); with limit < 0 the expert's form is silu(g) u instead.  A column whose expert the token did not choose is zero, so that one product with all the experts'
 // down matrices side by side gives the weighted sum.
 #include <math.h>
 #include "common.cuh"
@@ -28,7 +28,8 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const float* z, long long z_stride, int T, int E, int top, int groups, int keep, float* weights,
-                 int* chosen, const float* __restrict__ choice_bias, float weight_scale) {
+                 int* chosen, const float* __restrict__ choice_bias, float weight_scale,
+                 const float* __restrict__ logit_bias, int renorm) {
   extern __shared__ float smem[];               // per warp: E scores, E marks (as floats), `groups` group scores
   pdl_wait();
   pdl_trigger();
@@ -40,16 +41,17 @@ moe_route_kernel(const float* z, long long z_stride, int T, int E, int top, int 
   float* gs = ok + E;
   const float* zr = z + (long long)t * z_stride;
   float m = -INFINITY;
-  for (int e = lane; e < E; e += 32) m = fmaxf(m, zr[e]);
+  auto logit = [&](int e) { return logit_bias != nullptr ? zr[e] + logit_bias[e] : zr[e]; };
+  for (int e = lane; e < E; e += 32) m = fmaxf(m, logit(e));
   m = warp_max(m);
   float sum = 0.f;
   for (int e = lane; e < E; e += 32) {
-    const float p = expf(zr[e] - m);
+    const float p = expf(logit(e) - m);
     s[e] = p;
     sum += p;
   }
   sum = warp_sum(sum);
-  const float inv = 1.0f / sum;
+  const float inv = renorm ? 1.0f : 1.0f / sum;  // renorm: the chosen experts' exponentials are divided by their own sum
   for (int e = lane; e < E; e += 32) {
     s[e] *= inv;
     ok[e] = 1.f;
@@ -77,6 +79,7 @@ moe_route_kernel(const float* z, long long z_stride, int T, int E, int top, int 
       __syncwarp();
     }
   }
+  float chosen_sum = 0.f;
   for (int k = 0; k < top; ++k) {
     float bv = -INFINITY;
     int bi = 0x7fffffff;
@@ -94,8 +97,22 @@ moe_route_kernel(const float* z, long long z_stride, int T, int E, int top, int 
       weights[(long long)t * E + bi] = s[bi] * weight_scale;
       if (chosen != nullptr) chosen[(long long)t * top + k] = bi;
     }
+    chosen_sum += s[bi];
     __syncwarp();
   }
+  if (renorm) {
+    const float mul = weight_scale / chosen_sum;
+    for (int e = lane; e < E; e += 32)
+      if (ok[e] == 0.f) weights[(long long)t * E + e] = s[e] * mul;         // without groups, what is not allowed was chosen
+  }
+}
+
+// limit >= 0: g' sigmoid(1.702 g') (u' + 1), clamped; limit < 0: silu(g) u.
+__device__ __forceinline__ float expert_act(float g, float u, float limit) {
+  if (limit < 0.f) return g / (1.0f + expf(-g)) * u;
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return (g / (1.0f + expf(-1.702f * g))) * (u + 1.0f);
 }
 
 template <typename T>
@@ -115,9 +132,7 @@ __global__ void moe_expert_act_kernel(const T* gu, long long gu_stride, const fl
       // block > 0: gate and up values alternate in blocks of `block`; else F gates, then F ups
       const long long gi = block > 0 ? (long long)(c / block) * 2 * block + c % block : c;
       const long long ui = block > 0 ? gi + block : (long long)F + c;
-      const float g = fminf(to_f(gu[r * gu_stride + gi]), lim);
-      const float u = fminf(fmaxf(to_f(gu[r * gu_stride + ui]), -lim), lim);
-      y = w * (g / (1.0f + expf(-1.702f * g))) * (u + 1.0f);
+      y = w * expert_act(to_f(gu[r * gu_stride + gi]), to_f(gu[r * gu_stride + ui]), lim);
     }
     out[r * out_stride + c] = from_f<T>(y);
   }
@@ -147,10 +162,7 @@ __global__ void moe_expert_act_vec_kernel(const bf16* gu, long long gu_stride, c
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const float2 g = __bfloat1622float2(gp[i]), u = __bfloat1622float2(up[i]);
-        const float g0 = fminf(g.x, lim), g1 = fminf(g.y, lim);
-        const float u0 = fminf(fmaxf(u.x, -lim), lim), u1 = fminf(fmaxf(u.y, -lim), lim);
-        op[i] = __floats2bfloat162_rn(w * (g0 / (1.0f + expf(-1.702f * g0))) * (u0 + 1.0f),
-                                      w * (g1 / (1.0f + expf(-1.702f * g1))) * (u1 + 1.0f));
+        op[i] = __floats2bfloat162_rn(w * expert_act(g.x, u.x, lim), w * expert_act(g.y, u.y, lim));
       }
     }
     *reinterpret_cast<uint4*>(out + r * out_stride + c) = o;
@@ -188,25 +200,33 @@ __global__ void moe_plain_act_kernel(const T* u, long long u_stride, const float
 }
 }  // namespace
 
-// choice_bias ([E], may be null): added to the scores for the choice only; weight_scale multiplies the chosen scores.
+// choice_bias ([E], may be null): added to the scores for the choice only; weight_scale multiplies the chosen scores;
+// logit_bias ([E], may be null): added to the logits; renorm (without groups): a token's weights are the softmax over its
+// chosen experts' logits alone.
+FMX_EXPORT int fmx_moe_route_ex(const float* z, long long z_stride, int T, int E, int top, int groups, int keep, float* weights,
+                                int* chosen, const float* choice_bias, float weight_scale, const float* logit_bias, int renorm,
+                                cudaStream_t stream);
 FMX_EXPORT int fmx_moe_route_biased(const float* z, long long z_stride, int T, int E, int top, int groups, int keep,
                                     float* weights, int* chosen, const float* choice_bias, float weight_scale,
-                                    cudaStream_t stream);
+                                    cudaStream_t stream) {
+  return fmx_moe_route_ex(z, z_stride, T, E, top, groups, keep, weights, chosen, choice_bias, weight_scale, nullptr, 0, stream);
+}
 FMX_EXPORT int fmx_moe_route(const float* z, long long z_stride, int T, int E, int top, int groups, int keep, float* weights,
                              int* chosen, cudaStream_t stream) {
   return fmx_moe_route_biased(z, z_stride, T, E, top, groups, keep, weights, chosen, nullptr, 1.0f, stream);
 }
 
-FMX_EXPORT int fmx_moe_route_biased(const float* z, long long z_stride, int T, int E, int top, int groups, int keep,
-                                    float* weights, int* chosen, const float* choice_bias, float weight_scale,
-                                    cudaStream_t stream) {
+FMX_EXPORT int fmx_moe_route_ex(const float* z, long long z_stride, int T, int E, int top, int groups, int keep, float* weights,
+                                int* chosen, const float* choice_bias, float weight_scale, const float* logit_bias, int renorm,
+                                cudaStream_t stream) {
   if (T == 0) return 0;
+  if (renorm && groups > 1 && keep < groups) return fmx_fail("fmx_moe_route: weights over the chosen logits alone come without groups");
   if (T < 0 || E <= 0 || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || z_stride < E)
     return fmx_fail("fmx_moe_route: bad sizes T=%d E=%d top=%d groups=%d keep=%d", T, E, top, groups, keep);
   const size_t smem = (size_t)ROUTE_WARPS * (2 * (size_t)E + groups) * sizeof(float);
   if (smem > 48 * 1024) return fmx_fail("fmx_moe_route: %d experts are more than the kernel's shared memory holds", E);
   fmx_launch(moe_route_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, stream, z, z_stride, T, E,
-             top, groups, keep, weights, chosen, choice_bias, weight_scale);
+             top, groups, keep, weights, chosen, choice_bias, weight_scale, logit_bias, renorm);
   FMX_LAUNCH_CHECK();
   return 0;
 }

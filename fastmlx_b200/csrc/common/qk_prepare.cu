@@ -22,7 +22,7 @@ qk_prepare_kernel(const TI* qkv, long long row_stride, const int* positions, con
                   const long long* slot_mapping, float* q_out, T* kv, int nh, int nkv, int hd, int vd, int rot,
                   int interleaved, float norm_eps, int page_size, long long num_pages, int* status,
                   const float* __restrict__ bias, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
-                  int norm_first) {
+                  int norm_first, float amplitude, float v_scale) {
   extern __shared__ float smem[];               // [rot/2] sines, [rot/2] cosines, then a head per warp
   pdl_wait();
   pdl_trigger();
@@ -34,7 +34,12 @@ qk_prepare_kernel(const TI* qkv, long long row_stride, const int* positions, con
   float* buf = smem + rot + warp * hd;
   const TI* row = qkv + (long long)t * row_stride;
   const float pos = (float)positions[t];
-  for (int j = threadIdx.x; j < half; j += blockDim.x) sincosf(pos * inv_freq[j], &sn[j], &cs[j]);
+  for (int j = threadIdx.x; j < half; j += blockDim.x) {
+    float sj, cj;
+    sincosf(pos * inv_freq[j], &sj, &cj);
+    sn[j] = sj * amplitude;
+    cs[j] = cj * amplitude;
+  }
   long long slot = (kv != nullptr && slot_mapping != nullptr) ? slot_mapping[t] : -1;
   if (slot >= num_pages * page_size) {
     if (threadIdx.x == 0) fmx_set_status(status, FMX_BAD_SLOT, slot, t);
@@ -114,7 +119,7 @@ qk_prepare_kernel(const TI* qkv, long long row_stride, const int* positions, con
   T* vdst = kv + page * page_elems + (long long)nkv * page_size * hd;
   for (int it = threadIdx.x; it < nkv * vd; it += blockDim.x) {
     const int g = it / vd, e = it - g * vd;
-    vdst[((long long)g * page_size + off) * vd + e] = from_f<T>(to_f(vsrc[it]) + (vbias != nullptr ? vbias[it] : 0.f));
+    vdst[((long long)g * page_size + off) * vd + e] = from_f<T>((to_f(vsrc[it]) + (vbias != nullptr ? vbias[it] : 0.f)) * v_scale);
   }
 }
 
@@ -129,7 +134,7 @@ qk_prepare_whole_kernel(const TI* qkv, long long row_stride, const int* position
                         const long long* slot_mapping, float* q_out, T* kv, int nh, int nkv, int hd, int vd, int rot,
                         int interleaved, float norm_eps, int page_size, long long num_pages, int* status,
                         const float* __restrict__ bias, const float* __restrict__ q_weight,
-                        const float* __restrict__ k_weight, int values_from_keys) {
+                        const float* __restrict__ k_weight, int values_from_keys, float amplitude, float v_scale) {
   extern __shared__ float smem[];               // [rot/2] sines, [rot/2] cosines, then a head per warp
   pdl_wait();
   pdl_trigger();
@@ -141,7 +146,12 @@ qk_prepare_whole_kernel(const TI* qkv, long long row_stride, const int* position
   float* buf = smem + rot + warp * hd;
   const TI* row = qkv + (long long)t * row_stride;
   const float pos = (float)positions[t];
-  for (int j = threadIdx.x; j < half; j += blockDim.x) sincosf(pos * inv_freq[j], &sn[j], &cs[j]);
+  for (int j = threadIdx.x; j < half; j += blockDim.x) {
+    float sj, cj;
+    sincosf(pos * inv_freq[j], &sj, &cj);
+    sn[j] = sj * amplitude;
+    cs[j] = cj * amplitude;
+  }
   long long slot = (kv != nullptr && slot_mapping != nullptr) ? slot_mapping[t] : -1;
   if (slot >= num_pages * page_size) {
     if (threadIdx.x == 0) fmx_set_status(status, FMX_BAD_SLOT, slot, t);
@@ -175,7 +185,7 @@ qk_prepare_whole_kernel(const TI* qkv, long long row_stride, const int* position
                   : nullptr;
     for (int e = lane; e < hd; e += 32) {
       const float v = to_f(src[e]) + (bias != nullptr ? bias[(long long)h * hd + e] : 0.f);
-      if (vdst != nullptr) vdst[e] = from_f<T>(v);                 // the value: the key as it was projected
+      if (vdst != nullptr) vdst[e] = from_f<T>(v * v_scale);       // the value: the key as it was projected
       buf[e] = v * mul * (hw != nullptr ? hw[e] : 1.0f);
     }
     __syncwarp();
@@ -204,19 +214,21 @@ qk_prepare_whole_kernel(const TI* qkv, long long row_stride, const int* position
   T* vdst = kv + page * page_elems + (long long)nkv * page_size * hd;
   for (int it = threadIdx.x; it < nkv * vd; it += blockDim.x) {
     const int g = it / vd, e = it - g * vd;
-    vdst[((long long)g * page_size + off) * vd + e] = from_f<T>(to_f(vsrc[it]) + (vbias != nullptr ? vbias[it] : 0.f));
+    vdst[((long long)g * page_size + off) * vd + e] = from_f<T>((to_f(vsrc[it]) + (vbias != nullptr ? vbias[it] : 0.f)) * v_scale);
   }
 }
 }  // namespace
 
 // rot = 0: nothing is rotated; norm_eps < 0: heads are not normalised; kv or slot_mapping null:
 // nothing is stored (a layer that reads another's cache then passes nkv = 0 as well).  in_dtype: the
-// type of qkv; dtype: the cache's.  bias (the whole row's, 32-bit), q_weight, k_weight may be null.
+// type of qkv; dtype: the cache's.  bias (the whole row's, 32-bit), q_weight, k_weight may be null.  amplitude: what cosines
+// and sines are multiplied by (1: a plain rotation); v_scale: what the values are multiplied by, in 32-bit, on their way
+// into the cache.
 FMX_EXPORT int fmx_qk_prepare_ex(const void* qkv, long long row_stride, const int* positions, const float* inv_freq,
                                  const long long* slot_mapping, float* q_out, void* kv, int T, int nh, int nkv, int hd,
                                  int vd, int rot, int interleaved, float norm_eps, int page_size, long long num_pages,
                                  int in_dtype, int dtype, const float* bias, const float* q_weight, const float* k_weight,
-                                 int norm_first, int* status, cudaStream_t stream) {
+                                 int norm_first, float amplitude, float v_scale, int* status, cudaStream_t stream) {
   if (T == 0) return 0;
   if (T < 0 || nh < 0 || nkv < 0 || hd <= 0 || vd <= 0 || hd > 256 || rot < 0 || rot > hd || (rot & 1) || page_size <= 0)
     return fmx_fail("fmx_qk_prepare: bad sizes T=%d nh=%d nkv=%d hd=%d vd=%d rot=%d", T, nh, nkv, hd, vd, rot);
@@ -226,7 +238,7 @@ FMX_EXPORT int fmx_qk_prepare_ex(const void* qkv, long long row_stride, const in
 #define FMX_QKP(TI, TKV)                                                                                                  \
   fmx_launch(qk_prepare_kernel<TI, TKV>, dim3(T), dim3(QKP_WARPS * 32), smem, stream, (const TI*)qkv, row_stride, positions, \
              inv_freq, slot_mapping, q_out, (TKV*)kv, nh, nkv, hd, vd, rot, interleaved, norm_eps, page_size, num_pages,  \
-             status, bias, q_weight, k_weight, norm_first)
+             status, bias, q_weight, k_weight, norm_first, amplitude, v_scale)
   if (in_dtype == FMX_F32 && dtype == FMX_F32)
     FMX_QKP(float, float);
   else if (in_dtype == FMX_BF16 && dtype == FMX_BF16)
@@ -245,7 +257,7 @@ FMX_EXPORT int fmx_qk_prepare(const void* qkv, long long row_stride, const int* 
                               int rot, int interleaved, float norm_eps, int page_size, long long num_pages, int dtype,
                               int* status, cudaStream_t stream) {
   return fmx_qk_prepare_ex(qkv, row_stride, positions, inv_freq, slot_mapping, q_out, kv, T, nh, nkv, hd, vd, rot, interleaved,
-                           norm_eps, page_size, num_pages, dtype, dtype, nullptr, nullptr, nullptr, 0, status, stream);
+                           norm_eps, page_size, num_pages, dtype, dtype, nullptr, nullptr, nullptr, 0, 1.f, 1.f, status, stream);
 }
 
 // q and k normalised over the whole projection, before the rotation (q_weight [nh*hd], k_weight [nkv*hd], either may be
@@ -254,7 +266,7 @@ FMX_EXPORT int fmx_qk_prepare_whole(const void* qkv, long long row_stride, const
                                     const long long* slot_mapping, float* q_out, void* kv, int T, int nh, int nkv, int hd,
                                     int vd, int rot, int interleaved, float norm_eps, int page_size, long long num_pages,
                                     int in_dtype, int dtype, const float* bias, const float* q_weight, const float* k_weight,
-                                    int values_from_keys, int* status, cudaStream_t stream) {
+                                    int values_from_keys, float amplitude, float v_scale, int* status, cudaStream_t stream) {
   if (T == 0) return 0;
   if (T < 0 || nh < 0 || nkv < 0 || hd <= 0 || vd <= 0 || hd > 256 || rot < 0 || rot > hd || (rot & 1) || page_size <= 0)
     return fmx_fail("fmx_qk_prepare_whole: bad sizes T=%d nh=%d nkv=%d hd=%d vd=%d rot=%d", T, nh, nkv, hd, vd, rot);
@@ -266,7 +278,7 @@ FMX_EXPORT int fmx_qk_prepare_whole(const void* qkv, long long row_stride, const
 #define FMX_QKW(TI, TKV)                                                                                                 \
   fmx_launch(qk_prepare_whole_kernel<TI, TKV>, dim3(T), dim3(QKP_WARPS * 32), smem, stream, (const TI*)qkv, row_stride,  \
              positions, inv_freq, slot_mapping, q_out, (TKV*)kv, nh, nkv, hd, vd, rot, interleaved, norm_eps, page_size, \
-             num_pages, status, bias, q_weight, k_weight, values_from_keys)
+             num_pages, status, bias, q_weight, k_weight, values_from_keys, amplitude, v_scale)
   if (in_dtype == FMX_F32 && dtype == FMX_F32)
     FMX_QKW(float, float);
   else if (in_dtype == FMX_BF16 && dtype == FMX_BF16)

@@ -36,7 +36,7 @@ constexpr int BM = 128, BK = 64, UMMA_K = 16;
 constexpr int THREADS = 192;
 
 // RELU2: max(x, 0)^2.  EXPERT: a routed expert's gated activation, w g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit),
-// u' = clamp(u, -limit, limit) and w the row's weight, over gate/up blocks like SILU_MUL.  F32: the product as 32-bit floats.
+// u' = clamp(u, -limit, limit) and w the row's weight (limit < 0: w silu(g) u), over gate/up blocks like SILU_MUL.  F32: the product as 32-bit floats.
 // GELU_MUL: SILU_MUL with the tanh form of gelu on the gate.
 enum Epilogue { EPI_PLAIN = 0, EPI_SILU_MUL = 1, EPI_RESIDUAL = 2, EPI_RELU2 = 3, EPI_EXPERT = 4, EPI_F32 = 5, EPI_GELU_MUL = 6 };
 
@@ -236,9 +236,13 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
               f[i] = (EPI == EPI_SILU_MUL ? silu(g) : gelu_tanh(g)) * w;
             }
             if (EPI == EPI_EXPERT) {
-              const float g = fminf(f[i], gr.limit);
-              const float w = fminf(fmaxf(__uint_as_float(u[i]), -gr.limit), gr.limit);
-              f[i] = row_w * (g / (1.0f + expf(-1.702f * g))) * (w + 1.0f);
+              if (gr.limit < 0.f) {                  // silu(g) u, without clamps
+                f[i] = row_w * silu(f[i]) * __uint_as_float(u[i]);
+              } else {
+                const float g = fminf(f[i], gr.limit);
+                const float w = fminf(fmaxf(__uint_as_float(u[i]), -gr.limit), gr.limit);
+                f[i] = row_w * (g / (1.0f + expf(-1.702f * g))) * (w + 1.0f);
+              }
             }
             if (EPI == EPI_RELU2) {
               // as the unfused path rounds: the product to bfloat16 first, then the square of its positive part

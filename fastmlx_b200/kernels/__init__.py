@@ -340,7 +340,7 @@ def paged_attention_simple(qkv, kv, ctx, group, nh, nkv, hd, scale, window) -> t
 
 def qk_prepare(qkv, positions, inv_freq, rotary_dim, traditional, norm_eps, slot_mapping, kv, nh, nkv, hd, vd,
                status, bias=None, q_weight=None, k_weight=None, norm_first: bool = False, whole: bool = False,
-               values_from_keys: bool = False) -> torch.Tensor:
+               values_from_keys: bool = False, amplitude: float = 1.0, v_scale: float = 1.0) -> torch.Tensor:
     """Queries and keys of qkv[T, nh*hd + nkv*hd + nkv*vd] made ready for attention: rotated over their
     first `rotary_dim` dimensions, then (norm_eps not None) each head divided by its root mean square;
     keys and values are stored at slot_mapping in pages that hold [nkv, page, hd] keys and then
@@ -349,7 +349,8 @@ def qk_prepare(qkv, positions, inv_freq, rotary_dim, traditional, norm_eps, slot
     first; `q_weight` / `k_weight` ([hd], 32-bit) multiply the normalised heads; `norm_first` normalises
     before the rotation instead of after it.  `whole` (with `norm_first`): q and k are each divided by the root mean
     square of their whole projection, all heads at once, and the weights are that wide ([nh*hd], [nkv*hd]);
-    `values_from_keys`: qkv holds q | k only, and a token's values are its keys as projected (vd = hd)."""
+    `values_from_keys`: qkv holds q | k only, and a token's values are its keys as projected (vd = hd).  `amplitude`
+    multiplies the rotation's cosines and sines, `v_scale` the values on their way into the cache, both in 32-bit."""
     _need_cuda(qkv, positions, inv_freq, slot_mapping, kv, bias, q_weight, k_weight)
     assert qkv.dim() == 2 and qkv.stride(1) == 1 and positions.dtype == torch.int32
     T = qkv.shape[0]
@@ -368,13 +369,13 @@ def qk_prepare(qkv, positions, inv_freq, rotary_dim, traditional, norm_eps, slot
              _ptr(slot_mapping), q.data_ptr(), _ptr(kv), T, nh, nkv if kv is not None else 0, hd, vd, int(rotary_dim),
              int(bool(traditional)), -1.0 if norm_eps is None else float(norm_eps), page_size, num_pages, _dt(qkv),
              _dt(kv) if kv is not None else _dt(qkv), _ptr(bias), _ptr(q_weight), _ptr(k_weight), int(bool(values_from_keys)),
-             _ptr(status), _stream())
+             float(amplitude), float(v_scale), _ptr(status), _stream())
         return q
     call("common", "fmx_qk_prepare_ex", qkv.data_ptr(), qkv.stride(0), positions.data_ptr(), _ptr(inv_freq),
          _ptr(slot_mapping), q.data_ptr(), _ptr(kv), T, nh, nkv if kv is not None else 0, hd, vd, int(rotary_dim),
          int(bool(traditional)), -1.0 if norm_eps is None else float(norm_eps), page_size, num_pages, _dt(qkv),
          _dt(kv) if kv is not None else _dt(qkv), _ptr(bias), _ptr(q_weight), _ptr(k_weight), int(bool(norm_first)),
-         _ptr(status), _stream())
+         float(amplitude), float(v_scale), _ptr(status), _stream())
     return q
 
 
@@ -447,32 +448,38 @@ def wide_attention_splits(rows: int, nkv: int, keys: int, device=None, hd: int =
 
 
 def wide_attention_takes(q, kv, hd, vd, out=None) -> bool:
-    """`wide_attention_ok` for pages in either layout (keys and values, or keys that are the values too) and an
-    output that may be a slice of a wider buffer."""
-    return (kv is not None and kv.dtype == torch.bfloat16 and kv.dim() == 5 and q.dtype == torch.float32 and hd == vd
-            and hd % 16 == 0 and hd <= 256 and q.stride(0) % 2 == 0 and q.data_ptr() % 8 == 0
-            and (out is None or (out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0)))
+    """`wide_attention_ok` for pages in any layout (keys and values of equal or different widths, or keys that are the
+    values too) and an output that may be a slice of a wider buffer."""
+    return (kv is not None and kv.dtype == torch.bfloat16 and kv.dim() == (5 if hd == vd else 2) and q.dtype == torch.float32
+            and hd % 16 == 0 and hd <= 256 and vd % 16 == 0 and vd <= 256 and q.stride(0) % 2 == 0 and q.data_ptr() % 8 == 0
+            and kv.data_ptr() % 16 == 0 and (out is None or (out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0)))
+
+
+def wide_library(hd: int, vd: int) -> str:
+    return f"attn_hd{hd}" if hd == vd else f"attn_hd{hd}_vd{vd}"
 
 
 def _wide_launch(q, kv, ctx, group, nh, nkv, hd, scale, softcap, window, out, first_token: int = 0, splits: int = 1,
-                 keep_first: int = 0, chunk: int = 0, sinks=None) -> None:
+                 keep_first: int = 0, chunk: int = 0, sinks=None, vd: int = 0) -> None:
+    vd = vd or hd
     bt = group.block_tables
+    page_size = kv.shape[3] if kv.dim() == 5 else kv.shape[1] // (nkv * (hd + vd))
     scratch = None
     n_tokens = ctx.R
     if splits > 1:
-        scratch = attention_scratch(q.device, (first_token + n_tokens) * nh * splits * (hd + 2))
-    call(f"attn_hd{hd}", "fmx_attn_prefill_wide_masked", q.data_ptr(), q.stride(0), kv.data_ptr(), bt.data_ptr(), bt.stride(0),
+        scratch = attention_scratch(q.device, (first_token + n_tokens) * nh * splits * (vd + 2))
+    call(wide_library(hd, vd), "fmx_attn_prefill_wide_masked", q.data_ptr(), q.stride(0), kv.data_ptr(), bt.data_ptr(), bt.stride(0),
          ctx.row_start.data_ptr(), ctx.row_ctx.data_ptr(), ctx.positions.data_ptr(), out.data_ptr(), out.stride(0), ctx.R,
-         int(ctx.max_q_len), nh, nkv, kv.shape[3], kv.shape[0], float(scale), float(softcap or 0.0), int(window),
+         int(ctx.max_q_len), nh, nkv, page_size, kv.shape[0], float(scale), float(softcap or 0.0), int(window),
          _ptr(ctx.status), _ptr(scratch), scratch.numel() if scratch is not None else 0, int(splits),
-         first_token + n_tokens, int(keep_first), int(kv.shape[1] == 1), int(chunk), _ptr(sinks), _stream())
+         first_token + n_tokens, int(keep_first), int(kv.dim() == 5 and kv.shape[1] == 1), int(chunk), _ptr(sinks), _stream())
     if splits > 1:
-        call(f"attn_hd{hd}", "fmx_attn_wide_combine_sinks", scratch.data_ptr(), out.data_ptr(), out.stride(0), int(first_token),
+        call(wide_library(hd, vd), "fmx_attn_wide_combine_sinks", scratch.data_ptr(), out.data_ptr(), out.stride(0), int(first_token),
              n_tokens, nh, int(splits), _ptr(sinks), _stream())
 
 
 def paged_attention_wide(q, kv, ctx, group, nh, nkv, hd, scale, softcap, window, out=None, keep_first: int = 0,
-                         gate=None, chunk: int = 0, sinks=None, gate_group: int = 1) -> torch.Tensor:
+                         gate=None, chunk: int = 0, sinks=None, gate_group: int = 1, vd: int = 0) -> torch.Tensor:
     """Attention of any mix of rows on the tensor cores with 32-bit scores and weights: the 32-bit queries
     q[T, nh*hd] and the probabilities enter the products as two bfloat16 terms each, sums are 32-bit, scores may be
     capped (softcap > 0).  `out` may be a slice of a wider buffer.  -> [T, nh*hd] in bfloat16.  The one-token rows
@@ -482,28 +489,31 @@ def paged_attention_wide(q, kv, ctx, group, nh, nkv, hd, scale, softcap, window,
     hold keys that are the values too; `gate` ([T, nh*hd / gate_group]): the output is multiplied by sigmoid(gate)
     afterwards, one gate value per `gate_group` elements.  `chunk` c > 0 instead of a window: keys are seen within runs
     of c positions counted from position 0; `sinks` (32-bit [nh]): one more term exp(sink) per head in the
-    denominator, with no value."""
+    denominator, with no value.  `vd` (0: hd): the values' head size; pages of another width than the keys' are [pages,
+    nkv * page * (hd + vd)], and the output is [T, nh*vd]."""
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == nh)
-    out = _paged_attention_wide(q, kv, ctx, group, nh, nkv, hd, scale, softcap, window, out, int(keep_first), int(chunk), sinks)
+    out = _paged_attention_wide(q, kv, ctx, group, nh, nkv, hd, scale, softcap, window, out, int(keep_first), int(chunk), sinks, int(vd or hd))
     if gate is not None:
         sigmoid_gate(out, gate, int(gate_group))
     return out
 
 
-def _paged_attention_wide(q, kv, ctx, group, nh, nkv, hd, scale, softcap, window, out, keep_first, chunk=0, sinks=None) -> torch.Tensor:
+def _paged_attention_wide(q, kv, ctx, group, nh, nkv, hd, scale, softcap, window, out, keep_first, chunk=0, sinks=None,
+                          vd: int = 0) -> torch.Tensor:
+    vd = vd or hd
     T = q.shape[0]
     if out is None:
-        out = torch.empty((T, nh * hd), dtype=torch.bfloat16, device=q.device)
+        out = torch.empty((T, nh * vd), dtype=torch.bfloat16, device=q.device)
     assert out.dtype == torch.bfloat16 and out.stride(1) == 1 and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0
     d = ctx.R if ctx.all_decode else getattr(ctx, "decode_rows", 0)
-    more = dict(chunk=chunk, sinks=sinks)
+    more = dict(chunk=chunk, sinks=sinks, vd=vd)
     if d <= 0:
         _wide_launch(q, kv, ctx, group, nh, nkv, hd, scale, softcap, window, out, keep_first=keep_first, **more)
         return out
     longest = ctx.max_ctx_after if ctx.all_decode else ctx.decode_max_ctx
     keys = min(window + keep_first, longest) if window > 0 else (min(chunk, longest) if chunk > 0 else longest)
-    splits = wide_attention_splits(d, nkv, keys, q.device, hd)
-    if splits > 1 and d * nh * splits * (hd + 2) > ATTN_SCRATCH_FLOATS:
+    splits = wide_attention_splits(d, nkv, keys, q.device, max(hd, vd))
+    if splits > 1 and d * nh * splits * (vd + 2) > ATTN_SCRATCH_FLOATS:
         splits = 1
     if ctx.all_decode:
         _wide_launch(q, kv, ctx, group, nh, nkv, hd, scale, softcap, window, out, 0, splits, keep_first, **more)
@@ -766,6 +776,104 @@ def sigmoid_attention(q, kv, ctx, group, nh, nkv, hd, vd, scale, softcap, window
     return out
 
 
+# ----------------------------------------------------------------------------- decays per key channel, layer norm, capped logits
+def channel_delta_prepare(proj, b, z, conv_w, a_log, dt_bias, ctx, state, conv_off, H, G, D, Dv, taps):
+    """What the delta rule with a decay per key channel takes in: proj[T, >= C] holds q (G*D) | k (G*D) | v (H*Dv) channels,
+    b[T, H] (of proj's type, rows may be slices) the write strengths' and z[T, H*D] (32-bit) the decays' pre-activations.
+    Channels pass a causal convolution of `taps` taps (weights conv_w[C, taps]; inputs before a portion's start come
+    from the request's state slot, which then takes the portion's last inputs) and SiLU; q and k become unit vectors per
+    head, q times D^-1/2.  -> (q | k | v in 32-bit [T, C], decays exp(-exp(A_log) softplus(z + dt_bias)) in 32-bit
+    [T, H*D], write strengths sigmoid(b) in 32-bit [T, H])."""
+    _need_cuda(proj, b, z, conv_w, a_log, dt_bias, state)
+    T = proj.shape[0]
+    C = 2 * G * D + H * Dv
+    assert proj.stride(1) == 1 and b.stride(1) == 1 and b.dtype == proj.dtype and z.dtype == torch.float32 and z.stride(1) == 1
+    assert conv_w.dtype == torch.float32 and conv_w.is_contiguous() and conv_w.shape == (C, taps) and dt_bias.numel() == H * D
+    assert state.dtype == torch.float32 and state.is_contiguous()
+    qkv = torch.empty((T, C), dtype=torch.float32, device=proj.device)
+    g = torch.empty((T, H * D), dtype=torch.float32, device=proj.device)
+    beta = torch.empty((T, H), dtype=torch.float32, device=proj.device)
+    call("chan", "fmx_channel_delta_prepare", proj.data_ptr(), proj.stride(0), b.data_ptr(), b.stride(0), z.data_ptr(), z.stride(0),
+         conv_w.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(), ctx.token_row.data_ptr(), ctx.row_start.data_ptr(),
+         ctx.row_slot.data_ptr(), state.data_ptr(), state.stride(0), int(conv_off), qkv.data_ptr(), g.data_ptr(), beta.data_ptr(),
+         T, ctx.R, H, G, D, Dv, int(taps), state.shape[0], int(ctx.max_q_len == 1), _dt(proj), _ptr(ctx.status), _stream())
+    return qkv, g, beta
+
+
+def channel_gla_prepare(proj, z, bias, H, D, Dv, q_scale: float, tau: float):
+    """What gated linear attention takes in: proj[T, q (H*D) | k (H*D) | v (H*Dv) ...] and z[T, H*D] (32-bit).
+    -> (q * q_scale | k | v in 32-bit, sigmoid(z + bias)^(1/tau) in 32-bit [T, H*D])."""
+    _need_cuda(proj, z, bias)
+    T = proj.shape[0]
+    assert proj.stride(1) == 1 and z.dtype == torch.float32 and z.stride(1) == 1
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == H * D)
+    qkv = torch.empty((T, 2 * H * D + H * Dv), dtype=torch.float32, device=proj.device)
+    g = torch.empty((T, H * D), dtype=torch.float32, device=proj.device)
+    call("chan", "fmx_channel_gla_prepare", proj.data_ptr(), proj.stride(0), z.data_ptr(), z.stride(0), _ptr(bias), qkv.data_ptr(),
+         g.data_ptr(), T, H, D, Dv, float(q_scale), 1.0 / float(tau), _dt(proj), _stream())
+    return qkv, g
+
+
+def channel_scan(qkv, g, beta, ctx, state, H, G, D, Dv, cpt: int = 0) -> torch.Tensor:
+    """Linear attention with a decay per key channel over every request's tokens of the step, in order, from and into the
+    requests' state slots (S^T per head, [H, Dv, D], at the head of a slot): S <- diag(g) S, then the delta rule's write
+    u = beta (v - S^T k), S <- S + k u^T, or with beta None S <- S + k v^T; o = S^T q.  qkv[T, q (G*D) | k (G*D) |
+    v (H*Dv)], g[T, H*D], beta[T, H], all 32-bit.  `cpt` (1, 2, 4; 0: the library's choice): columns of S that a group of
+    lanes holds.  -> o in 32-bit, [T, H*Dv]."""
+    T = qkv.shape[0]
+    assert qkv.is_contiguous() and g.is_contiguous() and (beta is None or beta.is_contiguous())
+    out = torch.empty((T, H * Dv), dtype=torch.float32, device=qkv.device)
+    call("chan", "fmx_channel_scan", qkv.data_ptr(), g.data_ptr(), _ptr(beta), ctx.row_start.data_ptr(), ctx.row_slot.data_ptr(),
+         state.data_ptr(), state.stride(0), out.data_ptr(), ctx.R, H, G, D, Dv, state.shape[0], int(ctx.max_q_len == 1), int(cpt),
+         _stream())
+    return out
+
+
+def head_norm_gate(o, gate, weight, eps, H, Dv, out_dtype, act: str = "sigmoid", out=None) -> torch.Tensor:
+    """o[T, H*Dv] (32-bit) per head divided by its root mean square, times weight[Dv], times sigmoid(gate) (act="silu":
+    silu(gate)); gate (of its own type) and out may be slices of wider buffers."""
+    T = o.shape[0]
+    if out is None:
+        out = torch.empty((T, H * Dv), dtype=out_dtype, device=o.device)
+    assert act in ("sigmoid", "silu") and o.is_contiguous() and gate.stride(1) == 1 and out.stride(1) == 1
+    assert gate.shape == (T, H * Dv) and out.shape == (T, H * Dv) and weight.dtype == torch.float32
+    call("chan", "fmx_head_norm_gate", o.data_ptr(), gate.data_ptr(), gate.stride(0), _dt(gate), weight.data_ptr(), out.data_ptr(),
+         out.stride(0), _dt(out), T, H, Dv, float(eps), int(act == "silu"), _stream())
+    return out
+
+
+def layernorm_step(y, post, mult, residual, pre, out_dtype, out=None):
+    """One pass over the stream: residual <- residual + mult * post(y), out = pre(residual), all 32-bit.  post and pre are
+    (weight, eps) of a layer norm, (x - mean) / sqrt(variance + eps) * weight, or None for the identity; pre False:
+    nothing but the stream is written.  y (bfloat16 or 32-bit, rows may be a slice) may be None; residual None: the
+    stream starts at zero and gets an array of its own.  -> (out or None, residual)."""
+    ref = y if y is not None else residual
+    _need_cuda(y, residual, out)
+    assert ref is not None and ref.dim() == 2 and (y is None or y.stride(1) == 1)
+    rows, cols = ref.shape
+    assert residual is None or (residual.dtype == torch.float32 and residual.is_contiguous() and residual.shape == ref.shape)
+    res_in = residual
+    if residual is None:
+        residual = torch.empty((rows, cols), dtype=torch.float32, device=ref.device)
+    want_out = pre is not False
+    if want_out and out is None:
+        out = torch.empty((rows, cols), dtype=out_dtype, device=ref.device)
+    pw, pe = post if post else (None, 0.0)
+    qw, qe = pre if pre else (None, 0.0)
+    call("common", "fmx_layernorm_step", _ptr(y), y.stride(0) if y is not None else 0, _dt(y) if y is not None else F32, _ptr(pw),
+         float(pe), float(mult), _ptr(res_in), residual.data_ptr(), _ptr(qw), float(qe), _ptr(out) if want_out else None,
+         out.stride(0) if want_out else 0, _dt(out) if want_out else F32, rows, cols, _stream())
+    return (out if want_out else None), residual
+
+
+def logit_cap(x, scale: float, cap: float) -> torch.Tensor:
+    """x <- cap tanh(x scale / cap) (cap 0: x scale) in place, in 32-bit."""
+    _need_cuda(x)
+    assert x.dim() == 2 and x.dtype == torch.float32 and x.stride(1) == 1
+    call("common", "fmx_logit_cap", x.data_ptr(), x.stride(0), x.shape[0], x.shape[1], float(scale), float(cap or 0.0), _stream())
+    return x
+
+
 # ----------------------------------------------------------------------------- dynamic tanh, latents, gates, routed experts
 def dyt_step(y, post, mult, add, residual, pre, out_dtype, out=None, keep_stream: bool = True):
     """One pass over the stream: residual <- residual + mult * post(y) + add, out = pre(residual), all 32-bit.
@@ -822,21 +930,23 @@ def sigmoid_gate(o, gate, group: int = 1):
 
 
 def moe_route(logits, top: int, groups: int = 1, keep: int = 1, want_chosen: bool = False, experts: int | None = None,
-              correction=None, scale: float = 1.0):
+              correction=None, scale: float = 1.0, logit_bias=None, renorm: bool = False):
     """Router logits [T, E] (32-bit) -> weights [T, E] (32-bit): the softmax score where an expert is among the token's
     `top` best of the `keep` best groups (of `groups` groups of neighbours, each scored by its best member), else zero;
     not renormalised.  With `want_chosen` also the chosen indices, int32 [T, top].  `experts`: the row's first that many
     columns are the experts' logits (a row may hold other columns behind them).  `correction` (32-bit [E]): added to the
-    scores for the choice only; `scale` multiplies the chosen experts' scores."""
-    _need_cuda(logits, correction)
+    scores for the choice only; `scale` multiplies the chosen experts' scores.  `logit_bias` (32-bit [E]): added to the
+    logits; `renorm`: the weights are the softmax over the chosen logits alone."""
+    _need_cuda(logits, correction, logit_bias)
+    assert logit_bias is None or (logit_bias.dtype == torch.float32 and logit_bias.is_contiguous())
     assert logits.dim() == 2 and logits.dtype == torch.float32 and logits.stride(1) == 1
     T, E = logits.shape[0], int(experts if experts is not None else logits.shape[1])
     assert E <= logits.shape[1] and (correction is None or (correction.dtype == torch.float32 and correction.numel() == E
                                                              and correction.is_contiguous()))
     w = torch.empty((T, E), dtype=torch.float32, device=logits.device)
     chosen = torch.empty((T, top), dtype=torch.int32, device=logits.device) if want_chosen else None
-    call("common", "fmx_moe_route_biased", logits.data_ptr(), logits.stride(0), T, E, int(top), int(groups), int(keep),
-         w.data_ptr(), _ptr(chosen), _ptr(correction), float(scale), _stream())
+    call("common", "fmx_moe_route_ex", logits.data_ptr(), logits.stride(0), T, E, int(top), int(groups), int(keep),
+         w.data_ptr(), _ptr(chosen), _ptr(correction), float(scale), _ptr(logit_bias), int(bool(renorm)), _stream())
     return (w, chosen) if want_chosen else w
 
 
@@ -860,7 +970,8 @@ def moe_expert_act(gu, weights, E: int, ff: int, limit: float, limit_shared: flo
     """The experts' hidden layers side by side: gu[T, 2F] holds F gates then F ups, F = E*ff + the shared expert's
     width; -> [T, F]: w * g' sigmoid(1.702 g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit), w the
     token's weight for the column's expert (1 for the shared columns at the end), zero where it chose it not.
-    `block` > 0: gu holds gates and ups in alternating blocks of that many instead."""
+    `block` > 0: gu holds gates and ups in alternating blocks of that many instead.  A negative limit (SILU_EXPERTS) names the
+    other form, w * silu(g) * u without clamps, here and in the grouped products below."""
     _need_cuda(gu, weights)
     assert gu.dim() == 2 and gu.stride(1) == 1 and gu.shape[1] % 2 == 0 and weights.dtype == torch.float32
     T, F = gu.shape[0], gu.shape[1] // 2
@@ -870,6 +981,9 @@ def moe_expert_act(gu, weights, E: int, ff: int, limit: float, limit_shared: flo
     call("common", "fmx_moe_expert_act", gu.data_ptr(), gu.stride(0), weights.data_ptr(), out.data_ptr(), out.stride(0), T,
          int(E), int(ff), F, float(limit), float(limit_shared), _dt(gu), int(block), _stream())
     return out
+
+
+SILU_EXPERTS = -1.0         # as an expert's limit: silu(g) * u, without clamps
 
 
 def can_expert_tc(x, w) -> bool:

@@ -42,8 +42,8 @@ _SIGNATURES = {
         "fmx_activation": [_P, _L, _P, _L, _I, _I, _I, _I, _P],
         "fmx_paged_attention_masked": [_P, _L, _I, _P, _P, _I, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _L, _F, _F, _I, _I,
                                        _I, _P, _I, _I, _P, _L, _P],
-        "fmx_qk_prepare_ex": [_P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _L, _I, _I, _P, _P, _P, _I, _P,
-                              _P],
+        "fmx_qk_prepare_ex": [_P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _L, _I, _I, _P, _P, _P, _I, _F,
+                              _F, _P, _P],
         "fmx_dyt_step": [_P, _L, _I, _F, _P, _P, _F, _P, _P, _P, _F, _P, _P, _P, _L, _I, _I, _I, _P],
         "fmx_rmsnorm_rows": [_P, _L, _I, _P, _F, _P, _L, _I, _P, _L, _I, _I, _P, _P],
         "fmx_sigmoid_gate": [_P, _L, _I, _P, _L, _I, _I, _I, _I, _P],
@@ -53,7 +53,7 @@ _SIGNATURES = {
         "fmx_paged_attention_masked_ex": [_P, _L, _I, _P, _P, _I, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _L, _F, _F, _I, _I,
                                           _I, _P, _I, _I, _P, _L, _I, _P, _I, _P],
         "fmx_qk_prepare_whole": [_P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _L, _I, _I, _P, _P, _P, _I,
-                                 _P, _P],
+                                 _F, _F, _P, _P],
         "fmx_latent_rope_prepare": [_P, _L, _I, _P, _L, _P, _P, _P, _F, _P, _P, _L, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P],
         "fmx_ssm_prepare": [_P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _L, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
         "fmx_ssm_scan": [_P, _P, _P, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _P],
@@ -62,6 +62,9 @@ _SIGNATURES = {
         "fmx_embed_scaled": [_P, _I, _P, _P, _I, _I, _L, _F, _P, _I, _P],
         "fmx_rmsnorm_pair_mean": [_P, _L, _P, _L, _I, _P, _P, _F, _P, _L, _I, _I, _I, _P],
         "fmx_moe_route_biased": [_P, _L, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P],
+        "fmx_moe_route_ex": [_P, _L, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P, _I, _P],
+        "fmx_layernorm_step": [_P, _L, _I, _P, _F, _F, _P, _P, _P, _F, _P, _L, _I, _I, _I, _P],
+        "fmx_logit_cap": [_P, _L, _I, _I, _F, _F, _P],
         "fmx_moe_plain_act": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _P],
         "fmx_retention_prepare": [_P, _L, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _P],
         "fmx_retention_gate_norm": [_P, _P, _L, _I, _P, _L, _I, _I, _I, _I, _F, _P],
@@ -82,6 +85,13 @@ _SIGNATURES = {
         "fmx_expert_tcgen05": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _F, _I, _P, _P],
         "fmx_grouped_tcgen05": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _P, _F, _I, _I, _P, _P],
     },
+    "chan": {
+        "fmx_channel_delta_prepare": [_P, _L, _P, _L, _P, _L, _P, _P, _P, _P, _P, _P, _P, _L, _L, _P, _P, _P, _I, _I, _I, _I, _I,
+                                      _I, _I, _I, _I, _I, _P, _P],
+        "fmx_channel_gla_prepare": [_P, _L, _P, _L, _P, _P, _P, _I, _I, _I, _I, _F, _F, _I, _P],
+        "fmx_channel_scan": [_P, _P, _P, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+        "fmx_head_norm_gate": [_P, _P, _L, _I, _P, _P, _L, _I, _I, _I, _I, _F, _I, _P],
+    },
     "mixattn": {
         "fmx_mixattn": [_P, _L, _P, _P, _I, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _L, _F, _F, _I, _I, _P, _P, _I, _I, _P, _P],
         "fmx_mixattn_plan": [_I, _I, _I, _I, _I, _I, _I],
@@ -101,6 +111,9 @@ _SIGNATURES = {
     },
 }
 
+# a library for values of another width than the keys holds the kernel with 32-bit queries alone
+_SIGNATURES["attn_vd"] = {n: _SIGNATURES["attn"][n] for n in ("fmx_attn_prefill_wide_masked", "fmx_attn_wide_combine_sinks")}
+
 _libs: dict[str, ctypes.CDLL] = {}
 launches = 0          # entry-point calls so far; each launches at least one kernel of this package
 
@@ -114,7 +127,8 @@ def load(group: str) -> ctypes.CDLL:
         lib = ctypes.CDLL(path)
     except (OSError, _build.BuildError) as e:
         raise KernelError(f"the CUDA library of group {group!r} is not available: {e}") from None
-    if group.startswith("attn_hd"):
+    values_differ = group.startswith("attn_hd") and "_vd" in group
+    if group.startswith("attn_hd") and not values_differ:
         lib.fmx_attn_decode_scratch_floats.argtypes = [_I, _I, _I]
         lib.fmx_attn_decode_scratch_floats.restype = c_longlong
         lib.fmx_attn_decode_plan.argtypes = [_I, _I, _L, _I]
@@ -129,7 +143,7 @@ def load(group: str) -> ctypes.CDLL:
         lib.fmx_gemm_tcgen05_plan_width.argtypes = [_I, _I, _I]
         lib.fmx_gemm_tcgen05_plan_fills.argtypes = [_I, _I, _I]
     lib.fmx_last_error.restype = ctypes.c_char_p
-    family = "attn" if group.startswith("attn_hd") else "tc" if group == "tc_expiry" else \
+    family = "attn_vd" if values_differ else "attn" if group.startswith("attn_hd") else "tc" if group == "tc_expiry" else \
         "mixattn" if group.startswith("mixattn_v") else group
     for name, args in _SIGNATURES.get(family, {}).items():
         fn = getattr(lib, name)

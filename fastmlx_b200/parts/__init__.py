@@ -1,17 +1,18 @@
 from .attention import GQAAttention
-from .base import (FeedForward, Mixer, Norm, PagedKVSpec, Part, PositionEncoding, Run, Runtime,
+from .base import (FeedForward, FreeDim, Mixer, Norm, PagedKVSpec, Part, PositionEncoding, Run, Runtime,
                    StateSpec, StreamEncoding, WeightSpec)
-from .block import MixerOnly, PairMixer, ParallelBlock, PreNormBlock, SandwichBlock
-from .delta import GatedDeltaMixer
+from .block import MixerOnly, PairMixer, ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
+from .delta import ChannelDeltaMixer, GatedDeltaMixer
 from .embedding import BigramEmbedding, Embedding, LMHead
-from .linear import JoinedLinear, Linear
+from .gla import GatedLinearAttention
+from .linear import BlockDiagonalLinear, JoinedLinear, Linear
 from .mlp import DenseMLP, SwiGLU
 from .model import Model
 from .latent import LatentAttention
 from .loop import LoopInput, LoopPass
 from .moe import PlainRoutedExperts, RoutedExperts
 from .retention import RetentionMixer
-from .norm import DynamicTanh, Pending, RMSNorm
+from .norm import DynamicTanh, LayerNorm, Pending, RMSNorm
 from .ssm import StateSpaceMixer
 from .rope import NoPositionEncoding, RotaryEmbedding, inverse_frequencies
 
@@ -19,4 +20,5 @@ __all__ = ["GQAAttention", "FeedForward", "Mixer", "Norm", "PagedKVSpec", "Part"
            "Run", "Runtime", "StateSpec", "StreamEncoding", "WeightSpec", "PreNormBlock", "Embedding", "LMHead", "Linear",
            "SwiGLU", "DenseMLP", "JoinedLinear", "ParallelBlock", "GatedDeltaMixer", "Model", "RMSNorm", "NoPositionEncoding", "RotaryEmbedding", "inverse_frequencies", "SandwichBlock", "LatentAttention", "LoopInput", "LoopPass", "RoutedExperts",
            "DynamicTanh", "Pending", "BigramEmbedding", "StateSpaceMixer", "PairMixer", "PlainRoutedExperts",
-           "RetentionMixer", "MixerOnly"]
+           "RetentionMixer", "MixerOnly", "FreeDim", "PostNormBlock", "ChannelDeltaMixer", "GatedLinearAttention", "BlockDiagonalLinear",
+           "LayerNorm"]

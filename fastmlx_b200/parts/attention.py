@@ -46,6 +46,10 @@ class GQAAttention(Mixer):
     head (`head_bias`: its tensor's name, or None for no number); nothing is normalised over the keys.  `head_mix` (a
     tensor's name, [heads, heads]): the heads' weights are mixed, w'_h = sum_g M[h, g] w_g, before head h applies them to
     the values of its own key/value head.  Scores, weights and their sums over the keys are 32-bit.
+
+    `value_scale`: the values are multiplied by it, in 32-bit, before they are stored, and with them the heads' outputs
+    (`scale_output` sets it; a block that scales its mixers uses that).  A rotation whose cosines and sines have an
+    amplitude (`pos.amplitude`) takes this route too.
     """
 
     supports_cuda_graph = True
@@ -59,7 +63,7 @@ class GQAAttention(Mixer):
                  qk_norm_first: bool = False, keep_first: int = 0, gate: str | None = None, late_bias: bool = False,
                  out_bias: bool | None = None, values_from_keys: bool = False, qk_norm_whole: bool = False,
                  chunk: int = 0, sink: float | None = None, gate_per_head: bool = False, weights: str = "softmax",
-                 head_bias: str | None = None, head_mix: str | None = None):
+                 head_bias: str | None = None, head_mix: str | None = None, value_scale: float = 1.0):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are no multiple of {num_kv_heads} kv heads")
         self.nh, self.nkv, self.hd = int(num_heads), int(num_kv_heads), int(head_dim)
@@ -95,11 +99,14 @@ class GQAAttention(Mixer):
             raise ValueError("a weight or an order for the q/k norm needs its eps")
         self.general = (self.softcap > 0 or self.qk_norm_eps is not None or self.vd != self.hd or self.keep_first > 0
                         or self.gate_name is not None or self.late_bias or self.values_from_keys or self.chunk > 0
-                        or self.sink is not None or self.sigmoid)
+                        or self.sink is not None or self.sigmoid or pos.amplitude != 1.0)
         self.scale = float(scale) if scale is not None else float(head_dim) ** -0.5
         self.window = int(window)
         self.share_kv = bool(share_kv)
         self.pos = pos
+        self.value_scale = 1.0
+        if value_scale != 1.0:
+            self.scale_output(value_scale)
         qn, kn, vn, on = (f"{name}.{p}" for p in proj_names)
         outs = [(qn, self.nh * self.hd)]
         if not share_kv:
@@ -142,6 +149,13 @@ class GQAAttention(Mixer):
                 torch.eye(self.nh, dtype=torch.float32, device=rt.device)
             self.head_bias = to_f32_vector(tensors[self.head_bias_name], rt) if self.head_bias_name else None
 
+    def scale_output(self, s: float) -> None:
+        """The heads' outputs are multiplied by s: their values are, on the way into the cache."""
+        if self.share_kv:
+            raise ValueError("a layer that reads another's cache cannot scale its values")
+        self.value_scale = float(s)
+        self.general = self.general or self.value_scale != 1.0
+
     def weight_bytes(self):
         return super().weight_bytes() + 4 * (len(self.bias_names) and self.qkv_features)
 
@@ -170,6 +184,9 @@ class GQAAttention(Mixer):
         g = ctx.groups[cache.group]
         store = cache.writable and not self.share_kv
         more = dict(whole=True, values_from_keys=self.values_from_keys) if self.qk_norm_whole or self.values_from_keys else {}
+        if self.pos.amplitude != 1.0 or self.value_scale != 1.0:
+            more.update(amplitude=self.pos.amplitude, v_scale=self.value_scale)
+        wide = dict(vd=self.vd) if self.vd != self.hd else {}
         q = k.qk_prepare(qkv, ctx.positions, inv_freq, rot, trad, self.qk_norm_eps, g.slot_mapping if store else None,
                          cache.kv if store else None, self.nh, self.nkv, self.hd, self.vd, ctx.status,
                          **(dict(bias=self.row_bias, q_weight=self.q_weight, k_weight=self.k_weight,
@@ -185,7 +202,7 @@ class GQAAttention(Mixer):
             wide_ex = getattr(k, "wide_attention_takes", None) if getattr(k, "WIDE_HAS_SINKS", False) else None
             if wide_ex is not None and wide_ex(q, cache.kv, self.hd, self.vd, out):
                 return k.paged_attention_wide(q, cache.kv, ctx, g, self.nh, self.nkv, self.hd, self.scale, self.softcap,
-                                              self.window, out=out, keep_first=self.keep_first, **opts)
+                                              self.window, out=out, keep_first=self.keep_first, **opts, **wide)
             return k.paged_attention_general(q, cache.kv, ctx, g, self.nh, self.nkv, self.hd, self.vd, self.scale,
                                              self.softcap, self.window, g.page_size, out=out, keep_first=self.keep_first,
                                              **opts)
@@ -193,16 +210,15 @@ class GQAAttention(Mixer):
             wide_ex = getattr(k, "wide_attention_takes", None)
             if wide_ex is not None and wide_ex(q, cache.kv, self.hd, self.vd, out):
                 return k.paged_attention_wide(q, cache.kv, ctx, g, self.nh, self.nkv, self.hd, self.scale, self.softcap,
-                                              self.window, out=out, keep_first=self.keep_first, gate=gate)
+                                              self.window, out=out, keep_first=self.keep_first, gate=gate, **wide)
             return k.paged_attention_general(q, cache.kv, ctx, g, self.nh, self.nkv, self.hd, self.vd, self.scale,
                                              self.softcap, self.window, g.page_size, out=out, keep_first=self.keep_first,
                                              gate=gate)
-        wide = getattr(k, "wide_attention_ok", None)
-        if wide is not None and wide(q, cache.kv, self.hd, self.vd) and (out is None or (out.stride(0) % 2 == 0
-                                                                                         and out.data_ptr() % 4 == 0)):
+        takes = getattr(k, "wide_attention_takes", None)
+        if takes is not None and takes(q, cache.kv, self.hd, self.vd, out):
             # bfloat16 pages: the tiled tensor-core kernel, queries and weights as two bfloat16 terms each
             return k.paged_attention_wide(q, cache.kv, ctx, g, self.nh, self.nkv, self.hd, self.scale, self.softcap,
-                                          self.window, out=out)
+                                          self.window, out=out, **wide)
         return k.paged_attention_general(q, cache.kv, ctx, g, self.nh, self.nkv, self.hd, self.vd, self.scale,
                                          self.softcap, self.window, g.page_size, out=out)
 

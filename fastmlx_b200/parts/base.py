@@ -19,10 +19,22 @@ from typing import Any, Sequence
 import torch
 
 
+class FreeDim(int):
+    """A size in a `WeightSpec` that the configuration does not name and the checkpoint's tensors give (the rank of a
+    low-rank projection): dimensions with the same `key` must agree.  The integer itself is the size where tensors are
+    made up (random weights)."""
+    key: str
+
+    def __new__(cls, value: int, key: str):
+        d = super().__new__(cls, value)
+        d.key = key
+        return d
+
+
 @dataclass(frozen=True)
 class WeightSpec:
     """One checkpoint tensor: `kind` picks the random init (matrix, embedding and bias
-    N(0, 0.02); norm 1 + N(0, 0.02))."""
+    N(0, 0.02); norm 1 + N(0, 0.02)).  An entry of `shape` may be a `FreeDim`."""
     name: str
     shape: tuple[int, ...]
     kind: str = "matrix"
@@ -193,7 +205,9 @@ class Norm(Part):
 
 class PositionEncoding(Part):
     """Puts positions into the projected q and k of an attention mixer and stores k and v
-    in the layer's pages (one fused kernel)."""
+    in the layer's pages (one fused kernel).  `amplitude`: what cosines and sines are multiplied by."""
+
+    amplitude = 1.0
 
     def apply_and_store(self, qkv, ctx, cache, nh: int, nkv: int, hd: int) -> None:  # pragma: no cover
         raise NotImplementedError

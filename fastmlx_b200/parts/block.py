@@ -5,7 +5,7 @@ import torch
 
 from .base import FeedForward, Mixer, Norm, Part, WeightSpec, to_f32_vector
 from .linear import JoinedLinear, Linear
-from .norm import Pending
+from .norm import Pending, settle
 
 
 class PreNormBlock(Part):
@@ -136,10 +136,47 @@ class SandwichBlock(Part):
         return Pending(self.ffn.forward(h, ctx), self.norm2b, self.mult), residual
 
 
+class PostNormBlock(Part):
+    """x <- x + norm1(mixer(x)); x <- x + norm2(ffn(x)): the sublayers read the stream itself, and a norm stands behind
+    each of them only.  `ffn` (with its norm) may be None.
+
+    The block hands its last sublayer's output on as a `Pending` sum: the norm behind a sublayer, the sum into the 32-bit
+    stream and the copy of the stream that the next sublayer reads are one kernel, as with `SandwichBlock`."""
+
+    def __init__(self, mixer: Mixer, ffn: FeedForward | None, norm1: Norm, norm2: Norm | None):
+        if ffn is not None and norm2 is None:
+            raise ValueError("a feed-forward needs the norm behind it")
+        self.mixer, self.ffn, self.norm1, self.norm2 = mixer, ffn, norm1, norm2
+
+    def children(self):
+        return (self.mixer, self.norm1) + ((self.ffn, self.norm2) if self.ffn is not None else ())
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    def state_spec(self):
+        return self.mixer.state_spec()
+
+    @property
+    def supports_cuda_graph(self):
+        return bool(getattr(self.mixer, "supports_cuda_graph", False)) and \
+            bool(getattr(self.ffn, "supports_cuda_graph", True))
+
+    def forward(self, delta, residual, ctx, cache):
+        h, residual = settle(delta, residual, self.rt, out_dtype=self.rt.dtype)
+        pending = Pending(self.mixer.forward(h, ctx, cache), self.norm1)
+        if self.ffn is None:
+            return pending, residual
+        h, residual = settle(pending, residual, self.rt, out_dtype=self.rt.dtype)
+        return Pending(self.ffn.forward(h, ctx), self.norm2), residual
+
+
 class PairMixer(Mixer):
-    """Two mixers side by side on the same input: mixer(x) = (N_l(left(x)) + N_r(right(x))) / 2, each branch's output
+    """Two mixers side by side on the same input.  Either mixer(x) = (N_l(left(x)) + N_r(right(x))) / 2, each branch's output
     divided by its root mean square over the model width and multiplied by a plain weight of its own (`norm_names`:
-    the two tensors, under `name`) before the two are averaged, in 32-bit.
+    the two tensors, under `name`) before the two are averaged, in 32-bit; or, with `scales` = (s_l, s_r), mixer(x) =
+    s_l left(x) + s_r right(x): the branches (built with `output=False`, each with `scale_output`) multiply what they hand on,
+    and their output projections are one joined product that adds the two inside its 32-bit accumulators.
 
     The branches' input projections run as one product over x (their matrices are stacked at bind time and each
     branch is handed its slice, in 32-bit); either branch may keep pages and either a state slot, which the layer's
@@ -147,9 +184,14 @@ class PairMixer(Mixer):
     projection `o`; `left` takes its slice as `qkv` (a `GQAAttention`), `right` as `proj` (a `RetentionMixer`)."""
 
     def __init__(self, width: int, left: Mixer, right: Mixer, norm_eps: float, name: str,
-                 norm_names=("left.out", "right.out"), weight_suffix: str = ""):
+                 norm_names=("left.out", "right.out"), weight_suffix: str = "", scales=None):
         self.width, self.left, self.right, self.eps = int(width), left, right, float(norm_eps)
-        self.norm_tensors = tuple(f"{name}.{n}" for n in norm_names)
+        self.norm_tensors = () if scales is not None else tuple(f"{name}.{n}" for n in norm_names)
+        self.out = None
+        if scales is not None:
+            left.scale_output(scales[0])
+            right.scale_output(scales[1])
+            self.out = JoinedLinear(width, [left.out_piece, right.out_piece], bias_scales=scales)
         if left.cache_spec() is not None and right.cache_spec() is not None:
             raise ValueError("at most one branch keeps pages")
         if left.state_spec() is not None and right.state_spec() is not None:
@@ -165,16 +207,17 @@ class PairMixer(Mixer):
         return bool(getattr(self.left, "supports_cuda_graph", False)) and bool(getattr(self.right, "supports_cuda_graph", False))
 
     def children(self):
-        return (self.proj, self.left, self.right)
+        return tuple(p for p in (self.proj, self.left, self.right, self.out) if p is not None)
 
     def own_weight_specs(self):
         return [WeightSpec(n, (self.width,), "norm") for n in self.norm_tensors]
 
     def bind_own(self, tensors, rt):
-        self.w_left, self.w_right = (to_f32_vector(tensors[n], rt) for n in self.norm_tensors)
+        if self.norm_tensors:
+            self.w_left, self.w_right = (to_f32_vector(tensors[n], rt) for n in self.norm_tensors)
 
     def weight_bytes(self):
-        return super().weight_bytes() + 8 * self.width
+        return super().weight_bytes() + (8 * self.width if self.norm_tensors else 0)
 
     def cache_spec(self):
         return self.left.cache_spec() or self.right.cache_spec()
@@ -183,6 +226,13 @@ class PairMixer(Mixer):
         return self.left.state_spec() or self.right.state_spec()
 
     def forward(self, x, ctx, cache):
+        if self.out is not None:
+            proj = self.proj.forward(x)
+            joined = torch.empty((x.shape[0], self.out.in_features), dtype=self.rt.dtype, device=x.device)
+            m = self.left.inner_features
+            self.left.forward_inner(x, ctx, cache, qkv=proj[:, :self.split], out=joined[:, :m])
+            self.right.forward_inner(x, ctx, cache, proj=proj[:, self.split:], out=joined[:, m:])
+            return self.out.forward(joined)
         proj = self.proj.forward(x, out_dtype=torch.float32)
         a = self.left.forward_inner(x, ctx, cache, qkv=proj[:, :self.split])
         b = self.right.forward_inner(x, ctx, cache, proj=proj[:, self.split:])

@@ -91,13 +91,14 @@ class LMHead(Part):
     logits are wanted reach it."""
 
     def __init__(self, vocab: int, width: int, name: str | None, tied: Embedding | None = None,
-                 suffix: str = ".weight", scale: float = 1.0):
-        """`scale`: a constant the logits are multiplied by (in 32-bit, after the product)."""
+                 suffix: str = ".weight", scale: float = 1.0, softcap: float = 0.0):
+        """`scale`: a constant the logits are multiplied by (in 32-bit, after the product); `softcap` c > 0: the scaled
+        logits are capped, c tanh(z / c)."""
         if (name is None) == (tied is None):
             raise ValueError("LMHead takes either a tensor name or an embedding to tie to")
         self.vocab, self.width, self.name, self.tied = int(vocab), int(width), name, tied
         self.tensor = None if name is None else name + suffix
-        self.scale = float(scale)
+        self.scale, self.softcap = float(scale), float(softcap or 0.0)
         self.weight = None
 
     def own_weight_specs(self):
@@ -114,6 +115,8 @@ class LMHead(Part):
     def forward(self, x):
         w = self.tied.weight if self.tied is not None else self.weight
         logits = self.rt.k.linear(x, w, None, torch.float32)
+        if self.softcap > 0:
+            return self.rt.k.logit_cap(logits, self.scale, self.softcap)
         if self.scale != 1.0:
             logits.mul_(self.scale)
         return logits
@@ -127,14 +130,14 @@ class LMHead(Part):
         k = self.rt.k
         w = self.tied.weight if self.tied is not None else self.weight
         if self.scale > 0 and hasattr(k, "can_greedy_head") and k.can_greedy_head(x, w):
-            return k.greedy_head(x, w)                # a positive scale does not change the choice
+            return k.greedy_head(x, w)                # a positive scale and a cap, which is monotonic, do not change the choice
         return k.argmax(self.forward(x))
 
     def emit_after(self, b, delta, stream, norm) -> None:
         """Native program: final norm, then the step's logits."""
         from ..engine.native import F32, LOGITS, NotNative, OP_LINEAR, _dt
-        if self.scale != 1.0:
-            raise NotNative("the native executor's head does not scale its logits")
+        if self.scale != 1.0 or self.softcap > 0:
+            raise NotNative("the native executor's head neither scales nor caps its logits")
         x, _ = norm.emit(b, delta, stream)
         w = self.tied.weight if self.tied is not None else self.weight
         b.op(OP_LINEAR, in0=x, out0=LOGITS, w=b.ptr(w), w_dtype=_dt(w.dtype), ldw=w.stride(0), n=self.vocab, k=self.width,

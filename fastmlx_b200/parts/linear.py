@@ -3,7 +3,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import Part, Runtime, WeightSpec, to_compute, to_f32_vector
+from .base import FreeDim, Part, Runtime, WeightSpec, to_compute, to_f32_vector
 
 
 class Linear(Part):
@@ -19,8 +19,8 @@ class Linear(Part):
         stacked in alternating blocks of b, so that a tile of 2b output columns holds b rows
         of the first and the matching b rows of the second."""
         self.in_features = int(in_features)
-        self.names = [(n, int(o)) for n, o in names]
-        self.out_features = sum(o for _, o in self.names)
+        self.names = [(n, o if isinstance(o, FreeDim) else int(o)) for n, o in names]
+        self.out_features = sum(o for _, o in self.names)         # (a `FreeDim`'s true size is known once bound)
         self.has_bias = bool(bias)
         self.interleave = int(interleave)
         self.wsfx, self.bsfx = weight_suffix, bias_suffix
@@ -47,6 +47,7 @@ class Linear(Part):
             if bs is not None:
                 bs = [torch.stack([v.view(-1, b) for v in bs], dim=1).reshape(-1)]
         self.weight = ws[0].contiguous() if len(ws) == 1 else torch.cat(ws, dim=0).contiguous()
+        self.out_features = self.weight.shape[0]
         if bs is not None:
             self.bias = torch.cat(bs).contiguous()
 
@@ -72,10 +73,12 @@ class JoinedLinear(Part):
     [W1 | W2 | ...]^T (+ b1 + b2 ...).  The sum of the products x_i W_i^T is then taken inside one
     product's 32-bit accumulators and rounded once: how a block whose sublayers run side by side adds
     its mixer's and its feed-forward's outputs.  `pieces`: (weight tensor name, in features, bias
-    tensor name or None); `offsets[i]` is where piece i's inputs start in a row of x."""
+    tensor name or None); `offsets[i]` is where piece i's inputs start in a row of x.  `bias_scales`: what each piece's
+    bias is multiplied by, in 32-bit (a block that scales its sublayers scales their inputs here and their biases so)."""
 
-    def __init__(self, out_features: int, pieces):
+    def __init__(self, out_features: int, pieces, bias_scales=None):
         self.out_features = int(out_features)
+        self.bias_scales = [1.0] * len(pieces) if bias_scales is None else [float(s) for s in bias_scales]
         self.pieces = [(w, int(k), b) for w, k, b in pieces]
         self.offsets, at = [], 0
         for _, k, _ in self.pieces:
@@ -95,7 +98,8 @@ class JoinedLinear(Part):
         if len({w.dtype for w in ws}) > 1:
             ws = [w.float() for w in ws]
         self.weight = ws[0].contiguous() if len(ws) == 1 else torch.cat(ws, dim=1).contiguous()
-        bs = [to_f32_vector(tensors[b], rt) for _, _, b in self.pieces if b is not None]
+        bs = [to_f32_vector(tensors[b], rt) * s if s != 1.0 else to_f32_vector(tensors[b], rt)
+              for (_, _, b), s in zip(self.pieces, self.bias_scales) if b is not None]
         self.bias = None
         if bs:
             total = bs[0]
@@ -108,3 +112,33 @@ class JoinedLinear(Part):
 
     def forward(self, x, out_dtype=None):
         return self.rt.k.linear(x, self.weight, self.bias, out_dtype or self.rt.dtype)
+
+
+class BlockDiagonalLinear(Part):
+    """Several matrices applied side by side, each to its own run of inputs: y = [W1 x1 | W2 x2 | ...] for x = [x1 | x2 |
+    ...], as one product with the matrices on the diagonal of a larger one (zeros elsewhere).  For the second halves
+    of low-rank projections, whose inputs are so narrow that one launch is worth more than the zeros cost.  `pieces`:
+    (weight tensor name, out features, in features); the in features may be `FreeDim`s.  `in_features` and
+    `out_features` are those of the whole once it is bound."""
+
+    def __init__(self, pieces):
+        self.pieces = list(pieces)
+        self.in_features = sum(k for _, _, k in self.pieces)
+        self.out_features = sum(o for _, o, _ in self.pieces)
+        self.weight = None
+
+    def own_weight_specs(self):
+        return [WeightSpec(n, (o, k), "matrix") for n, o, k in self.pieces]
+
+    def bind_own(self, tensors, rt: Runtime):
+        ws = [to_compute(tensors[n], rt) for n, _, _ in self.pieces]
+        if len({w.dtype for w in ws}) > 1:
+            ws = [w.float() for w in ws]
+        self.weight = ws[0].contiguous() if len(ws) == 1 else torch.block_diag(*ws).contiguous()
+        self.out_features, self.in_features = self.weight.shape
+
+    def weight_bytes(self):
+        return self.weight.numel() * self.weight.element_size()
+
+    def forward(self, x, out_dtype=None):
+        return self.rt.k.linear(x, self.weight, None, out_dtype or self.rt.dtype)

@@ -6,7 +6,7 @@ from typing import Sequence
 import torch
 
 from ..weights.loader import WeightError
-from .base import Norm, Part, Run, Runtime
+from .base import FreeDim, Norm, Part, Run, Runtime
 from dataclasses import replace
 
 from .embedding import Embedding, LMHead
@@ -76,8 +76,16 @@ class Model(Part):
         kept = {n: t for n, t in tensors.items() if not any(d in n for d in self.drop)}
         missing = sorted(n for n in specs if n not in kept)
         unexpected = sorted(n for n in kept if n not in specs)
-        wrong = sorted((n, tuple(kept[n].shape), specs[n].shape) for n in specs
-                       if n in kept and tuple(kept[n].shape) != tuple(specs[n].shape))
+        free: dict[str, int] = {}                      # sizes that only the tensors give: the first one met counts
+        wrong = []
+        for n in sorted(specs):
+            if n not in kept:
+                continue
+            got, want = tuple(kept[n].shape), tuple(specs[n].shape)
+            if len(got) == len(want):
+                want = tuple(free.setdefault(w.key, g) if isinstance(w, FreeDim) and g > 0 else w for g, w in zip(got, want))
+            if got != want:
+                wrong.append((n, got, want))
         if missing or unexpected or wrong:
             lines = ["checkpoint does not match the configuration:"]
             if missing:

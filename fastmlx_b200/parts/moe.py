@@ -16,6 +16,10 @@ class RoutedExperts(FeedForward):
     Expert (no biases): g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit), W_down (g sigmoid(1.702 g) (u + 1)).
     The shared expert has the same form with a width and a limit of its own and weight 1.
 
+    Other forms: `activation="silu"`: the experts are W_down (silu(W_gate x) * (W_up x)), without clamps; `router_bias`: a
+    tensor of one number per expert, added to the logits; `weights="chosen"` (without groups): the chosen experts' weights
+    are the softmax over their logits alone, so that they sum to one.
+
     Two ways to compute it, chosen once by size (`sparse`), neither of which loops on the host or makes a token's
     result depend on what else is in the batch, so that a decode step can be captured:
 
@@ -38,9 +42,15 @@ class RoutedExperts(FeedForward):
     def __init__(self, width: int, experts: int, top: int, ff: int, limit: float, name: str, groups: int = 1,
                  keep: int = 1, shared_ff: int = 0, shared_limit: float = 0.0, weight_suffix: str = "",
                  expert_prefix: str = "e", shared_name: str = "shared", router_name: str = "router",
-                 proj_names=("gate", "up", "down"), sparse: bool | None = None):
+                 proj_names=("gate", "up", "down"), sparse: bool | None = None, activation: str = "clamped",
+                 router_bias: str | None = None, weights: str = "scores"):
         """`sparse`: grouped products (True), all experts side by side (False), or by size (None): grouped where the
         experts' matrices together pass SPARSE_MIN_BYTES and more than twice as many experts exist as a token uses."""
+        if activation not in ("clamped", "silu") or weights not in ("scores", "chosen"):
+            raise ValueError(f"unknown activation {activation!r} or weights {weights!r}")
+        self.activation, self.renorm = activation, weights == "chosen"
+        if activation == "silu":
+            limit = shared_limit = -1.0                # how the kernels are told the form without clamps
         self.width, self.E, self.top, self.ff, self.limit = int(width), int(experts), int(top), int(ff), float(limit)
         self.groups, self.keep = max(1, int(groups)), max(1, int(keep))
         if self.E % self.groups or not 0 < self.top <= self.E:
@@ -56,11 +66,17 @@ class RoutedExperts(FeedForward):
         self.up_names = [(f"{p}.{u}{weight_suffix}", w) for p, w in zip(pre, widths)]
         self.down_names = [(f"{p}.{d}{weight_suffix}", w) for p, w in zip(pre, widths)]
         self.router_name = f"{name}.{router_name}{weight_suffix}"
+        self.router_bias_name = f"{name}.{router_bias}" if router_bias else None
+        self.router_bias = None
+        if self.renorm and self.groups > 1 and self.keep < self.groups:
+            raise ValueError("weights over the chosen logits alone come without groups")
         self.want_sparse = sparse
         self.sparse = False
 
     def own_weight_specs(self):
         specs = [WeightSpec(self.router_name, (self.E, self.width), "matrix")]
+        if self.router_bias_name:
+            specs.append(WeightSpec(self.router_bias_name, (self.E,), "bias"))
         specs += [WeightSpec(n, (w, self.width), "matrix") for n, w in self.gate_names + self.up_names]
         specs += [WeightSpec(n, (self.width, w), "matrix") for n, w in self.down_names]
         return specs
@@ -69,6 +85,7 @@ class RoutedExperts(FeedForward):
 
     def bind_own(self, tensors, rt: Runtime):
         self.router = to_compute(tensors[self.router_name], rt)
+        self.router_bias = to_f32_vector(tensors[self.router_bias_name], rt) if self.router_bias_name else None
         mats = [to_compute(tensors[n], rt) for n, _ in self.gate_names + self.up_names + self.down_names]
         can = (rt.dtype == torch.bfloat16 and all(m.dtype == torch.bfloat16 for m in mats) and self.width % 8 == 0
                and self.ff % 8 == 0 and rt.device.type == "cuda" and hasattr(rt.k, "moe_sort"))
@@ -117,10 +134,13 @@ class RoutedExperts(FeedForward):
         used = min(self.E, tokens * self.top)
         return e * (self.router.numel() + 3 * used * self.ff * self.width + 3 * self.shared_ff * self.width)
 
-    def route(self, x):
-        """-> the tokens' weights over the experts, 32-bit [T, E], zero where an expert is not chosen."""
+    def route(self, x, want_chosen: bool = False):
+        """-> the tokens' weights over the experts, 32-bit [T, E], zero where an expert is not chosen (with `want_chosen` also
+        the chosen indices)."""
         k = self.rt.k
-        return k.moe_route(k.linear(x, self.router, None, torch.float32), self.top, self.groups, self.keep)
+        more = dict(logit_bias=self.router_bias, renorm=self.renorm) if self.router_bias is not None or self.renorm else {}
+        return k.moe_route(k.linear(x, self.router, None, torch.float32), self.top, self.groups, self.keep, want_chosen=want_chosen,
+                           **more)
 
     def forward(self, x, ctx):
         k = self.rt.k
@@ -133,7 +153,7 @@ class RoutedExperts(FeedForward):
 
     def forward_grouped(self, x):
         k, T = self.rt.k, x.shape[0]
-        w, chosen = k.moe_route(k.linear(x, self.router, None, torch.float32), self.top, self.groups, self.keep, want_chosen=True)
+        w, chosen = self.route(x, want_chosen=True)
         plan = k.moe_sort(chosen, w)
         y = k.moe_grouped_gate_up(x, plan, self.gate_up, self.E, self.ff, self.limit, self.block)
         pairs = k.moe_grouped_down(y, plan, self.down, self.E, self.ff, stacked=bool(self.block), tokens=T)

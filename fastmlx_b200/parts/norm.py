@@ -1,4 +1,4 @@
-"""Norms with the residual sum fused in front of them: RMSNorm, and the dynamic tanh."""
+"""Norms with the residual sum fused in front of them: RMSNorm, layer norm, and the dynamic tanh."""
 from __future__ import annotations
 
 import torch
@@ -62,10 +62,10 @@ class RMSNorm(Norm):
 @dataclass
 class Pending:
     """A sublayer's output that is not in the stream yet: the stream is residual + mult * norm(x) + add, where
-    `norm` (a DynamicTanh or None) stands behind the sublayer and `add` is a vector or None.  A block hands this
-    on instead of a finished sum, so that the next norm's kernel does the sum in the same pass."""
+    `norm` (a DynamicTanh, a LayerNorm or None) stands behind the sublayer and `add` is a vector or None.  A block hands
+    this on instead of a finished sum, so that the next norm's kernel does the sum in the same pass."""
     x: torch.Tensor
-    norm: "DynamicTanh | None" = None
+    norm: "DynamicTanh | LayerNorm | None" = None
     mult: float = 1.0
     add: torch.Tensor | None = None
 
@@ -103,10 +103,43 @@ class DynamicTanh(Norm):
                                   self.rt.dtype, out=out)
 
 
+class LayerNorm(Norm):
+    """(x - mean) / sqrt(variance + eps) * w, no bias, the variance being the mean of the squared deviations; all in
+    32-bit.  `forward(x, residual)` takes for x a tensor (added to the stream as it is) or a `Pending` whose norm, if it has
+    one, is a layer norm too: one kernel norms the sublayer's output, adds it to the 32-bit stream and norms the sum."""
+
+    def __init__(self, width: int, eps: float, name: str, suffix: str = ".weight"):
+        self.width, self.eps, self.tensor = int(width), float(eps), name + suffix
+
+    def own_weight_specs(self):
+        return [WeightSpec(self.tensor, (self.width,), "norm")]
+
+    def bind_own(self, tensors, rt: Runtime):
+        self.weight = to_f32_vector(tensors[self.tensor], rt)
+
+    def weight_bytes(self):
+        return 4 * self.width
+
+    def args(self):
+        return (self.weight, self.eps)
+
+    def forward(self, x, residual):
+        p = x if isinstance(x, Pending) else Pending(x)
+        if isinstance(p.norm, DynamicTanh) or p.add is not None:
+            _, residual = settle(p, residual, self.rt)
+            p = Pending(None)
+        return self.rt.k.layernorm_step(p.x, p.norm.args() if p.norm is not None else None, p.mult, residual, self.args(),
+                                        self.rt.dtype)
+
+
 def settle(x, residual, rt: Runtime, out=None, out_dtype=None):
     """The stream with a pending output added, and (where `out_dtype` or `out` asks for it) a copy of the sum in
     the activations' type, e.g. into a slice of a wider buffer.  -> (copy or None, residual)."""
     p = x if isinstance(x, Pending) else Pending(x)
     want = out is not None or out_dtype is not None
+    if isinstance(p.norm, LayerNorm):
+        if p.add is not None:
+            raise ValueError("a vector beside an output that passes a layer norm is not built")
+        return rt.k.layernorm_step(p.x, p.norm.args(), p.mult, residual, None if want else False, out_dtype or rt.dtype, out=out)
     return rt.k.dyt_step(p.x, p.norm.args() if p.norm is not None else None, p.mult, p.add, residual,
                          None if want else False, out_dtype or rt.dtype, out=out)

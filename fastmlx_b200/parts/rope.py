@@ -5,6 +5,7 @@ import math
 
 import torch
 
+from ..config.llama import YarnScaling
 from .base import PositionEncoding, Runtime
 
 
@@ -17,11 +18,19 @@ def inverse_frequencies(rotary_dim: int, theta: float, scaling=None) -> torch.Te
     compute/testdata/llama_args.json:161-183, and never applies it) rescales by wavelength
     l_j = 2 pi / f_j: shorter than orig/high_freq_factor keeps f_j; longer than
     orig/low_freq_factor gives f_j/factor; between, with s = (orig/l_j - low)/(high - low),
-    (1 - s) f_j/factor + s f_j."""
+    (1 - s) f_j/factor + s f_j.  A `YarnScaling` blends by pair number instead: pair i keeps f_i up to lo and gets
+    f_i/factor from hi on, linear in between, lo and hi being the pairs that turn `fast` and `slow` times over the original
+    length, t(n) = dims ln(original / (2 pi n)) / (2 ln theta), rounded down and up and clipped to [0, dims - 1]."""
     j = torch.arange(0, rotary_dim, 2, dtype=torch.float64)
     f = torch.pow(torch.tensor(float(theta), dtype=torch.float64), -j / rotary_dim)
     if scaling is None:
         return f
+    if isinstance(scaling, YarnScaling):
+        def pair_of(turns):
+            return rotary_dim * math.log(scaling.original / (2 * math.pi * turns)) / (2 * math.log(theta))
+        lo, hi = max(math.floor(pair_of(scaling.fast)), 0), min(math.ceil(pair_of(scaling.slow)), rotary_dim - 1)
+        ramp = ((j / 2 - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return f / scaling.factor * ramp + f * (1.0 - ramp)
     orig = float(scaling.original_max_position_embeddings)
     lo, hi, factor = scaling.low_freq_factor, scaling.high_freq_factor, scaling.factor
     lam = 2 * math.pi / f
@@ -42,6 +51,7 @@ class RotaryEmbedding(PositionEncoding):
         if self.rotary_dim % 2 or not 0 <= self.rotary_dim <= self.head_dim:
             raise ValueError(f"rotary_dim {self.rotary_dim} must be even and at most head_dim {self.head_dim}")
         self.theta, self.scaling, self.traditional = float(theta), scaling, bool(traditional)
+        self.amplitude = float(getattr(scaling, "amplitude", 1.0))
         self.inv_freq = None
 
     def bind_own(self, tensors, rt: Runtime):
@@ -49,6 +59,8 @@ class RotaryEmbedding(PositionEncoding):
             .to(torch.float32).to(rt.device).contiguous()
 
     def apply_and_store(self, qkv, ctx, cache, nh, nkv, hd):
+        if self.amplitude != 1.0:
+            raise ValueError("a rotation with an amplitude runs on the route with 32-bit scores (qk_prepare)")
         g = ctx.groups[cache.group] if cache.kv is not None else None
         self.rt.k.rope_kv_write(
             qkv, ctx.positions, self.inv_freq, self.rotary_dim, self.traditional,

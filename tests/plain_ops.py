@@ -190,7 +190,8 @@ def _rotate(heads, positions, inv_freq, rotary_dim, traditional):
 
 
 def qk_prepare(qkv, positions, inv_freq, rotary_dim, traditional, norm_eps, slot_mapping, kv, nh, nkv, hd, vd, status,
-               bias=None, q_weight=None, k_weight=None, norm_first=False, whole=False, values_from_keys=False):
+               bias=None, q_weight=None, k_weight=None, norm_first=False, whole=False, values_from_keys=False, amplitude=1.0,
+               v_scale=1.0):
     T = qkv.shape[0]
     n_qk = (nh + nkv) * hd
     row = qkv[:, :n_qk + (0 if values_from_keys else nkv * vd)].to(F64)
@@ -213,8 +214,11 @@ def qk_prepare(qkv, positions, inv_freq, rotary_dim, traditional, norm_eps, slot
             return h / torch.sqrt(ms + norm_eps) * w
         return h / torch.sqrt((h * h).mean(-1, keepdim=True) + norm_eps) * w
 
-    heads = _rotate(norm(heads), positions, inv_freq, rotary_dim, traditional) if norm_first \
-        else norm(_rotate(heads, positions, inv_freq, rotary_dim, traditional))
+    def turn(h):
+        h = _rotate(h, positions, inv_freq, rotary_dim, traditional)
+        return torch.cat([h[..., :rotary_dim] * amplitude, h[..., rotary_dim:]], -1)
+
+    heads = turn(norm(heads)) if norm_first else norm(turn(heads))
     q = heads[:, :nh].reshape(T, nh * hd).to(torch.float32)
     if kv is not None and slot_mapping is not None and nkv:
         pages = kv.shape[0]
@@ -231,7 +235,7 @@ def qk_prepare(qkv, positions, inv_freq, rotary_dim, traditional, norm_eps, slot
             for g in range(nkv):
                 flat[pg, (g * ps + off) * hd:(g * ps + off + 1) * hd] = heads[t, nh + g].to(kv.dtype)
                 at = nkv * ps * hd + (g * ps + off) * vd
-                flat[pg, at:at + vd] = row[t, n_qk + g * vd:n_qk + (g + 1) * vd].to(kv.dtype)
+                flat[pg, at:at + vd] = (row[t, n_qk + g * vd:n_qk + (g + 1) * vd] * v_scale).to(kv.dtype)
     return q
 
 
@@ -333,9 +337,11 @@ def sigmoid_gate(o, gate, group=1):
     return o
 
 
-def moe_route(logits, top, groups=1, keep=1, want_chosen=False, experts=None, correction=None, scale=1.0):
+def moe_route(logits, top, groups=1, keep=1, want_chosen=False, experts=None, correction=None, scale=1.0, logit_bias=None,
+              renorm=False):
     T, E = logits.shape[0], int(experts if experts is not None else logits.shape[1])
-    s = torch.softmax(logits[:, :E].to(torch.float32), -1)
+    z = logits[:, :E].to(torch.float32) + (logit_bias if logit_bias is not None else 0.0)
+    s = torch.softmax(z, -1)
     pick = s if correction is None else s + correction.to(torch.float32)
     w = torch.zeros(T, E, dtype=torch.float32)
     chosen = torch.full((T, top), -1, dtype=torch.int32)
@@ -350,6 +356,8 @@ def moe_route(logits, top, groups=1, keep=1, want_chosen=False, experts=None, co
         for i, e in enumerate(order):
             w[t, e] = s[t, e] * scale
             chosen[t, i] = e
+        if renorm:                                 # the softmax over the chosen logits alone
+            w[t, order] = torch.softmax(z[t, order].to(F64), -1).to(torch.float32) * scale
     return (w, chosen) if want_chosen else w
 
 
@@ -457,6 +465,13 @@ def moe_expert_act(gu, weights, E, ff, limit, limit_shared=0.0, out=None, block=
         g, u = v[:, :, 0].reshape(T, F), v[:, :, 1].reshape(T, F)
     else:
         g, u = gu[:, :F].to(F64), gu[:, F:].to(F64)
+    if limit < 0:                                  # the form without clamps
+        w = torch.cat([weights.to(F64).repeat_interleave(ff, dim=1), torch.ones(T, F - E * ff, dtype=F64)], 1)
+        y = (w * _silu(g) * u).to(gu.dtype)
+        if out is not None:
+            out.copy_(y)
+            return out
+        return y
     lim = torch.full((F,), float(limit), dtype=F64)
     lim[E * ff:] = float(limit_shared)
     w = torch.ones(T, F, dtype=F64)
@@ -605,3 +620,100 @@ def act_mul(gate_up, kind, block=None):
     else:
         raise ValueError(kind)
     return (a * u).to(gate_up.dtype)
+
+
+# ----------------------------------------------------------------------------- decays per key channel, layer norm, capped logits
+def _softplus(z):
+    return torch.clamp(z, min=0) + torch.log1p(torch.exp(-z.abs()))
+
+
+def channel_delta_prepare(proj, b, z, conv_w, a_log, dt_bias, ctx, state, conv_off, H, G, D, Dv, taps):
+    T, C = proj.shape[0], 2 * G * D + H * Dv
+    qkv = torch.zeros(T, C, dtype=torch.float32)
+    w = conv_w.to(F64)
+    for r in range(ctx.R):
+        slot = int(ctx.row_slot[r])
+        a, e = int(ctx.row_start[r]), int(ctx.row_start[r + 1])
+        if slot < 0 or e <= a:
+            continue
+        hist = state[slot, conv_off:conv_off + (taps - 1) * C].to(F64).reshape(taps - 1, C)
+        u = torch.cat([hist, proj[a:e, :C].to(F64)], 0)
+        y = torch.stack([_silu((u[t:t + taps] * w.t()).sum(0)) for t in range(e - a)])
+        state[slot, conv_off:conv_off + (taps - 1) * C] = u[u.shape[0] - (taps - 1):].reshape(-1).to(torch.float32)
+        qk = y[:, :2 * G * D].reshape(e - a, 2 * G, D)
+        qk = qk / torch.sqrt((qk * qk).sum(-1, keepdim=True) + 1e-6)
+        qk[:, :G] *= D ** -0.5
+        qkv[a:e] = torch.cat([qk.reshape(e - a, -1), y[:, 2 * G * D:]], 1).to(torch.float32)
+    rate = torch.exp(a_log.to(F64)).repeat_interleave(D)
+    g = torch.exp(-rate * _softplus(z.to(F64) + dt_bias.to(F64))).to(torch.float32)
+    return qkv, g, torch.sigmoid(b.to(F64)).to(torch.float32)
+
+
+def channel_gla_prepare(proj, z, bias, H, D, Dv, q_scale, tau):
+    qkv = proj[:, :2 * H * D + H * Dv].to(F64).clone()
+    qkv[:, :H * D] *= q_scale
+    x = z.to(F64) + (bias.to(F64) if bias is not None else 0.0)
+    return qkv.to(torch.float32), (torch.sigmoid(x) ** (1.0 / tau)).to(torch.float32)
+
+
+def channel_scan(qkv, g, beta, ctx, state, H, G, D, Dv):
+    T, per = qkv.shape[0], H // G
+    out = torch.zeros(T, H * Dv, dtype=torch.float32)
+    x = qkv.to(F64)
+    for r in range(ctx.R):
+        slot = int(ctx.row_slot[r])
+        a, e = int(ctx.row_start[r]), int(ctx.row_start[r + 1])
+        if slot < 0 or e <= a:
+            continue
+        S = state[slot, :H * Dv * D].to(F64).reshape(H, Dv, D)                 # S^T of every head
+        for t in range(a, e):
+            q = x[t, :G * D].reshape(G, D).repeat_interleave(per, 0)
+            k = x[t, G * D:2 * G * D].reshape(G, D).repeat_interleave(per, 0)
+            u = x[t, 2 * G * D:].reshape(H, Dv)
+            S = S * g[t].to(F64).reshape(H, 1, D)
+            if beta is not None:
+                u = beta[t].to(F64)[:, None] * (u - (S * k[:, None, :]).sum(-1))
+            S = S + u[:, :, None] * k[:, None, :]
+            out[t] = (S * q[:, None, :]).sum(-1).reshape(-1).to(torch.float32)
+        state[slot, :H * Dv * D] = S.reshape(-1).to(torch.float32)
+    return out
+
+
+def head_norm_gate(o, gate, weight, eps, H, Dv, out_dtype, act="sigmoid", out=None):
+    T = o.shape[0]
+    v = o.to(F64).reshape(T, H, Dv)
+    v = (v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps) * weight.to(F64)).reshape(T, H * Dv)
+    z = gate.to(F64)
+    res = (v * (torch.sigmoid(z) if act == "sigmoid" else _silu(z))).to(out_dtype)
+    if out is not None:
+        out.copy_(res)
+        return out
+    return res
+
+
+def layernorm_step(y, post, mult, residual, pre, out_dtype, out=None):
+    def norm(v, w, eps):
+        d = v - v.mean(-1, keepdim=True)
+        return d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps) * w.to(F64)
+
+    ref = y if y is not None else residual
+    s = residual.to(F64) if residual is not None else torch.zeros(ref.shape, dtype=F64)
+    if y is not None:
+        s = s + mult * (norm(y.to(F64), *post) if post else y.to(F64))
+    if residual is None:
+        residual = s.to(torch.float32)
+    else:
+        residual.copy_(s.to(torch.float32))
+    if pre is False:
+        return None, residual
+    o = norm(residual.to(F64), *pre) if pre else residual.to(F64)
+    if out is not None:
+        out.copy_(o.to(out.dtype))
+        return out, residual
+    return o.to(out_dtype), residual
+
+
+def logit_cap(x, scale, cap):
+    v = x.to(F64) * scale
+    x.copy_((cap * torch.tanh(v / cap) if cap and cap > 0 else v).to(x.dtype))
+    return x

@@ -31,9 +31,11 @@ delta rule layers to one layer of capped sliding-window attention, a dense feed-
 the Llama layers: a 2,048-token prompt whole and in portions of 512, and steady decoding at batch 8 and 64.
 `--design-set llama,medirax,gekavik` chooses the designs; a Gekavik model of those sizes has windowed attention that
 keeps the first tokens, latent attention in every fourth layer, and a mixture of 32 experts (4 per token and a shared
-one) whose active parameters equal the Llama layer's; `sorupel` and `kafepel` name the other two designs (a Kafepel model of
+one) whose active parameters equal the Llama layer's; `sorupel`, `kafepel` and `bonerax` name the other designs (a Kafepel model of
 those sizes: sigmoid attention with mixed heads beside a retention in every layer, gated feed-forwards alternating with a
-mixture of 8 squared-relu experts and a gated shared one).
+mixture of 8 squared-relu experts and a gated shared one; a Bonerax model: gated linear attention, a delta rule with a decay
+per key channel, and windowed attention beside such a delta rule, gated feed-forwards alternating with a mixture of 16
+gated experts, 4 per token).
 
 Every timed step reads well over 126 MB (weights alone are 2.5 GB), so no input stays in L2
 between iterations.  tamnd/fastmlx publishes no number to compare with, and cannot run here
@@ -461,6 +463,28 @@ def kafepel_like(shape: dict, layers: int) -> dict:
             "layers": [{"type": "parallel", "mixer": mixer, "mlp": moe if i % 2 else dense} for i in range(layers)]}
 
 
+def bonerax_like(shape: dict, layers: int, window: int = 1024) -> dict:
+    """A Bonerax configuration with a Llama shape's width, heads and vocabulary: layers in the pattern gated linear
+    attention, channel delta rule, a pair of the shape's attention (sliding window, q and k normed, half of each head
+    rotated with YaRN's frequencies) and a channel delta rule of half the heads, and the channel delta rule of the second
+    layer once more (its weights, a state of its own); feed-forwards are the Llama layer's gated one, and in the delta
+    layers 16 experts of a quarter of its hidden size, 4 per token (the parameters a token uses are the same)."""
+    d, nh, nkv, hd = shape["hidden_size"], shape["num_attention_heads"], shape["num_key_value_heads"], shape["head_dim"]
+    ff = shape["intermediate_size"]
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 4}, "expert": {"ff": ff // 4}}
+    gla = {"type": "gla", "mlp": dense, "mixer": {"heads": nh, "dim": hd, "vdim": hd, "tau": 16.0}}
+    dl = {"type": "channel_delta", "mlp": moe, "mixer": {"heads": nh, "kv_heads": nkv, "dim": hd, "vdim": hd, "conv": 4}}
+    left = {"heads": nh, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": window},
+            "rot": {"dims": hd // 2, "base": 500000.0, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    pair = {"type": "parallel", "mlp": dense, "mixer": {"left": left, "right": dict(dl["mixer"], heads=nh // 2), "left_scale": 0.75,
+                                                        "right_scale": 0.5}}
+    out = [gla if i % 4 == 0 else dl if i % 2 else pair for i in range(layers)]
+    out = [dict(x, weights_of=i - 2) if i % 4 == 3 else x for i, x in enumerate(out)]
+    return {"architecture": "Bonerax", "vocab": shape["vocab_size"], "width": d, "logit_scale": 1.0, "logit_softcap": 30.0,
+            "norm": {"eps": 1e-6}, "layers": out}
+
+
 def step_weight_bytes(model, tokens: int) -> int:
     """Bytes of weights a step of `tokens` tokens must read: every run of the schedule reads its layer (a looped layer
     once per pass); a routed feed-forward with grouped products reads the experts its tokens chose, at most."""
@@ -527,7 +551,7 @@ def compare_designs(shapes, layers: int, context: int, steps: int, warmup: int, 
         name, shape = SHAPES[key]
         make = {"llama": lambda: dict(shape, num_hidden_layers=layers), "medirax": lambda: medirax_like(shape, layers),
                 "gekavik": lambda: gekavik_like(shape, layers), "sorupel": lambda: sorupel_like(shape, layers),
-                "kafepel": lambda: kafepel_like(shape, layers)}
+                "kafepel": lambda: kafepel_like(shape, layers), "bonerax": lambda: bonerax_like(shape, layers)}
         out[key] = {"layers": layers, "context": context}
         for design in which:
             out[key][design] = design_numbers(make[design](), shape["vocab_size"], pk, context, steps, warmup)
@@ -553,7 +577,7 @@ def main() -> int:
                     "layers of equal size are measured side by side; prints that comparison alone")
     ap.add_argument("--design-layers", type=int, default=8, help="layers of each model of the --designs comparison")
     ap.add_argument("--design-set", default="llama,medirax", help="which designs the --designs comparison measures "
-                    "(comma-separated, of llama, medirax, gekavik, sorupel, kafepel)")
+                    "(comma-separated, of llama, medirax, gekavik, sorupel, kafepel, bonerax)")
     ap.add_argument("--only-steps", type=int, default=0,
                     help="for a profiler's launch list: fill the batch, run this many decode steps and stop (no timing, no JSON line); "
                     "with --designs: a 2,048-token prompt step and the decode steps of the first design named, at the first size named")
@@ -579,14 +603,14 @@ def main() -> int:
     if args.designs:
         keys = [k for k in args.designs.split(",") if k]
         which = [w for w in args.design_set.split(",") if w]
-        if any(w not in ("llama", "medirax", "gekavik", "sorupel", "kafepel") for w in which):
-            print(f"bench.py: --design-set takes llama, medirax, gekavik, sorupel, kafepel (got {args.design_set!r})")
+        if any(w not in ("llama", "medirax", "gekavik", "sorupel", "kafepel", "bonerax") for w in which):
+            print(f"bench.py: --design-set takes llama, medirax, gekavik, sorupel, kafepel, bonerax (got {args.design_set!r})")
             return 2
         if args.only_steps > 0:
             shape = SHAPES[keys[0]][1]
             make = {"llama": lambda: dict(shape, num_hidden_layers=args.design_layers), "medirax": lambda: medirax_like(shape, args.design_layers),
                     "gekavik": lambda: gekavik_like(shape, args.design_layers), "sorupel": lambda: sorupel_like(shape, args.design_layers),
-                    "kafepel": lambda: kafepel_like(shape, args.design_layers)}
+                    "kafepel": lambda: kafepel_like(shape, args.design_layers), "bonerax": lambda: bonerax_like(shape, args.design_layers)}
             design_steps(make[which[0]](), shape["vocab_size"], args.batch, min(args.context, 4096), args.only_steps, warmup,
                          not args.no_cuda_graphs)
             print(f"ran a {PREFILL_TOKENS}-token prompt step and {args.only_steps} decode steps of batch {args.batch} of {which[0]} at the {keys[0]} sizes")

@@ -7,6 +7,7 @@ launches), for tuning and for profiler captures on a small case.
     python -m fastmlx_b200.kernels.microbench --kernel gemm --M 2048 --N 16384 --K 2048
     python -m fastmlx_b200.kernels.microbench --kernel sample --batch 8 --N 128256
     python -m fastmlx_b200.kernels.microbench --kernel recurrence --batch 1 --qlen 2048 --nh 64 --hd 64 --state 128
+    python -m fastmlx_b200.kernels.microbench --kernel channel --batch 1 --qlen 2048 --nh 32 --hd 64 --state 64
     python -m fastmlx_b200.kernels.microbench --kernel attn_masked --batch 64 --qlen 1 --ctx 4096 --hd 64
     python -m fastmlx_b200.kernels.microbench --kernel attn_mixed --batch 64 --qlen 1 --ctx 4096 --hd 64
 """
@@ -140,6 +141,46 @@ def _recurrence(a) -> int:
     return 0
 
 
+def _channel(a) -> int:
+    """Linear attention with a decay per key channel: --nh heads of --hd values over --state rows of state, --groups key heads
+    (gated linear attention: as many as heads); --batch requests of --qlen tokens each.  The kernels of both mixers, the
+    recurrence with every number of columns per group of lanes, and the layer norm step over rows of --K.  Per kernel:
+    microseconds (events, L2 flushed) and the bytes it must move over that time."""
+    H, P, N, G, taps, B, q = a.nh, a.hd, a.state, a.groups, a.taps, a.batch, a.qlen
+    T, inner = B * q, a.nh * a.hd
+    ctx = _rows_ctx(B, q)
+    flush = _flush()
+    gen = lambda *s: torch.randn(*s, device=DEV)
+    C, Cg = 2 * G * N + inner, 2 * H * N + inner
+    proj, z = gen(T, C + H).bfloat16(), gen(T, H * N + inner)
+    conv, a_log, dtb = gen(C, taps) * 0.5, torch.log(torch.rand(H, device=DEV) * 0.9 + 0.05), gen(H * N) * 0.5 - 1
+    state = gen(B, -(-(inner * N + (taps - 1) * C) // 4) * 4) * 0.1
+    norm_w = torch.rand(P, device=DEV) + 0.5
+    delta = lambda: k.channel_delta_prepare(proj, proj[:, C:], z[:, :H * N], conv, a_log, dtb, ctx, state, inner * N, H, G, N, P, taps)
+    qkv, g, beta = delta()
+    projg = gen(T, Cg + inner).bfloat16()
+    gla = lambda: k.channel_gla_prepare(projg, z[:, :H * N], dtb, H, N, P, N ** -0.5, 16.0)
+    qkv2, g2 = gla()
+    o = k.channel_scan(qkv, g, beta, ctx, state, H, G, N, P)
+    y, res, w = gen(T, a.K).bfloat16(), gen(T, a.K), torch.rand(a.K, device=DEV)
+    moved = lambda c: 2 * B * inner * N * 4 + T * (c + H * N + H + inner) * 4
+    rows = [("channel_delta_prepare", delta, T * (C + H) * 2 + T * H * N * 4 + T * (C + H * N + H) * 4 + B * (taps - 1) * C * 8),
+            ("channel_gla_prepare", gla, T * Cg * 2 + T * H * N * 4 + T * (Cg + H * N) * 4)]
+    for cpt in (0, 1, 2, 4):
+        rows += [(f"delta_scan cpt={cpt}", lambda cpt=cpt: k.channel_scan(qkv, g, beta, ctx, state, H, G, N, P, cpt=cpt), moved(C)),
+                 (f"gla_scan cpt={cpt}", lambda cpt=cpt: k.channel_scan(qkv2, g2, None, ctx, state, H, H, N, P, cpt=cpt), moved(Cg))]
+    rows += [("head_norm_gate", lambda: k.head_norm_gate(o, z[:, H * N:], norm_w, 1e-6, H, P, torch.bfloat16), T * inner * (4 + 4 + 2)),
+             (f"layernorm_step width={a.K}", lambda: k.layernorm_step(y, (w, 1e-6), 1.0, res, None, torch.bfloat16), T * a.K * (2 + 4 + 4 + 2))]
+    for name, fn, nbytes in rows:
+        if not name.startswith(a.only):
+            continue
+        us = _time_events(fn, a.replays, flush)
+        print(f"{name} B={B} qlen={q} heads={H} vdim={P} state={N} groups={G} taps={taps}: {us:.1f} us, {nbytes / 1e6:.1f} MB, "
+              f"{nbytes / us / 1e3:.0f} GB/s")
+    print("status", ctx.status.tolist())
+    return 0
+
+
 def _attn_masked(a) -> int:
     """The tiled two-term attention kernel over bfloat16 pages with a sliding window (keys and values apart) and with
     runs of positions, one more term in the denominator and values that are read from a second plane, at equal sizes;
@@ -223,7 +264,7 @@ def _attn_mixed(a) -> int:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
-    ap.add_argument("--kernel", required=True, choices=["attn_decode", "attn_prefill", "gemv", "gemm", "sample", "recurrence", "attn_masked", "attn_mixed"])
+    ap.add_argument("--kernel", required=True, choices=["attn_decode", "attn_prefill", "gemv", "gemm", "sample", "recurrence", "channel", "attn_masked", "attn_mixed"])
     ap.add_argument("--simple", action="store_true", help="attn_mixed: time the kernel of one warp per token, head and value head too")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--ctx", type=int, default=8192, help="tokens already in the cache")
@@ -248,6 +289,8 @@ def main(argv=None) -> int:
     a = ap.parse_args(argv)
     if a.kernel == "recurrence":
         return _recurrence(a)
+    if a.kernel == "channel":
+        return _channel(a)
     if a.kernel == "attn_masked":
         return _attn_masked(a)
     if a.kernel == "attn_mixed":

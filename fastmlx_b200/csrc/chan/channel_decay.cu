@@ -498,20 +498,32 @@ FMX_EXPORT int fmx_channel_gla_prepare(const void* proj, long long stride, const
   return 0;
 }
 
-// beta null: gated linear attention; else the delta rule.  single: every row brings one token.  cpt: columns per group of
-// lanes (1, 2 or 4; 0: the choice is made here).
+// beta null: gated linear attention; else the delta rule.  single: every row brings one token.  lanes (8, 16, 32): lanes that
+// share a column, cpt (1, 2, 4): columns that they hold; 0: the choice is made here.
 FMX_EXPORT int fmx_channel_scan(const float* qkv, const float* decay, const float* beta, const int* row_start,
                                 const int* row_slot, float* state, long long slot_stride, float* out, int R, int H, int G, int D,
-                                int Dv, int max_slots, int single, int cpt, cudaStream_t stream) {
+                                int Dv, int max_slots, int single, int lanes, int cpt, cudaStream_t stream) {
   if (R == 0) return 0;
   if (R < 0 || H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || D > 512)
     return fmx_fail("fmx_channel_scan: bad sizes R=%d H=%d G=%d D=%d Dv=%d", R, H, G, D, Dv);
   if (H > 65535 || R > 65535) return fmx_fail("fmx_channel_scan: batch too large");
-  const int lanes = D <= 64 ? 8 : D <= 128 ? 16 : 32;
-  const int most = D > 256 ? 1 : lanes / 4 > 4 ? 4 : lanes / 4;               // four tokens' sums of a lane's columns fit its lanes
+  // Measured (us for 2,048 tokens of one request, 32 heads; delta rule / gated linear attention): 64 x 64 state: 8 lanes with one
+  // column 418 / 291, with two 461 / 318, 16 lanes with two 389 / 265; 128 x 128: 16 lanes with one column 820 / 610, two
+  // 630 / 453, four 747 / 358.  64 single tokens: 64 x 64: 8 lanes with two columns 23 / 23, 16 with two 31 / 29; 128 x 128: 16
+  // lanes with one column 88 / 66, with four 68 / 59.
+  const long long heads = (long long)R * H;
+  const bool few = !single && heads * ((Dv + 15) / 16) < fmx_num_sms() * 3 / 2;           // one warp per scheduler at most
+  if (lanes == 0) lanes = D <= 64 ? (few && D > 32 ? 16 : 8) : D <= 128 ? 16 : 32;
+  if (lanes == 8 && D > 64) lanes = 16;
+  if (lanes == 16 && D > 128) lanes = 32;
+  if (lanes == 32 && D <= 128) lanes = 16;
+  if (lanes != 8 && lanes != 16 && lanes != 32) return fmx_fail("fmx_channel_scan: 8, 16 or 32 lanes per column, not %d", lanes);
+  const int most = D > 256 ? 1 : lanes == 8 ? 2 : 4;                          // four tokens' sums of a lane's columns fit its lanes
   if (cpt == 0) {                                 // as many columns per group of lanes as leave every multiprocessor a block
     cpt = most;
-    while (cpt > 1 && (long long)R * H * ((Dv + 128 / lanes * cpt - 1) / (128 / lanes * cpt)) < fmx_num_sms() * 3 / 4) cpt /= 2;
+    while (cpt > 1 && heads * ((Dv + 128 / lanes * cpt - 1) / (128 / lanes * cpt)) < fmx_num_sms() * 3 / 4) cpt /= 2;
+    if (beta != nullptr && !single && cpt == 4 && heads * ((Dv + 512 / lanes - 1) / (512 / lanes)) < fmx_num_sms()) cpt = 2;
+    if (few && D <= 64 && lanes == 16) cpt = 2;
   }
   if (cpt != 1 && cpt != 2 && cpt != 4) return fmx_fail("fmx_channel_scan: 1, 2 or 4 columns per group of lanes, not %d", cpt);
   if (cpt > most) cpt = most;
@@ -531,11 +543,21 @@ FMX_EXPORT int fmx_channel_scan(const float* qkv, const float* decay, const floa
     else if (single) FMX_CS(false, RPL, L, CPT, 1, 4);                                                                 \
     else FMX_CS(false, RPL, L, CPT, 4, TB);                                                                            \
   } while (0)
-  if (D <= 32) { if (cpt == 1) FMX_CS_G(4, 8, 1, 16); else FMX_CS_G(4, 8, 2, 16); }
-  else if (D <= 64) { if (cpt == 1) FMX_CS_G(8, 8, 1, 16); else FMX_CS_G(8, 8, 2, 16); }
-  else if (D <= 128) { if (cpt == 1) FMX_CS_G(8, 16, 1, 16); else if (cpt == 2) FMX_CS_G(8, 16, 2, 16); else FMX_CS_G(8, 16, 4, 16); }
-  else if (D <= 256) { if (cpt == 1) FMX_CS_G(8, 32, 1, 16); else if (cpt == 2) FMX_CS_G(8, 32, 2, 16); else FMX_CS_G(8, 32, 4, 16); }
+#define FMX_CS_C(RPL, L, TB)                                                                                          \
+  do {                                                                                                                 \
+    if (cpt == 1) FMX_CS_G(RPL, L, 1, TB);                                                                             \
+    else if (cpt == 2) FMX_CS_G(RPL, L, 2, TB);                                                                        \
+    else FMX_CS_G(RPL, L, 4, TB);                                                                                      \
+  } while (0)
+  if (lanes == 8) {
+    if (D <= 32) { if (cpt == 1) FMX_CS_G(4, 8, 1, 16); else FMX_CS_G(4, 8, 2, 16); }
+    else { if (cpt == 1) FMX_CS_G(8, 8, 1, 16); else FMX_CS_G(8, 8, 2, 16); }
+  } else if (lanes == 16) {
+    if (D <= 64) FMX_CS_C(4, 16, 16);
+    else FMX_CS_C(8, 16, 16);
+  } else if (D <= 256) FMX_CS_C(8, 32, 16);
   else FMX_CS_G(16, 32, 1, 8);
+#undef FMX_CS_C
 #undef FMX_CS_G
 #undef FMX_CS
   FMX_LAUNCH_CHECK();

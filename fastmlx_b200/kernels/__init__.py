@@ -814,17 +814,17 @@ def channel_gla_prepare(proj, z, bias, H, D, Dv, q_scale: float, tau: float):
     return qkv, g
 
 
-def channel_scan(qkv, g, beta, ctx, state, H, G, D, Dv, cpt: int = 0) -> torch.Tensor:
+def channel_scan(qkv, g, beta, ctx, state, H, G, D, Dv, lanes: int = 0, cpt: int = 0) -> torch.Tensor:
     """Linear attention with a decay per key channel over every request's tokens of the step, in order, from and into the
     requests' state slots (S^T per head, [H, Dv, D], at the head of a slot): S <- diag(g) S, then the delta rule's write
     u = beta (v - S^T k), S <- S + k u^T, or with beta None S <- S + k v^T; o = S^T q.  qkv[T, q (G*D) | k (G*D) |
-    v (H*Dv)], g[T, H*D], beta[T, H], all 32-bit.  `cpt` (1, 2, 4; 0: the library's choice): columns of S that a group of
-    lanes holds.  -> o in 32-bit, [T, H*Dv]."""
+    v (H*Dv)], g[T, H*D], beta[T, H], all 32-bit.  `lanes` (8, 16, 32) and `cpt` (1, 2, 4; 0: the library's choice): lanes
+    that share a column of S, and columns that they hold.  -> o in 32-bit, [T, H*Dv]."""
     T = qkv.shape[0]
     assert qkv.is_contiguous() and g.is_contiguous() and (beta is None or beta.is_contiguous())
     out = torch.empty((T, H * Dv), dtype=torch.float32, device=qkv.device)
     call("chan", "fmx_channel_scan", qkv.data_ptr(), g.data_ptr(), _ptr(beta), ctx.row_start.data_ptr(), ctx.row_slot.data_ptr(),
-         state.data_ptr(), state.stride(0), out.data_ptr(), ctx.R, H, G, D, Dv, state.shape[0], int(ctx.max_q_len == 1), int(cpt),
+         state.data_ptr(), state.stride(0), out.data_ptr(), ctx.R, H, G, D, Dv, state.shape[0], int(ctx.max_q_len == 1), int(lanes), int(cpt),
          _stream())
     return out
 

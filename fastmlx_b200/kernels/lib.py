@@ -89,7 +89,7 @@ _SIGNATURES = {
         "fmx_channel_delta_prepare": [_P, _L, _P, _L, _P, _L, _P, _P, _P, _P, _P, _P, _P, _L, _L, _P, _P, _P, _I, _I, _I, _I, _I,
                                       _I, _I, _I, _I, _I, _P, _P],
         "fmx_channel_gla_prepare": [_P, _L, _P, _L, _P, _P, _P, _I, _I, _I, _I, _F, _F, _I, _P],
-        "fmx_channel_scan": [_P, _P, _P, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+        "fmx_channel_scan": [_P, _P, _P, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
         "fmx_head_norm_gate": [_P, _P, _L, _I, _P, _P, _L, _I, _I, _I, _I, _F, _I, _P],
     },
     "mixattn": {

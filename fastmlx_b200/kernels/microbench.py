@@ -166,9 +166,9 @@ def _channel(a) -> int:
     moved = lambda c: 2 * B * inner * N * 4 + T * (c + H * N + H + inner) * 4
     rows = [("channel_delta_prepare", delta, T * (C + H) * 2 + T * H * N * 4 + T * (C + H * N + H) * 4 + B * (taps - 1) * C * 8),
             ("channel_gla_prepare", gla, T * Cg * 2 + T * H * N * 4 + T * (Cg + H * N) * 4)]
-    for cpt in (0, 1, 2, 4):
-        rows += [(f"delta_scan cpt={cpt}", lambda cpt=cpt: k.channel_scan(qkv, g, beta, ctx, state, H, G, N, P, cpt=cpt), moved(C)),
-                 (f"gla_scan cpt={cpt}", lambda cpt=cpt: k.channel_scan(qkv2, g2, None, ctx, state, H, H, N, P, cpt=cpt), moved(Cg))]
+    for ln, cpt in ((0, 0),) + tuple((n, c) for n in (8, 16, 32) for c in (1, 2, 4) if 4 * c <= n and 4 * n < N + 32 <= 8 * n + 32):
+        rows += [(f"delta_scan lanes={ln} cpt={cpt}", lambda ln=ln, cpt=cpt: k.channel_scan(qkv, g, beta, ctx, state, H, G, N, P, ln, cpt), moved(C)),
+                 (f"gla_scan lanes={ln} cpt={cpt}", lambda ln=ln, cpt=cpt: k.channel_scan(qkv2, g2, None, ctx, state, H, H, N, P, ln, cpt), moved(Cg))]
     rows += [("head_norm_gate", lambda: k.head_norm_gate(o, z[:, H * N:], norm_w, 1e-6, H, P, torch.bfloat16), T * inner * (4 + 4 + 2)),
              (f"layernorm_step width={a.K}", lambda: k.layernorm_step(y, (w, 1e-6), 1.0, res, None, torch.bfloat16), T * a.K * (2 + 4 + 4 + 2))]
     for name, fn, nbytes in rows:

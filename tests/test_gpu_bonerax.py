@@ -36,7 +36,9 @@ CASES = {
 }
 # A router that takes bfloat16 inputs sees its logits moved a little; where the plain model's own choice of experts is
 # decided by less (in some layer), either choice is right, and the recurrences carry the other choice on: such a position
-# and the SPAN - 1 after it are not compared in bfloat16.
+# and the SPAN - 1 after it are not compared in bfloat16.  Nor is a sequence's first token: there a recurrence's read-out is
+# one value times q . k, and the norm behind it leaves of that number its sign alone, whose rounding nothing bounds (in
+# 32-bit that position is compared like all others).
 CLOSE_CALL, SPAN = 0.05, 10
 
 
@@ -45,6 +47,7 @@ def _unsure(cfg, W, toks):
     margins = []
     ref = pb.forward(cfg, W, toks, margins=margins)
     skip = torch.zeros(len(toks), dtype=torch.bool)
+    skip[0] = True
     if margins:
         for u in torch.nonzero(torch.stack(margins).min(0).values < CLOSE_CALL).flatten().tolist():
             skip[u:u + SPAN] = True

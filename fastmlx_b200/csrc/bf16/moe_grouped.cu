@@ -18,12 +18,16 @@
 #include "common.cuh"
 
 namespace {
-constexpr int BM = 128, BK = 32, ROWP = BK + 8, THREADS = 256, STAGES = 3;
-template <bool GATED> struct Tile {
+constexpr int BM = 128, BK = 32, ROWP = BK + 8, THREADS = 256;
+// ROWS: the rows of a tile that may hold pairs.  A token takes an expert once, so a step of T tokens puts at most T pairs
+// into an expert's first tile: steps of few tokens keep fewer rows of A and a deeper ring of the weights' tiles, whose
+// bytes in flight are what they are bound by.
+template <bool GATED, int ROWS> struct Tile {
+  static constexpr int STAGES = ROWS <= 16 ? 8 : ROWS <= 64 ? 6 : 3;
   static constexpr int BN = GATED ? 64 : 128;            // hidden columns (of gate and of up), or output columns
   static constexpr int WM = GATED ? 4 : 2, WN = GATED ? 2 : 4;      // warps along rows and columns
   static constexpr int MT = BM / WM / 16;                // 16-row tiles of a warp: 2 or 4; a warp spans 32 columns
-  static constexpr int STAGE = (BM + (GATED ? 2 : 1) * BN) * ROWP;  // elements of one stage: A, W0 (, W1)
+  static constexpr int STAGE = (ROWS + (GATED ? 2 : 1) * BN) * ROWP;  // elements of one stage: A, W0 (, W1)
   static constexpr size_t SMEM = (size_t)STAGES * STAGE * sizeof(bf16);
 };
 
@@ -117,13 +121,13 @@ __device__ __forceinline__ void warp_step(float (&acc)[MT][4][4], const bf16* as
 
 // GATED: W0 = the expert's gate rows, W1 = its up rows, out = activation (bf16); else W0 alone, out = product (32-bit).
 // Rows of padding are neither read nor written.
-template <bool GATED>
+template <bool GATED, int ROWS>
 __global__ void __launch_bounds__(THREADS)
 moe_grouped_kernel(const bf16* a, long long lda, const int* sorted_token, const float* sorted_w, const int* tile_expert,
                    const bf16* w0, const bf16* w1, long long ldw, long long expert_stride, void* out, long long ldo, int N,
                    int K, float limit, int block) {
-  using TL = Tile<GATED>;
-  constexpr int BN = TL::BN, MT = TL::MT;
+  using TL = Tile<GATED, ROWS>;
+  constexpr int BN = TL::BN, MT = TL::MT, STAGES = TL::STAGES;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* smem = reinterpret_cast<bf16*>(smem_raw);
   __shared__ int toks[BM];
@@ -138,16 +142,17 @@ moe_grouped_kernel(const bf16* a, long long lda, const int* sorted_token, const 
   if (tid < BM) toks[tid] = tok_mine;
   // the pairs of a tile stand at its start: a decode step's tiles hold a few, and a warp multiplies only the 16-row
   // tiles that hold any (the expert's weights stream either way)
-  const int n_real = __syncthreads_count(tok_mine >= 0);
+  const int n_real = min(ROWS, __syncthreads_count(tok_mine >= 0));
   const bf16* we0 = w0 + (long long)e * expert_stride;
   const bf16* we1 = GATED ? w1 + (long long)e * expert_stride : nullptr;
   auto stage_a = [&](int s) { return smem + (size_t)s * TL::STAGE; };
-  auto stage_w0 = [&](int s) { return smem + (size_t)s * TL::STAGE + BM * ROWP; };
-  auto stage_w1 = [&](int s) { return smem + (size_t)s * TL::STAGE + (BM + BN) * ROWP; };
+  auto stage_w0 = [&](int s) { return smem + (size_t)s * TL::STAGE + ROWS * ROWP; };
+  auto stage_w1 = [&](int s) { return smem + (size_t)s * TL::STAGE + (ROWS + BN) * ROWP; };
   auto load = [&](int stage, int k0) {
 #pragma unroll
-    for (int it = 0; it < (BM * (BK / 8)) / THREADS; ++it) {
+    for (int it = 0; it < (ROWS * (BK / 8) + THREADS - 1) / THREADS; ++it) {
       const int item = tid + it * THREADS;
+      if ((ROWS * (BK / 8)) % THREADS != 0 && item >= ROWS * (BK / 8)) break;
       const int r = item / (BK / 8), ch = item - r * (BK / 8);
       const int k = k0 + ch * 8;
       const int tok = toks[r];                       // rows of A: gathered by token (GATED), or the sorted rows themselves
@@ -324,24 +329,33 @@ FMX_EXPORT int fmx_moe_sort(const int* chosen, const float* weights, int T, int 
 
 // x [T, K] bf16 (rows of ldx); w_gate / w_up: expert e's rows start e * expert_stride elements in, rows of ldw;
 // y [max_tiles * 64, ff] bf16.
-// block > 0: gate and up rows alternate in blocks of `block` (w_up = w_gate + block rows).
+// block > 0: gate and up rows alternate in blocks of `block` (w_up = w_gate + block rows).  tokens: the step's tokens (an
+// expert then has at most that many pairs; 0: unknown).
 FMX_EXPORT int fmx_moe_grouped_gate_up(const void* x, long long ldx, const int* sorted_token, const float* sorted_w,
                                        const int* tile_expert, const void* w_gate, const void* w_up, long long ldw,
                                        long long expert_stride, void* y, int max_tiles, int ff, int K, float limit,
-                                       int block, cudaStream_t stream) {
+                                       int block, int tokens, cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
   if (ff <= 0 || K <= 0 || K % 8 || ldx % 8 || ldw % 8 || expert_stride % 8 || ((uintptr_t)x & 15) || ((uintptr_t)w_gate & 15) ||
       ((uintptr_t)w_up & 15))
     return fmx_fail("fmx_moe_grouped_gate_up: rows of 16 bytes wanted (K=%d)", K);
   if (max_tiles > 65535) return fmx_fail("fmx_moe_grouped_gate_up: too many tiles for one launch");
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(moe_grouped_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Tile<true>::SMEM);
-    if (e != cudaSuccess) return fmx_fail("fmx_moe_grouped_gate_up: shared memory of %zu bytes refused: %s", Tile<true>::SMEM, cudaGetErrorString(e));
-    configured = true;
-  }
-  fmx_launch(moe_grouped_kernel<true>, dim3((ff + Tile<true>::BN - 1) / Tile<true>::BN, max_tiles), dim3(THREADS), Tile<true>::SMEM, stream, (const bf16*)x, ldx, sorted_token,
-             sorted_w, tile_expert, (const bf16*)w_gate, (const bf16*)w_up, ldw, expert_stride, y, (long long)ff, ff, K, limit, block);
+  cudaError_t e = cudaSuccess;
+#define FMX_MGU(ROWS)                                                                                                  \
+  do {                                                                                                                 \
+    using TL = Tile<true, ROWS>;                                                                                       \
+    static const cudaError_t set = cudaFuncSetAttribute(moe_grouped_kernel<true, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TL::SMEM); \
+    e = set;                                                                                                           \
+    if (e == cudaSuccess)                                                                                              \
+      fmx_launch(moe_grouped_kernel<true, ROWS>, dim3((ff + TL::BN - 1) / TL::BN, max_tiles), dim3(THREADS), TL::SMEM, stream, (const bf16*)x, \
+                 ldx, sorted_token, sorted_w, tile_expert, (const bf16*)w_gate, (const bf16*)w_up, ldw, expert_stride, y, (long long)ff, ff, K, \
+                 limit, block);                                                                                        \
+  } while (0)
+  if (tokens > 0 && tokens <= 16) FMX_MGU(16);
+  else if (tokens > 0 && tokens <= 64) FMX_MGU(64);
+  else FMX_MGU(128);
+#undef FMX_MGU
+  if (e != cudaSuccess) return fmx_fail("fmx_moe_grouped_gate_up: shared memory refused: %s", cudaGetErrorString(e));
   FMX_LAUNCH_CHECK();
   return 0;
 }
@@ -350,20 +364,27 @@ FMX_EXPORT int fmx_moe_grouped_gate_up(const void* x, long long ldx, const int* 
 // pair_out [max_tiles * 64, d] float.
 FMX_EXPORT int fmx_moe_grouped_down(const void* y, const int* sorted_token, const int* tile_expert, const void* w_down,
                                     long long ldw, long long expert_stride, float* pair_out, int max_tiles, int d, int ff,
-                                    cudaStream_t stream) {
+                                    int tokens, cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
   if (ff <= 0 || d <= 0 || ff % 8 || ldw % 8 || expert_stride % 8 || ((uintptr_t)y & 15) || ((uintptr_t)w_down & 15))
     return fmx_fail("fmx_moe_grouped_down: rows of 16 bytes wanted (ff=%d)", ff);
   if (max_tiles > 65535) return fmx_fail("fmx_moe_grouped_down: too many tiles for one launch");
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(moe_grouped_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Tile<false>::SMEM);
-    if (e != cudaSuccess) return fmx_fail("fmx_moe_grouped_down: shared memory of %zu bytes refused: %s", Tile<false>::SMEM, cudaGetErrorString(e));
-    configured = true;
-  }
-  fmx_launch(moe_grouped_kernel<false>, dim3((d + Tile<false>::BN - 1) / Tile<false>::BN, max_tiles), dim3(THREADS), Tile<false>::SMEM, stream, (const bf16*)y, (long long)ff,
-             sorted_token, (const float*)nullptr, tile_expert, (const bf16*)w_down, (const bf16*)nullptr, ldw, expert_stride,
-             (void*)pair_out, (long long)d, d, ff, 0.f, 0);
+  cudaError_t e = cudaSuccess;
+#define FMX_MGD(ROWS)                                                                                                  \
+  do {                                                                                                                 \
+    using TL = Tile<false, ROWS>;                                                                                      \
+    static const cudaError_t set = cudaFuncSetAttribute(moe_grouped_kernel<false, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TL::SMEM); \
+    e = set;                                                                                                           \
+    if (e == cudaSuccess)                                                                                              \
+      fmx_launch(moe_grouped_kernel<false, ROWS>, dim3((d + TL::BN - 1) / TL::BN, max_tiles), dim3(THREADS), TL::SMEM, stream, (const bf16*)y, \
+                 (long long)ff, sorted_token, (const float*)nullptr, tile_expert, (const bf16*)w_down, (const bf16*)nullptr, ldw, \
+                 expert_stride, (void*)pair_out, (long long)d, d, ff, 0.f, 0);                                     \
+  } while (0)
+  if (tokens > 0 && tokens <= 16) FMX_MGD(16);
+  else if (tokens > 0 && tokens <= 64) FMX_MGD(64);
+  else FMX_MGD(128);
+#undef FMX_MGD
+  if (e != cudaSuccess) return fmx_fail("fmx_moe_grouped_down: shared memory refused: %s", cudaGetErrorString(e));
   FMX_LAUNCH_CHECK();
   return 0;
 }

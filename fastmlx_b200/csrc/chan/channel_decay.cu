@@ -25,8 +25,15 @@ __device__ __forceinline__ float softplus_f(float a) { return fmaxf(a, 0.f) + lo
 
 // proj [T, stride]: q (G*D) | k (G*D) | v (H*Dv) | ...; b [T, b_stride] the write strengths' pre-activations; z [T, z_stride]
 // 32-bit: the decays' pre-activations (H*D).  out_qkv [T, C], out_g [T, H*D], out_beta [T, H], 32-bit.
-// MAXI: values of a q or k head that a lane holds (D <= 32 MAXI).
-template <typename T, int MAXI>
+// MAXI: values of a q or k head that a lane holds (D <= 32 MAXI).  W: neighbouring channels that a lane takes at a time (2
+// where D, Dv and the rows' starts allow it).
+template <typename T> __device__ __forceinline__ float2 load2(const T* p);
+template <> __device__ __forceinline__ float2 load2<float>(const float* p) { return *reinterpret_cast<const float2*>(p); }
+template <> __device__ __forceinline__ float2 load2<bf16>(const bf16* p) {
+  return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+}
+
+template <typename T, int MAXI, int W>
 __global__ void __launch_bounds__(128)
 channel_delta_prepare_kernel(const T* proj, long long stride, const T* b, long long b_stride, const float* z, long long z_stride,
                              const float* __restrict__ conv_w, const float* __restrict__ a_log, const float* __restrict__ dt_bias,
@@ -42,9 +49,15 @@ channel_delta_prepare_kernel(const T* proj, long long stride, const T* b, long l
   if (item >= 2 * G + H) {                        // a head's decays and its write strength
     const int h = item - 2 * G - H;
     const float rate = expf(a_log[h]);
-    for (int e = lane; e < D; e += 32) {
+    for (int e = W * lane; e < D; e += 32 * W) {
       const long long c = (long long)h * D + e;
-      out_g[(long long)t * H * D + c] = expf(-rate * softplus_f(z[(long long)t * z_stride + c] + dt_bias[c]));
+      if (W == 2) {
+        const float2 x = load2(z + (long long)t * z_stride + c), b2 = load2(dt_bias + c);
+        *reinterpret_cast<float2*>(out_g + (long long)t * H * D + c) =
+            make_float2(expf(-rate * softplus_f(x.x + b2.x)), expf(-rate * softplus_f(x.y + b2.y)));
+      } else {
+        out_g[(long long)t * H * D + c] = expf(-rate * softplus_f(z[(long long)t * z_stride + c] + dt_bias[c]));
+      }
     }
     if (lane == 0) out_beta[(long long)t * H + h] = 1.0f / (1.0f + expf(-to_f(b[(long long)t * b_stride + h])));
     return;
@@ -74,8 +87,41 @@ channel_delta_prepare_kernel(const T* proj, long long stride, const T* b, long l
     }
     return silu_f(acc);
   };
+  auto channels = [&](int e) -> float2 {          // channels e and e + 1
+    const int c = c0 + e;
+    float2 acc = make_float2(0.f, 0.f);
+    for (int j = 0; j < taps; ++j) {
+      const int n = i - (taps - 1) + j;
+      const float2 x = n >= 0 ? load2(proj + (long long)(first + n) * stride + c) : load2(cs + (long long)(taps - 1 + n) * C + c);
+      acc.x = fmaf(conv_w[(long long)c * taps + j], x.x, acc.x);
+      acc.y = fmaf(conv_w[(long long)(c + 1) * taps + j], x.y, acc.y);
+      if (single && j > 0) *reinterpret_cast<float2*>(cs + (long long)(j - 1) * C + c) = x;
+    }
+    return make_float2(silu_f(acc.x), silu_f(acc.y));
+  };
   if (item >= 2 * G) {
-    for (int e = lane; e < n_c; e += 32) dst[e] = channel(e);
+    for (int e = W * lane; e < n_c; e += 32 * W) {
+      if (W == 2) *reinterpret_cast<float2*>(dst + e) = channels(e);
+      else dst[e] = channel(e);
+    }
+    return;
+  }
+  if (W == 2) {
+    float2 v[MAXI / 2];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < MAXI / 2; ++k) {
+      const int e = 2 * lane + 64 * k;
+      v[k] = e < D ? channels(e) : make_float2(0.f, 0.f);
+      ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, ss));
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f);
+    const float mul = item < G ? inv * (1.0f / sqrtf((float)D)) : inv;         // q heads come first
+#pragma unroll
+    for (int k = 0; k < MAXI / 2; ++k) {
+      const int e = 2 * lane + 64 * k;
+      if (e < D) *reinterpret_cast<float2*>(dst + e) = make_float2(v[k].x * mul, v[k].y * mul);
+    }
     return;
   }
   float v[MAXI], ss = 0.f;
@@ -116,6 +162,48 @@ channel_gla_prepare_kernel(const T* proj, long long stride, const float* z, long
       const float x = z[t * z_stride + e] + (bias != nullptr ? bias[e] : 0.f);
       out_g[t * HD + e] = expf(-softplus_f(-x) * inv_tau);                     // sigmoid(x)^(1/tau)
     }
+  }
+}
+
+// four neighbouring values of any element type in one access
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const bf16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(bf16* p, float4 v) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<unsigned*>(&a);
+  u.y = *reinterpret_cast<unsigned*>(&b);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+
+// The same with four neighbouring columns per access (HD, C and every row start multiples of four).
+template <typename T>
+__global__ void __launch_bounds__(128)
+channel_gla_prepare_vec_kernel(const T* proj, long long stride, const float* z, long long z_stride, const float* __restrict__ bias,
+                               float* out_qkv, float* out_g, int HD, int C, float q_scale, float inv_tau) {
+  pdl_wait();
+  pdl_trigger();
+  const long long t = blockIdx.x;
+  const int c = (blockIdx.y * 128 + threadIdx.x) * 4;
+  if (c < C) {
+    float4 x = load4(proj + t * stride + c);
+    if (c < HD) x = make_float4(x.x * q_scale, x.y * q_scale, x.z * q_scale, x.w * q_scale);
+    store4(out_qkv + t * C + c, x);
+  } else if (c < C + HD) {
+    const int e = c - C;
+    float4 x = load4(z + t * z_stride + e);
+    if (bias != nullptr) {
+      const float4 b = load4(bias + e);
+      x = make_float4(x.x + b.x, x.y + b.y, x.z + b.z, x.w + b.w);
+    }
+    store4(out_g + t * HD + e, make_float4(expf(-softplus_f(-x.x) * inv_tau), expf(-softplus_f(-x.y) * inv_tau),
+                                           expf(-softplus_f(-x.z) * inv_tau), expf(-softplus_f(-x.w) * inv_tau)));
   }
 }
 
@@ -442,6 +530,30 @@ head_norm_gate_kernel(const float* o, const TG* gate, long long gate_stride, con
     dst[e] = from_f<T>(op[e] * rstd * w[e] * (silu ? x * sg : sg));
   }
 }
+
+// The same with four neighbouring values per lane: LG = Dv / 4 lanes (8, 16 or 32) per (token, head).
+template <typename TG, typename T, int LG>
+__global__ void __launch_bounds__(128)
+head_norm_gate_vec_kernel(const float* o, const TG* gate, long long gate_stride, const float* __restrict__ w, T* out,
+                          long long out_stride, long long n_items, int H, float eps, int silu) {
+  pdl_wait();
+  pdl_trigger();
+  const long long item = (long long)blockIdx.x * (128 / LG) + threadIdx.x / LG;
+  const int e = 4 * (threadIdx.x % LG), Dv = 4 * LG;
+  const bool live = item < n_items;                // (every lane takes part in the exchange)
+  const long long t = live ? item / H : 0;
+  const int h = live ? (int)(item - t * H) : 0;
+  const float4 x = live ? load4(o + item * Dv + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+  float ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w)));
+#pragma unroll
+  for (int d = LG / 2; d >= 1; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+  if (!live) return;
+  const float rstd = 1.0f / sqrtf(ss / (float)Dv + eps);
+  const float4 g = load4(gate + t * gate_stride + (long long)h * Dv + e), ww = load4(w + e);
+  auto act = [&](float v) { const float sg = 1.0f / (1.0f + expf(-v)); return silu ? v * sg : sg; };
+  store4(out + t * out_stride + (long long)h * Dv + e, make_float4(x.x * rstd * ww.x * act(g.x), x.y * rstd * ww.y * act(g.y),
+                                                                  x.z * rstd * ww.z * act(g.z), x.w * rstd * ww.w * act(g.w)));
+}
 }  // namespace
 
 // single: every row of the step brings one token; the convolution state then moves on inside the kernel.
@@ -456,8 +568,17 @@ FMX_EXPORT int fmx_channel_delta_prepare(const void* proj, long long stride, con
     return fmx_fail("fmx_channel_delta_prepare: bad sizes T=%d R=%d H=%d G=%d D=%d Dv=%d taps=%d", T, R, H, G, D, Dv, taps);
   const int C = 2 * G * D + H * Dv;
   if (stride < C || b_stride < H || z_stride < (long long)H * D) return fmx_fail("fmx_channel_delta_prepare: rows too narrow");
+  // two channels at a time: every head, row and slot starts on a pair
+  const bool two = D % 2 == 0 && Dv % 2 == 0 && stride % 2 == 0 && z_stride % 2 == 0 && slot_stride % 2 == 0 && conv_off % 2 == 0 &&
+                   ((uintptr_t)z & 7) == 0 && ((uintptr_t)dt_bias & 7) == 0 && ((uintptr_t)state & 7) == 0 &&
+                   ((uintptr_t)out_qkv & 7) == 0 && ((uintptr_t)out_g & 7) == 0 && ((uintptr_t)proj & (dtype == FMX_F32 ? 7 : 3)) == 0;
 #define FMX_CDP(TT, MAXI)                                                                                              \
-  fmx_launch(channel_delta_prepare_kernel<TT, MAXI>, dim3(T, (2 * G + 2 * H + 3) / 4), dim3(128), 0, stream, (const TT*)proj, stride, \
+  do {                                                                                                                 \
+    if (two) FMX_CDP_W(TT, MAXI, 2);                                                                                   \
+    else FMX_CDP_W(TT, MAXI, 1);                                                                                       \
+  } while (0)
+#define FMX_CDP_W(TT, MAXI, W)                                                                                         \
+  fmx_launch(channel_delta_prepare_kernel<TT, MAXI, W>, dim3(T, (2 * G + 2 * H + 3) / 4), dim3(128), 0, stream, (const TT*)proj, stride, \
              (const TT*)b, b_stride, z, z_stride, conv_w, a_log, dt_bias, token_row, row_start, row_slot, state, slot_stride, \
              conv_off, out_qkv, out_g, out_beta, H, G, D, Dv, taps, R, max_slots, single, status)
 #define FMX_CDP_T(TT)                                                                                                  \
@@ -473,6 +594,7 @@ FMX_EXPORT int fmx_channel_delta_prepare(const void* proj, long long stride, con
   else if (dtype == FMX_BF16) FMX_CDP_T(bf16);
   else return fmx_fail("fmx_channel_delta_prepare: unknown dtype %d", dtype);
 #undef FMX_CDP_T
+#undef FMX_CDP_W
 #undef FMX_CDP
   FMX_LAUNCH_CHECK();
   return 0;
@@ -486,6 +608,18 @@ FMX_EXPORT int fmx_channel_gla_prepare(const void* proj, long long stride, const
   if (T < 0 || H <= 0 || D <= 0 || Dv <= 0 || stride < C || z_stride < HD)
     return fmx_fail("fmx_channel_gla_prepare: bad sizes T=%d H=%d D=%d Dv=%d", T, H, D, Dv);
   const dim3 grid(T, (C + HD + 511) / 512);
+  auto a16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  if (HD % 4 == 0 && C % 4 == 0 && stride % 4 == 0 && z_stride % 4 == 0 && a16(z) && a16(bias) && a16(out_qkv) && a16(out_g) &&
+      ((uintptr_t)proj & (dtype == FMX_F32 ? 15 : 7)) == 0 && (dtype == FMX_F32 || dtype == FMX_BF16)) {
+    if (dtype == FMX_F32)
+      fmx_launch(channel_gla_prepare_vec_kernel<float>, grid, dim3(128), 0, stream, (const float*)proj, stride, z, z_stride, bias,
+                 out_qkv, out_g, HD, C, q_scale, inv_tau);
+    else
+      fmx_launch(channel_gla_prepare_vec_kernel<bf16>, grid, dim3(128), 0, stream, (const bf16*)proj, stride, z, z_stride, bias,
+                 out_qkv, out_g, HD, C, q_scale, inv_tau);
+    FMX_LAUNCH_CHECK();
+    return 0;
+  }
   if (dtype == FMX_F32)
     fmx_launch(channel_gla_prepare_kernel<float>, grid, dim3(128), 0, stream, (const float*)proj, stride, z, z_stride, bias, out_qkv,
                out_g, HD, C, q_scale, inv_tau);
@@ -572,6 +706,28 @@ FMX_EXPORT int fmx_head_norm_gate(const float* o, const void* gate, long long ga
     return fmx_fail("fmx_head_norm_gate: bad sizes T=%d H=%d Dv=%d", T, H, Dv);
   const long long items = (long long)T * H, grid = (items + 3) / 4;
   if (grid > 2147483647LL) return fmx_fail("fmx_head_norm_gate: batch too large");
+  const bool vec = (Dv == 32 || Dv == 64 || Dv == 128) && gate_stride % 4 == 0 && out_stride % 4 == 0 && ((uintptr_t)o & 15) == 0 &&
+                   ((uintptr_t)w & 15) == 0 && ((uintptr_t)gate & (g_dtype == FMX_F32 ? 15 : 7)) == 0 &&
+                   ((uintptr_t)out & (dtype == FMX_F32 ? 15 : 7)) == 0;
+#define FMX_HNG_V(TG, TO, LG)                                                                                          \
+  fmx_launch(head_norm_gate_vec_kernel<TG, TO, LG>, dim3((unsigned)((items + 128 / (LG) - 1) / (128 / (LG)))), dim3(128), 0, stream, o, \
+             (const TG*)gate, gate_stride, w, (TO*)out, out_stride, items, H, eps, silu)
+#define FMX_HNG_VEC(TG, TO)                                                                                            \
+  do {                                                                                                                 \
+    if (Dv == 32) FMX_HNG_V(TG, TO, 8);                                                                                \
+    else if (Dv == 64) FMX_HNG_V(TG, TO, 16);                                                                          \
+    else FMX_HNG_V(TG, TO, 32);                                                                                        \
+  } while (0)
+  if (vec) {
+    if (g_dtype == FMX_F32 && dtype == FMX_F32) FMX_HNG_VEC(float, float);
+    else if (g_dtype == FMX_F32 && dtype == FMX_BF16) FMX_HNG_VEC(float, bf16);
+    else if (g_dtype == FMX_BF16 && dtype == FMX_BF16) FMX_HNG_VEC(bf16, bf16);
+    else return fmx_fail("fmx_head_norm_gate: unknown dtypes %d, %d", g_dtype, dtype);
+    FMX_LAUNCH_CHECK();
+    return 0;
+  }
+#undef FMX_HNG_VEC
+#undef FMX_HNG_V
 #define FMX_HNG(TG, TO)                                                                                                \
   fmx_launch(head_norm_gate_kernel<TG, TO>, dim3((unsigned)grid), dim3(128), 0, stream, o, (const TG*)gate, gate_stride, w, (TO*)out, \
              out_stride, items, H, Dv, eps, silu)

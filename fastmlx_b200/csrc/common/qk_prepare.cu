@@ -49,7 +49,8 @@ qk_prepare_kernel(const TI* qkv, long long row_stride, const int* positions, con
   const int off = slot >= 0 ? (int)(slot - page * page_size) : 0;
   const long long page_elems = (long long)nkv * page_size * (hd + vd);
   __syncthreads();
-  for (int h = warp; h < nh + nkv; h += QKP_WARPS) {
+  // the grid's y shares a token's heads out over blocks; the first block takes the values too
+  for (int h = blockIdx.y * QKP_WARPS + warp; h < nh + nkv; h += QKP_WARPS * gridDim.y) {
     const TI* src = row + (long long)h * hd;
     const float* hw = h < nh ? q_weight : k_weight;
     float ss0 = 0.f;
@@ -113,7 +114,7 @@ qk_prepare_kernel(const TI* qkv, long long row_stride, const int* positions, con
     }
     __syncwarp();
   }
-  if (slot < 0) return;
+  if (slot < 0 || blockIdx.y != 0) return;
   const TI* vsrc = row + (long long)(nh + nkv) * hd;
   const float* vbias = bias != nullptr ? bias + (long long)(nh + nkv) * hd : nullptr;
   T* vdst = kv + page * page_elems + (long long)nkv * page_size * hd;
@@ -235,8 +236,11 @@ FMX_EXPORT int fmx_qk_prepare_ex(const void* qkv, long long row_stride, const in
   if (rot > 0 && inv_freq == nullptr) return fmx_fail("fmx_qk_prepare: rot=%d needs a frequency table", rot);
   if (row_stride < (long long)(nh + nkv) * hd + (long long)nkv * vd) return fmx_fail("fmx_qk_prepare: row stride too small");
   const size_t smem = ((size_t)rot + (size_t)QKP_WARPS * hd) * sizeof(float);
+  // few tokens: a warp per head, so that the heads are not walked one after another; many: a few heads per warp
+  const int passes = (nh + nkv + QKP_WARPS - 1) / QKP_WARPS;
+  const int head_blocks = passes < 1 ? 1 : T <= 256 ? passes : (passes + 2) / 3;
 #define FMX_QKP(TI, TKV)                                                                                                  \
-  fmx_launch(qk_prepare_kernel<TI, TKV>, dim3(T), dim3(QKP_WARPS * 32), smem, stream, (const TI*)qkv, row_stride, positions, \
+  fmx_launch(qk_prepare_kernel<TI, TKV>, dim3(T, head_blocks), dim3(QKP_WARPS * 32), smem, stream, (const TI*)qkv, row_stride, positions, \
              inv_freq, slot_mapping, q_out, (TKV*)kv, nh, nkv, hd, vd, rot, interleaved, norm_eps, page_size, num_pages,  \
              status, bias, q_weight, k_weight, norm_first, amplitude, v_scale)
   if (in_dtype == FMX_F32 && dtype == FMX_F32)

@@ -1060,7 +1060,7 @@ def moe_grouped_gate_up(x, plan, gate_up, E: int, ff: int, limit: float, block: 
     else:
         w_up, stride = gate_up.data_ptr() + 2 * E * ff * K, ff * K
     call("bf16", "fmx_moe_grouped_gate_up", x.data_ptr(), x.stride(0), sorted_token.data_ptr(), sorted_w.data_ptr(),
-         tile_expert.data_ptr(), gate_up.data_ptr(), w_up, K, stride, y.data_ptr(), tiles, ff, K, float(limit), int(block), _stream())
+         tile_expert.data_ptr(), gate_up.data_ptr(), w_up, K, stride, y.data_ptr(), tiles, ff, K, float(limit), int(block), T, _stream())
     return y
 
 
@@ -1081,7 +1081,7 @@ def moe_grouped_down(y, plan, down, E: int, ff: int, stacked: bool = False, toke
         return out
     ldw, stride = (ff, d * ff) if stacked else (E * ff, ff)
     call("bf16", "fmx_moe_grouped_down", y.data_ptr(), sorted_token.data_ptr(), tile_expert.data_ptr(), down.data_ptr(), ldw, stride,
-         out.data_ptr(), tiles, d, ff, _stream())
+         out.data_ptr(), tiles, d, ff, int(tokens), _stream())
     return out
 
 

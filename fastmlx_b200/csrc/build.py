@@ -40,6 +40,7 @@ GROUPS = {
 }
 EXTRA_FLAGS = {"tc_expiry": ["-DFMX_WAIT_CYCLES=100000LL", "-DFMX_SKIP_LAST_STAGE=1"]}
 HEAD_DIMS = tuple(range(16, 257, 16))
+VALUE_DIMS = ((64, 128), (128, 64), (32, 64))     # (keys, values) of other widths that `build_all` builds ahead of a model
 MIXATTN_SIZES = (1, 2, 4, 8)          # values per lane (value heads up to 32 times that), and query heads per key head
 
 
@@ -190,6 +191,7 @@ def build(group: str, force: bool = False, verbose: bool = False) -> str:
 def build_all(force: bool = False, verbose: bool = False, head_dims=HEAD_DIMS) -> list[str]:
     """Every library: the plain groups and the attention kernels of every head size."""
     groups = [g for g in GROUPS if g not in ("attn", "mixattn") and sources(g)] + [f"attn_hd{hd}" for hd in head_dims] + \
+        [f"attn_hd{hd}_vd{vd}" for hd, vd in VALUE_DIMS if head_dims is HEAD_DIMS] + \
         [f"mixattn_v{v}_p{p}" for v in MIXATTN_SIZES for p in MIXATTN_SIZES]
     with ThreadPoolExecutor(max_workers=max(1, (os.cpu_count() or 2) // 2)) as ex:
         return list(ex.map(lambda g: build(g, force, verbose), groups))

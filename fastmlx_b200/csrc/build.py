@@ -40,7 +40,7 @@ GROUPS = {
 }
 EXTRA_FLAGS = {"tc_expiry": ["-DFMX_WAIT_CYCLES=100000LL", "-DFMX_SKIP_LAST_STAGE=1"]}
 HEAD_DIMS = tuple(range(16, 257, 16))
-VALUE_DIMS = ((64, 128), (128, 64), (32, 64))     # (keys, values) of other widths that `build_all` builds ahead of a model
+VALUE_DIMS = ((64, 32), (128, 64), (32, 64))      # (keys, values) of other widths that `build_all` builds ahead of a model
 MIXATTN_SIZES = (1, 2, 4, 8)          # values per lane (value heads up to 32 times that), and query heads per key head
 
 

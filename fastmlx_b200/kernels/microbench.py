@@ -166,7 +166,8 @@ def _channel(a) -> int:
     moved = lambda c: 2 * B * inner * N * 4 + T * (c + H * N + H + inner) * 4
     rows = [("channel_delta_prepare", delta, T * (C + H) * 2 + T * H * N * 4 + T * (C + H * N + H) * 4 + B * (taps - 1) * C * 8),
             ("channel_gla_prepare", gla, T * Cg * 2 + T * H * N * 4 + T * (Cg + H * N) * 4)]
-    for ln, cpt in ((0, 0),) + tuple((n, c) for n in (8, 16, 32) for c in (1, 2, 4) if 4 * c <= n and 4 * n < N + 32 <= 8 * n + 32):
+    for ln, cpt in ((0, 0),) + tuple((n, c) for n in ((8, 16) if N <= 64 else (16,) if N <= 128 else (32,))
+                             for c in (1, 2, 4) if 4 * c <= n):
         rows += [(f"delta_scan lanes={ln} cpt={cpt}", lambda ln=ln, cpt=cpt: k.channel_scan(qkv, g, beta, ctx, state, H, G, N, P, ln, cpt), moved(C)),
                  (f"gla_scan lanes={ln} cpt={cpt}", lambda ln=ln, cpt=cpt: k.channel_scan(qkv2, g2, None, ctx, state, H, H, N, P, ln, cpt), moved(Cg))]
     rows += [("head_norm_gate", lambda: k.head_norm_gate(o, z[:, H * N:], norm_w, 1e-6, H, P, torch.bfloat16), T * inner * (4 + 4 + 2)),
@@ -200,6 +201,11 @@ def _attn_masked(a) -> int:
     cases = [("window", lambda: k.paged_attention_wide(qq, kv, ctx, grp, nh, nkv, hd, hd ** -0.5, 30.0, span), seen, kvb(span + q)),
              ("runs of positions, one more term", lambda: k.paged_attention_wide(qq, kv, ctx, grp, nh, nkv, hd, hd ** -0.5, 30.0, 0, chunk=span, sinks=sinks0),
               seen_c, kvb((c + q - 1) % span + 1 if q == 1 else span))]
+    if hd <= 128:                                   # values twice as wide as keys: another library of the same kernel
+        kv2 = torch.randn(B * per + 8, nkv * ps * 3 * hd, device=DEV).bfloat16()
+        cases.append(("window, values twice as wide", lambda: k.paged_attention_wide(qq, kv2, ctx, grp, nh, nkv, hd, hd ** -0.5, 0.0, span, vd=2 * hd),
+                      1.5 * seen, 1.5 * kvb(span + q)))
+        cases.append(("window, no cap", lambda: k.paged_attention_wide(qq, kv, ctx, grp, nh, nkv, hd, hd ** -0.5, 0.0, span), seen, kvb(span + q)))
     lat = torch.randn(B * per + 8, 1, 1, ps, hd, device=DEV).bfloat16()
     every = sum(p + 1 for p in range(c, c + q)) * B
     cases += [("latent, causal", lambda: k.paged_attention_wide(qq, lat, ctx, grp, nh, 1, hd, hd ** -0.5, 0.0, 0), every, B * (c + q) * hd * 2),

@@ -14,7 +14,8 @@
 //
 // Epilogues: bias; residual add (in place when out is the residual); SiLU(gate) * up for a
 // weight whose rows alternate in blocks of `blk` gate rows and their `blk` up rows; an
-// activation of the product (blk = -1: relu(x)^2, -2: gelu in its tanh form, -3: silu).
+// activation of the product (blk = -1 - kind, kinds as in activations.cuh), which a gate per row may multiply.
+#include "activations.cuh"
 #include "common.cuh"
 
 namespace {
@@ -53,8 +54,10 @@ template <int NT, bool HI, bool DUAL, int U, int WARPS, typename TO, bool GREEDY
 __global__ void __launch_bounds__(WARPS * 32)
 gemv_kernel(const bf16* x, long long ldx, const bf16* __restrict__ W, long long ldw, const float* __restrict__ bias,
             const bf16* residual, long long ldr, TO* out, long long ldo, int M, int N, int K, int blk_in,
-            GreedyOut greedy = GreedyOut{nullptr, nullptr, nullptr, 0}) {
-  // a gated product's block size carries the gate's activation above GATE_SHIFT (0: silu, 1: the tanh form of gelu)
+            GreedyOut greedy = GreedyOut{nullptr, nullptr, nullptr, 0}, float limit = 0.f, const float* row_gate = nullptr,
+            long long row_gate_stride = 0) {
+  // a gated product's block size carries the gate's activation above GATE_SHIFT (0: silu, 1: the tanh form of gelu, 2: the clamped
+  // form with `limit`)
   const int gate_kind = DUAL ? (blk_in >> GATE_SHIFT) : 0;
   const int blk = DUAL ? (blk_in & ((1 << GATE_SHIFT) - 1)) : blk_in;
   constexpr int TILES = DUAL ? 2 * NT : NT;
@@ -181,16 +184,12 @@ gemv_kernel(const bf16* x, long long ldx, const bf16* __restrict__ W, long long 
 #pragma unroll
       for (int w = 0; w < WARPS; ++w) up += red[w][NT + i][tok][f];
       const float gte = bf16r(v);
-      const float act = gate_kind == 1 ? 0.5f * gte * (1.0f + tanhf(0.7978845608028654f * (gte + 0.044715f * gte * gte * gte)))
-                                       : gte / (1.0f + expf(-gte));
-      v = act * bf16r(up);
+      v = gate_kind == 2 ? clamped_gate(gte, bf16r(up), limit) : act_f(gate_kind == 1 ? 1 : 2, gte) * bf16r(up);
     }
     if (bias != nullptr) v += bias[n];
     if (!DUAL && blk < 0) {                         // as the unfused path rounds: the product first, then its activation
-      const float z = bf16r(v);
-      if (blk == -1) { const float p = fmaxf(z, 0.f); v = p * p; }
-      else if (blk == -2) v = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-      else v = z / (1.0f + expf(-z));
+      v = act_f(-1 - blk, bf16r(v));
+      if (row_gate != nullptr) v *= sigmoid_f(row_gate[(long long)tok * row_gate_stride]);
     }
     if (residual != nullptr) v = bf16r(v) + __bfloat162float(residual[(long long)tok * ldr + n]);
     store_out<TO>(out + (long long)tok * ldo + n, v);
@@ -223,11 +222,12 @@ gemv_kernel(const bf16* x, long long ldx, const bf16* __restrict__ W, long long 
 
 template <int NT, bool HI, bool DUAL, int U, int WARPS, typename TO>
 void launch(const void* x, long long ldx, const void* W, long long ldw, const float* bias, const void* residual,
-            long long ldr, void* out, long long ldo, int M, int N, int K, int blk, cudaStream_t stream) {
+            long long ldr, void* out, long long ldo, int M, int N, int K, int blk, float limit, const float* row_gate,
+            long long row_gate_stride, cudaStream_t stream) {
   const int n_out = DUAL ? N / 2 : N;
   fmx_launch(gemv_kernel<NT, HI, DUAL, U, WARPS, TO>, dim3((n_out + 8 * NT - 1) / (8 * NT)), dim3(WARPS * 32), 0, stream,
              (const bf16*)x, ldx, (const bf16*)W, ldw, bias, (const bf16*)residual, ldr, (TO*)out, ldo, M, N, K, blk,
-             GreedyOut{nullptr, nullptr, nullptr, 0});
+             GreedyOut{nullptr, nullptr, nullptr, 0}, limit, row_gate, row_gate_stride);
 }
 }  // namespace
 
@@ -248,10 +248,10 @@ FMX_EXPORT int fmx_gemv_argmax(const void* x, long long ldx, const void* W, long
   const dim3 grid(blocks < resident ? blocks : resident);
   if (M > 8)
     fmx_launch(gemv_kernel<4, true, false, 2, 8, float, true>, grid, dim3(256), 0, stream, (const bf16*)x, ldx, (const bf16*)W, ldw,
-               (const float*)nullptr, (const bf16*)nullptr, 0LL, (float*)nullptr, 0LL, M, N, K, 0, g);
+               (const float*)nullptr, (const bf16*)nullptr, 0LL, (float*)nullptr, 0LL, M, N, K, 0, g, 0.f, (const float*)nullptr, 0LL);
   else
     fmx_launch(gemv_kernel<4, false, false, 4, 8, float, true>, grid, dim3(256), 0, stream, (const bf16*)x, ldx, (const bf16*)W, ldw,
-               (const float*)nullptr, (const bf16*)nullptr, 0LL, (float*)nullptr, 0LL, M, N, K, 0, g);
+               (const float*)nullptr, (const bf16*)nullptr, 0LL, (float*)nullptr, 0LL, M, N, K, 0, g, 0.f, (const float*)nullptr, 0LL);
   FMX_LAUNCH_CHECK();
   return 0;
 }
@@ -275,19 +275,22 @@ FMX_EXPORT int fmx_gemv_plan_warps(int n_out, int K, int wide, int sms) {
 // x [M <= 16, K] and W [N, K] bfloat16, rows 16-byte aligned; out [M, N] bfloat16 (out_dtype 1)
 // or float (0); bias float[N] or null; residual bfloat16 [M, n_out] or null (may be `out`).
 // blk > 0: W's rows alternate in blocks of blk gate rows and blk up rows, out is [M, N/2] =
-// silu(gate) * up in bfloat16 (blk + (1 << 20): the tanh form of gelu instead of silu).  blk < 0: out = act(product + bias) in bfloat16, act = relu^2 (-1), gelu-tanh (-2), silu (-3).  wide: 8, 16 or 32 output features per block; warps: 8 or 16
+// silu(gate) * up in bfloat16 (blk + (1 << 20): the tanh form of gelu instead of silu).  blk < 0: out = act(product + bias) in bfloat16, act = relu^2 (-1), gelu-tanh (-2), silu (-3), gelu (-4).
+// limit: of the clamped gate (blk + (2 << 20)); row_gate (blk < 0, may be null): out is multiplied by sigmoid(row_gate[row * stride]).
+// wide: 8, 16 or 32 output features per block; warps: 8 or 16
 // per block (16 when few blocks must keep many bytes in flight over a long K).
-FMX_EXPORT int fmx_gemv(const void* x, long long ldx, const void* W, long long ldw, const float* bias, const void* residual,
-                        long long ldr, void* out, long long ldo, int M, int N, int K, int out_dtype, int blk, int wide,
-                        int warps, cudaStream_t stream) {
+FMX_EXPORT int fmx_gemv_ex(const void* x, long long ldx, const void* W, long long ldw, const float* bias, const void* residual,
+                           long long ldr, void* out, long long ldo, int M, int N, int K, int out_dtype, int blk, int wide,
+                           int warps, float limit, const float* row_gate, long long row_gate_stride, cudaStream_t stream) {
   if (M == 0 || N == 0) return 0;
   if (M < 0 || M > 16 || N < 0 || K <= 0) return fmx_fail("fmx_gemv: takes 1..16 rows, got M=%d N=%d K=%d", M, N, K);
   if (K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)x & 15) || ((uintptr_t)W & 15))
     return fmx_fail("fmx_gemv: rows must be 16-byte aligned (K=%d ldx=%lld ldw=%lld)", K, ldx, ldw);
   const int gate_flag = blk > 0 ? (blk >> GATE_SHIFT) << GATE_SHIFT : 0;
   if (blk > 0) blk -= gate_flag;
-  if (gate_flag >> GATE_SHIFT > 1) return fmx_fail("fmx_gemv: the gate's activation is silu (0) or gelu (1), not %d", gate_flag >> GATE_SHIFT);
-  if (blk < -3 || blk == 0 && gate_flag || (blk > 0 && (blk % 16 || N % (2 * blk))))
+  if (gate_flag >> GATE_SHIFT > 2) return fmx_fail("fmx_gemv: the gate's activation is silu (0), gelu (1) or clamped (2), not %d", gate_flag >> GATE_SHIFT);
+  if (row_gate != nullptr && blk >= 0) return fmx_fail("fmx_gemv: a gate per row goes with an activation of the product");
+  if (blk < -FMX_ACTS || blk == 0 && gate_flag || (blk > 0 && (blk % 16 || N % (2 * blk))))
     return fmx_fail("fmx_gemv: gate/up blocks of %d do not tile %d rows", blk, N);
   if (blk < 0 && out_dtype != FMX_BF16) return fmx_fail("fmx_gemv: an activation epilogue writes bfloat16");
   if (blk > 0 && out_dtype != FMX_BF16) return fmx_fail("fmx_gemv: the SiLU-mul epilogue writes bfloat16");
@@ -300,7 +303,7 @@ FMX_EXPORT int fmx_gemv(const void* x, long long ldx, const void* W, long long l
   if (wide != 8 && wide != 16 && wide != 32) return fmx_fail("fmx_gemv: 8, 16 or 32 features per block, not %d", wide);
   if (blk > 0 && blk % wide) return fmx_fail("fmx_gemv: %d features per block do not tile gate/up blocks of %d", wide, blk);
 #define FMX_GV1(NT_, HI_, DUAL_, U_, W_, TO_) \
-  launch<NT_, HI_, DUAL_, U_, W_, TO_>(x, ldx, W, ldw, bias, residual, ldr, out, ldo, M, N, K, blk | gate_flag, stream)
+  launch<NT_, HI_, DUAL_, U_, W_, TO_>(x, ldx, W, ldw, bias, residual, ldr, out, ldo, M, N, K, blk | gate_flag, limit, row_gate, row_gate_stride, stream)
 #define FMX_GV(NT_, HI_, DUAL_, U_, TO_)                 \
   do {                                                   \
     if (warps == 16) FMX_GV1(NT_, HI_, DUAL_, U_, 16, TO_); \
@@ -329,4 +332,10 @@ FMX_EXPORT int fmx_gemv(const void* x, long long ldx, const void* W, long long l
 #undef FMX_GV
   FMX_LAUNCH_CHECK();
   return 0;
+}
+
+FMX_EXPORT int fmx_gemv(const void* x, long long ldx, const void* W, long long ldw, const float* bias, const void* residual,
+                        long long ldr, void* out, long long ldo, int M, int N, int K, int out_dtype, int blk, int wide,
+                        int warps, cudaStream_t stream) {
+  return fmx_gemv_ex(x, ldx, W, ldw, bias, residual, ldr, out, ldo, M, N, K, out_dtype, blk, wide, warps, 0.f, nullptr, 0, stream);
 }

@@ -11,10 +11,12 @@
 // U = X W_up^T side by side (mma.sync m16n8k16, bf16 in, 32-bit sums, a three-stage cp.async ring of tiles of 32 along K),
 // and in the epilogue y = w * g' sigmoid(1.702 g') (u' + 1), g' = min(G, limit), u' = clamp(U, -limit, limit) (with limit < 0:
 // y = w silu(G) U), w the
-// pair's weight; rows are gathered from the step's activations by token.  fmx_moe_grouped_down: pair outputs
+// pair's weight; rows are gathered from the step's activations by token.  fmx_moe_grouped_up: the same for experts without a
+// gate, 128 x 128 per tile: y = w act(X W_up^T), or act(w X W_up^T).  fmx_moe_grouped_down: pair outputs
 // Y W_down^T in 32-bit, 128 x 128 per tile.  fmx_moe_combine: a token's pair outputs added in the order of its choices, plus the shared
 // expert's output, rounded once.
 #include <math.h>
+#include "activations.cuh"
 #include "common.cuh"
 
 namespace {
@@ -22,7 +24,9 @@ constexpr int BM = 128, BK = 32, ROWP = BK + 8, THREADS = 256;
 // ROWS: the rows of a tile that may hold pairs.  A token takes an expert once, so a step of T tokens puts at most T pairs
 // into an expert's first tile: steps of few tokens keep fewer rows of A and a deeper ring of the weights' tiles, whose
 // bytes in flight are what they are bound by.
-template <bool GATED, int ROWS> struct Tile {
+enum Mode { DOWN = 0, GATED_UP = 1, PLAIN_UP = 2 };
+template <int MODE, int ROWS> struct Tile {
+  static constexpr bool GATED = MODE == GATED_UP;
   static constexpr int STAGES = ROWS <= 16 ? 8 : ROWS <= 64 ? 6 : 3;
   static constexpr int BN = GATED ? 64 : 128;            // hidden columns (of gate and of up), or output columns
   static constexpr int WM = GATED ? 4 : 2, WN = GATED ? 2 : 4;      // warps along rows and columns
@@ -119,14 +123,16 @@ __device__ __forceinline__ void warp_step(float (&acc)[MT][4][4], const bf16* as
   }
 }
 
-// GATED: W0 = the expert's gate rows, W1 = its up rows, out = activation (bf16); else W0 alone, out = product (32-bit).
-// Rows of padding are neither read nor written.
-template <bool GATED, int ROWS>
+// GATED_UP: W0 = the expert's gate rows, W1 = its up rows, out = activation (bf16).  PLAIN_UP: W0 = its up rows, out = activation `act`
+// (bf16), weighed behind it or (pre) in front of it.  DOWN: W0 alone, out = product (32-bit).  Rows of padding are neither
+// read nor written.
+template <int MODE, int ROWS>
 __global__ void __launch_bounds__(THREADS)
 moe_grouped_kernel(const bf16* a, long long lda, const int* sorted_token, const float* sorted_w, const int* tile_expert,
                    const bf16* w0, const bf16* w1, long long ldw, long long expert_stride, void* out, long long ldo, int N,
-                   int K, float limit, int block) {
-  using TL = Tile<GATED, ROWS>;
+                   int K, float limit, int block, int act, int pre) {
+  using TL = Tile<MODE, ROWS>;
+  constexpr bool GATED = MODE == GATED_UP, GATHER = MODE != DOWN;
   constexpr int BN = TL::BN, MT = TL::MT, STAGES = TL::STAGES;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* smem = reinterpret_cast<bf16*>(smem_raw);
@@ -155,8 +161,8 @@ moe_grouped_kernel(const bf16* a, long long lda, const int* sorted_token, const 
       if ((ROWS * (BK / 8)) % THREADS != 0 && item >= ROWS * (BK / 8)) break;
       const int r = item / (BK / 8), ch = item - r * (BK / 8);
       const int k = k0 + ch * 8;
-      const int tok = toks[r];                       // rows of A: gathered by token (GATED), or the sorted rows themselves
-      const long long arow = GATED ? tok : row0 + r;
+      const int tok = toks[r];                       // rows of A: gathered by token, or the sorted rows themselves
+      const long long arow = GATHER ? tok : row0 + r;
       const bool av = k < K && tok >= 0;
       cp16(stage_a(stage) + r * ROWP + ch * 8, av ? a + arow * lda + k : a, av);
     }
@@ -211,7 +217,7 @@ moe_grouped_kernel(const bf16* a, long long lda, const int* sorted_token, const 
       const int r = am + 16 * i + gq + 8 * x;
       const long long row = row0 + r;
       if (toks[r] < 0) continue;
-      const float w = GATED ? sorted_w[row] : 0.f;
+      const float w = GATHER ? sorted_w[row] : 0.f;
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int n = n0 + bn + 8 * j + 2 * tq;
@@ -223,11 +229,12 @@ moe_grouped_kernel(const bf16* a, long long lda, const int* sorted_token, const 
             if (limit < 0.f) {
               y = w * (g / (1.0f + expf(-g))) * u;
             } else {
-              g = fminf(g, limit);
-              u = fminf(fmaxf(u, -limit), limit);
-              y = w * (g / (1.0f + expf(-1.702f * g))) * (u + 1.0f);
+              y = w * clamped_gate(g, u, limit);
             }
             reinterpret_cast<bf16*>(out)[row * ldo + n + c] = __float2bfloat16_rn(y);
+          } else if (MODE == PLAIN_UP) {
+            const float u = acc0[i][j][2 * x + c];
+            reinterpret_cast<bf16*>(out)[row * ldo + n + c] = __float2bfloat16_rn(pre ? act_f(act, w * u) : w * act_f(act, u));
           } else {
             reinterpret_cast<float*>(out)[row * ldo + n + c] = acc0[i][j][2 * x + c];
           }
@@ -343,19 +350,49 @@ FMX_EXPORT int fmx_moe_grouped_gate_up(const void* x, long long ldx, const int* 
   cudaError_t e = cudaSuccess;
 #define FMX_MGU(ROWS)                                                                                                  \
   do {                                                                                                                 \
-    using TL = Tile<true, ROWS>;                                                                                       \
-    static const cudaError_t set = cudaFuncSetAttribute(moe_grouped_kernel<true, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TL::SMEM); \
+    using TL = Tile<GATED_UP, ROWS>;                                                                                       \
+    static const cudaError_t set = cudaFuncSetAttribute(moe_grouped_kernel<GATED_UP, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TL::SMEM); \
     e = set;                                                                                                           \
     if (e == cudaSuccess)                                                                                              \
-      fmx_launch(moe_grouped_kernel<true, ROWS>, dim3((ff + TL::BN - 1) / TL::BN, max_tiles), dim3(THREADS), TL::SMEM, stream, (const bf16*)x, \
+      fmx_launch(moe_grouped_kernel<GATED_UP, ROWS>, dim3((ff + TL::BN - 1) / TL::BN, max_tiles), dim3(THREADS), TL::SMEM, stream, (const bf16*)x, \
                  ldx, sorted_token, sorted_w, tile_expert, (const bf16*)w_gate, (const bf16*)w_up, ldw, expert_stride, y, (long long)ff, ff, K, \
-                 limit, block);                                                                                        \
+                 limit, block, 0, 0);                                                                                      \
   } while (0)
   if (tokens > 0 && tokens <= 16) FMX_MGU(16);
   else if (tokens > 0 && tokens <= 64) FMX_MGU(64);
   else FMX_MGU(128);
 #undef FMX_MGU
   if (e != cudaSuccess) return fmx_fail("fmx_moe_grouped_gate_up: shared memory refused: %s", cudaGetErrorString(e));
+  FMX_LAUNCH_CHECK();
+  return 0;
+}
+
+// The same for experts without a gate: w_up: expert e's ff rows start e * expert_stride elements in, rows of ldw; y [max_tiles * 128, ff]
+// bf16 = w act(x w_up^T), or act(w x w_up^T) with pre.
+FMX_EXPORT int fmx_moe_grouped_up(const void* x, long long ldx, const int* sorted_token, const float* sorted_w,
+                                  const int* tile_expert, const void* w_up, long long ldw, long long expert_stride, void* y,
+                                  int max_tiles, int ff, int K, int act, int pre, int tokens, cudaStream_t stream) {
+  if (max_tiles <= 0) return 0;
+  if (ff <= 0 || K <= 0 || K % 8 || ldx % 8 || ldw % 8 || expert_stride % 8 || ((uintptr_t)x & 15) || ((uintptr_t)w_up & 15))
+    return fmx_fail("fmx_moe_grouped_up: rows of 16 bytes wanted (K=%d)", K);
+  if (act < 0 || act >= FMX_ACTS) return fmx_fail("fmx_moe_grouped_up: unknown activation %d", act);
+  if (max_tiles > 65535) return fmx_fail("fmx_moe_grouped_up: too many tiles for one launch");
+  cudaError_t e = cudaSuccess;
+#define FMX_MPU(ROWS)                                                                                                  \
+  do {                                                                                                                 \
+    using TL = Tile<PLAIN_UP, ROWS>;                                                                                   \
+    static const cudaError_t set = cudaFuncSetAttribute(moe_grouped_kernel<PLAIN_UP, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TL::SMEM); \
+    e = set;                                                                                                           \
+    if (e == cudaSuccess)                                                                                              \
+      fmx_launch(moe_grouped_kernel<PLAIN_UP, ROWS>, dim3((ff + TL::BN - 1) / TL::BN, max_tiles), dim3(THREADS), TL::SMEM, stream, (const bf16*)x, \
+                 ldx, sorted_token, sorted_w, tile_expert, (const bf16*)w_up, (const bf16*)nullptr, ldw, expert_stride, y, (long long)ff, ff, K, \
+                 0.f, 0, act, pre);                                                                                    \
+  } while (0)
+  if (tokens > 0 && tokens <= 16) FMX_MPU(16);
+  else if (tokens > 0 && tokens <= 64) FMX_MPU(64);
+  else FMX_MPU(128);
+#undef FMX_MPU
+  if (e != cudaSuccess) return fmx_fail("fmx_moe_grouped_up: shared memory refused: %s", cudaGetErrorString(e));
   FMX_LAUNCH_CHECK();
   return 0;
 }
@@ -372,13 +409,13 @@ FMX_EXPORT int fmx_moe_grouped_down(const void* y, const int* sorted_token, cons
   cudaError_t e = cudaSuccess;
 #define FMX_MGD(ROWS)                                                                                                  \
   do {                                                                                                                 \
-    using TL = Tile<false, ROWS>;                                                                                      \
-    static const cudaError_t set = cudaFuncSetAttribute(moe_grouped_kernel<false, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TL::SMEM); \
+    using TL = Tile<DOWN, ROWS>;                                                                                      \
+    static const cudaError_t set = cudaFuncSetAttribute(moe_grouped_kernel<DOWN, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TL::SMEM); \
     e = set;                                                                                                           \
     if (e == cudaSuccess)                                                                                              \
-      fmx_launch(moe_grouped_kernel<false, ROWS>, dim3((d + TL::BN - 1) / TL::BN, max_tiles), dim3(THREADS), TL::SMEM, stream, (const bf16*)y, \
+      fmx_launch(moe_grouped_kernel<DOWN, ROWS>, dim3((d + TL::BN - 1) / TL::BN, max_tiles), dim3(THREADS), TL::SMEM, stream, (const bf16*)y, \
                  (long long)ff, sorted_token, (const float*)nullptr, tile_expert, (const bf16*)w_down, (const bf16*)nullptr, ldw, \
-                 expert_stride, (void*)pair_out, (long long)d, d, ff, 0.f, 0);                                     \
+                 expert_stride, (void*)pair_out, (long long)d, d, ff, 0.f, 0, 0, 0);                                     \
   } while (0)
   if (tokens > 0 && tokens <= 16) FMX_MGD(16);
   else if (tokens > 0 && tokens <= 64) FMX_MGD(64);

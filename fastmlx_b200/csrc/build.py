@@ -32,6 +32,8 @@ GROUPS = {
     "tc": "tc",
     # linear attention with a decay per key channel (gated linear attention, the delta rule's form)
     "chan": "chan",
+    # the matrix memory with exponential gates
+    "mlstm": "mlstm",
     # host code: the native step executor (no kernel of its own)
     "host": "host",
     # the tensor-core product built for one test: a wait limit of 100,000 clocks and a producer that

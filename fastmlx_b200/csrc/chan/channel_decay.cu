@@ -13,12 +13,12 @@
 //                           state also moves it on, else conv_state_update does.
 //   channel_gla_prepare     per token: q scaled, k, v in 32-bit, g = sigmoid(z + bias)^(1/tau).
 //   channel_scan            the recurrence, see there.
-//   head_norm_gate          o of each head divided by its root mean square, times a weight, times sigmoid or silu of a gate.
 //
 // Everything is 32-bit but the projections that come in and the activations that go out.
 #include <math.h>
 #include "common.cuh"
 #include "conv_state.cuh"
+#include "packed.cuh"
 
 namespace {
 __device__ __forceinline__ float softplus_f(float a) { return fmaxf(a, 0.f) + log1pf(expf(-fabsf(a))); }
@@ -165,23 +165,6 @@ channel_gla_prepare_kernel(const T* proj, long long stride, const float* z, long
   }
 }
 
-// four neighbouring values of any element type in one access
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const bf16* p) {
-  const uint2 u = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
-  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
-  return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void store4(bf16* p, float4 v) {
-  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-  uint2 u;
-  u.x = *reinterpret_cast<unsigned*>(&a);
-  u.y = *reinterpret_cast<unsigned*>(&b);
-  *reinterpret_cast<uint2*>(p) = u;
-}
-
 // The same with four neighbouring columns per access (HD, C and every row start multiples of four).
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -205,54 +188,6 @@ channel_gla_prepare_vec_kernel(const T* proj, long long stride, const float* z, 
     store4(out_g + t * HD + e, make_float4(expf(-softplus_f(-x.x) * inv_tau), expf(-softplus_f(-x.y) * inv_tau),
                                            expf(-softplus_f(-x.z) * inv_tau), expf(-softplus_f(-x.w) * inv_tau)));
   }
-}
-
-// ---- pairs of floats in one 64-bit register: the packed multiply-add of sm_100
-typedef unsigned long long f32x2;
-__device__ __forceinline__ f32x2 pair_of(float lo, float hi) {
-  f32x2 r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
-  return r;
-}
-__device__ __forceinline__ float pair_sum(f32x2 a) {
-  float lo, hi;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(a));
-  return lo + hi;
-}
-__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
-  f32x2 r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-  return r;
-}
-__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
-  f32x2 r;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-  return r;
-}
-
-// NV values of every lane added up across L lanes (NV <= L, both powers of two): each round halves what a lane holds,
-// and lane `sub` is left with the sum of value sub * NV / L.  The pairs of lanes that meet are the same for every value.
-template <int NV, int L> __device__ __forceinline__ float reduce_scatter(float (&v)[NV], int sub) {
-  int d = L / 2;
-#pragma unroll
-  for (int w = NV / 2; w >= 1; w >>= 1, d >>= 1) {
-    const bool upper = (sub & d) != 0;
-#pragma unroll
-    for (int i = 0; i < w; ++i) {
-      const float give = upper ? v[i] : v[i + w], keep = upper ? v[i + w] : v[i];
-      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, d);
-    }
-  }
-#pragma unroll
-  for (int e = L / NV / 2; e >= 1; e >>= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], e);
-  return v[0];
-}
-// The same, and every lane gets all the sums.
-template <int NV, int L> __device__ __forceinline__ void all_reduce(float (&v)[NV], int sub) {
-  const float mine = reduce_scatter<NV, L>(v, sub);
-  const int base = (threadIdx.x & 31) - sub;
-#pragma unroll
-  for (int i = 0; i < NV; ++i) v[i] = __shfl_sync(0xffffffffu, mine, base + i * (L / NV));
 }
 
 // The recurrence over every row's tokens of a step, in order, from and into the rows' state slots.
@@ -507,53 +442,6 @@ channel_scan_kernel(const float* qkv, const float* decay, const float* beta, con
   }
 }
 
-// One warp per (token, head): out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * act(gate[t, h, :]), act sigmoid or silu.
-template <typename TG, typename T>
-__global__ void __launch_bounds__(128)
-head_norm_gate_kernel(const float* o, const TG* gate, long long gate_stride, const float* __restrict__ w, T* out,
-                      long long out_stride, long long n_items, int H, int Dv, float eps, int silu) {
-  pdl_wait();
-  pdl_trigger();
-  const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31;
-  if (item >= n_items) return;
-  const long long t = item / H;
-  const int h = (int)(item - t * H);
-  const float* op = o + item * Dv;
-  const TG* gp = gate + t * gate_stride + (long long)h * Dv;
-  T* dst = out + t * out_stride + (long long)h * Dv;
-  float ss = 0.f;
-  for (int e = lane; e < Dv; e += 32) ss = fmaf(op[e], op[e], ss);
-  const float rstd = 1.0f / sqrtf(warp_sum(ss) / (float)Dv + eps);
-  for (int e = lane; e < Dv; e += 32) {
-    const float x = to_f(gp[e]), sg = 1.0f / (1.0f + expf(-x));
-    dst[e] = from_f<T>(op[e] * rstd * w[e] * (silu ? x * sg : sg));
-  }
-}
-
-// The same with four neighbouring values per lane: LG = Dv / 4 lanes (8, 16 or 32) per (token, head).
-template <typename TG, typename T, int LG>
-__global__ void __launch_bounds__(128)
-head_norm_gate_vec_kernel(const float* o, const TG* gate, long long gate_stride, const float* __restrict__ w, T* out,
-                          long long out_stride, long long n_items, int H, float eps, int silu) {
-  pdl_wait();
-  pdl_trigger();
-  const long long item = (long long)blockIdx.x * (128 / LG) + threadIdx.x / LG;
-  const int e = 4 * (threadIdx.x % LG), Dv = 4 * LG;
-  const bool live = item < n_items;                // (every lane takes part in the exchange)
-  const long long t = live ? item / H : 0;
-  const int h = live ? (int)(item - t * H) : 0;
-  const float4 x = live ? load4(o + item * Dv + e) : make_float4(0.f, 0.f, 0.f, 0.f);
-  float ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w)));
-#pragma unroll
-  for (int d = LG / 2; d >= 1; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
-  if (!live) return;
-  const float rstd = 1.0f / sqrtf(ss / (float)Dv + eps);
-  const float4 g = load4(gate + t * gate_stride + (long long)h * Dv + e), ww = load4(w + e);
-  auto act = [&](float v) { const float sg = 1.0f / (1.0f + expf(-v)); return silu ? v * sg : sg; };
-  store4(out + t * out_stride + (long long)h * Dv + e, make_float4(x.x * rstd * ww.x * act(g.x), x.y * rstd * ww.y * act(g.y),
-                                                                  x.z * rstd * ww.z * act(g.z), x.w * rstd * ww.w * act(g.w)));
-}
 }  // namespace
 
 // single: every row of the step brings one token; the convolution state then moves on inside the kernel.
@@ -694,48 +582,6 @@ FMX_EXPORT int fmx_channel_scan(const float* qkv, const float* decay, const floa
 #undef FMX_CS_C
 #undef FMX_CS_G
 #undef FMX_CS
-  FMX_LAUNCH_CHECK();
-  return 0;
-}
-
-// o [T, H*Dv] 32-bit; gate rows of gate_stride elements of type g_dtype; out rows of out_stride elements of type dtype.
-FMX_EXPORT int fmx_head_norm_gate(const float* o, const void* gate, long long gate_stride, int g_dtype, const float* w, void* out,
-                                  long long out_stride, int dtype, int T, int H, int Dv, float eps, int silu, cudaStream_t stream) {
-  if (T == 0) return 0;
-  if (T < 0 || H <= 0 || Dv <= 0 || gate_stride < (long long)H * Dv || out_stride < (long long)H * Dv)
-    return fmx_fail("fmx_head_norm_gate: bad sizes T=%d H=%d Dv=%d", T, H, Dv);
-  const long long items = (long long)T * H, grid = (items + 3) / 4;
-  if (grid > 2147483647LL) return fmx_fail("fmx_head_norm_gate: batch too large");
-  const bool vec = (Dv == 32 || Dv == 64 || Dv == 128) && gate_stride % 4 == 0 && out_stride % 4 == 0 && ((uintptr_t)o & 15) == 0 &&
-                   ((uintptr_t)w & 15) == 0 && ((uintptr_t)gate & (g_dtype == FMX_F32 ? 15 : 7)) == 0 &&
-                   ((uintptr_t)out & (dtype == FMX_F32 ? 15 : 7)) == 0;
-#define FMX_HNG_V(TG, TO, LG)                                                                                          \
-  fmx_launch(head_norm_gate_vec_kernel<TG, TO, LG>, dim3((unsigned)((items + 128 / (LG) - 1) / (128 / (LG)))), dim3(128), 0, stream, o, \
-             (const TG*)gate, gate_stride, w, (TO*)out, out_stride, items, H, eps, silu)
-#define FMX_HNG_VEC(TG, TO)                                                                                            \
-  do {                                                                                                                 \
-    if (Dv == 32) FMX_HNG_V(TG, TO, 8);                                                                                \
-    else if (Dv == 64) FMX_HNG_V(TG, TO, 16);                                                                          \
-    else FMX_HNG_V(TG, TO, 32);                                                                                        \
-  } while (0)
-  if (vec) {
-    if (g_dtype == FMX_F32 && dtype == FMX_F32) FMX_HNG_VEC(float, float);
-    else if (g_dtype == FMX_F32 && dtype == FMX_BF16) FMX_HNG_VEC(float, bf16);
-    else if (g_dtype == FMX_BF16 && dtype == FMX_BF16) FMX_HNG_VEC(bf16, bf16);
-    else return fmx_fail("fmx_head_norm_gate: unknown dtypes %d, %d", g_dtype, dtype);
-    FMX_LAUNCH_CHECK();
-    return 0;
-  }
-#undef FMX_HNG_VEC
-#undef FMX_HNG_V
-#define FMX_HNG(TG, TO)                                                                                                \
-  fmx_launch(head_norm_gate_kernel<TG, TO>, dim3((unsigned)grid), dim3(128), 0, stream, o, (const TG*)gate, gate_stride, w, (TO*)out, \
-             out_stride, items, H, Dv, eps, silu)
-  if (g_dtype == FMX_F32 && dtype == FMX_F32) FMX_HNG(float, float);
-  else if (g_dtype == FMX_F32 && dtype == FMX_BF16) FMX_HNG(float, bf16);
-  else if (g_dtype == FMX_BF16 && dtype == FMX_BF16) FMX_HNG(bf16, bf16);
-  else return fmx_fail("fmx_head_norm_gate: unknown dtypes %d, %d", g_dtype, dtype);
-#undef FMX_HNG
   FMX_LAUNCH_CHECK();
   return 0;
 }

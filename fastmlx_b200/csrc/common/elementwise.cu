@@ -1,6 +1,7 @@
 // Row gather (token embedding, and the choice of the rows whose logits are wanted),
 // RMSNorm with the residual sum in front of it, and SiLU-and-multiply.
 #include <math.h>
+#include "activations.cuh"
 #include "common.cuh"
 
 // out[t, :] = table[ids[t], :] * scale in 32-bit: an embedding that is multiplied by a constant and starts the
@@ -98,7 +99,7 @@ FMX_EXPORT int fmx_gather_rows(const void* table, const int* ids, void* out, int
 // sum of squares is taken in a fixed order that depends on the row's width only.
 template <typename T, typename TR, int BLOCK>
 __global__ void add_rmsnorm_kernel(const T* x, TR* residual, const float* __restrict__ w, T* __restrict__ out, int d,
-                                   float eps, int init) {
+                                   float eps, int init, const float* __restrict__ w2, T* __restrict__ out2) {
   pdl_wait();
   pdl_trigger();
   const long long row = blockIdx.x;
@@ -117,7 +118,11 @@ __global__ void add_rmsnorm_kernel(const T* x, TR* residual, const float* __rest
   ss = block_sum<BLOCK>(ss);
   const float rstd = 1.0f / sqrtf(ss / (float)d + eps);
   T* o = out + row * d;
-  for (int i = threadIdx.x; i < d; i += BLOCK) o[i] = from_f<T>((rr ? to_f(rr[i]) : to_f(xr[i])) * rstd * w[i]);
+  for (int i = threadIdx.x; i < d; i += BLOCK) {
+    const float v = (rr ? to_f(rr[i]) : to_f(xr[i])) * rstd;
+    o[i] = from_f<T>(v * w[i]);
+    if (out2 != nullptr) out2[row * d + i] = from_f<T>(v * w2[i]);
+  }
 }
 
 // bfloat16 rows whose width is a multiple of 8: 16-byte loads, the row kept in registers
@@ -127,7 +132,7 @@ __global__ void add_rmsnorm_kernel(const T* x, TR* residual, const float* __rest
 template <int BLOCK, int CH, bool RES_F32>
 __global__ void __launch_bounds__(BLOCK)
 add_rmsnorm_bf16_vec_kernel(const bf16* x, void* residual, const float* __restrict__ w, bf16* out, int d, float eps,
-                            int init) {
+                            int init, const float* __restrict__ w2, bf16* out2) {
   pdl_wait();
   pdl_trigger();
   const long long row = blockIdx.x;
@@ -192,6 +197,11 @@ add_rmsnorm_bf16_vec_kernel(const bf16* x, void* residual, const float* __restri
   const float rstd = 1.0f / sqrtf(ss / (float)d + eps);
   uint4* o = reinterpret_cast<uint4*>(out + row * d);
   const float4* w4 = reinterpret_cast<const float4*>(w);
+  for (int pass = 0; pass < (out2 != nullptr ? 2 : 1); ++pass) {
+  if (pass == 1) {
+    o = reinterpret_cast<uint4*>(out2 + row * d);
+    w4 = reinterpret_cast<const float4*>(w2);
+  }
 #pragma unroll
   for (int c = 0; c < CH; ++c) {
     const int i = threadIdx.x + c * BLOCK;
@@ -206,55 +216,62 @@ add_rmsnorm_bf16_vec_kernel(const bf16* x, void* residual, const float* __restri
       o[i] = r;
     }
   }
+  }
 }
 
 static bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 
 template <bool RES_F32>
 static void launch_add_rmsnorm_vec(const void* x, void* residual, const float* w, void* out, int rows, int d, float eps,
-                                   int init, cudaStream_t stream) {
+                                   int init, const float* w2, void* out2, cudaStream_t stream) {
   if (d <= 128 * 8)
     fmx_launch(add_rmsnorm_bf16_vec_kernel<128, 1, RES_F32>, dim3(rows), dim3(128), 0, stream, (const bf16*)x, residual, w,
-               (bf16*)out, d, eps, init);
+               (bf16*)out, d, eps, init, w2, (bf16*)out2);
   else if (d <= 256 * 8)
     fmx_launch(add_rmsnorm_bf16_vec_kernel<256, 1, RES_F32>, dim3(rows), dim3(256), 0, stream, (const bf16*)x, residual, w,
-               (bf16*)out, d, eps, init);
+               (bf16*)out, d, eps, init, w2, (bf16*)out2);
   else
     fmx_launch(add_rmsnorm_bf16_vec_kernel<256, 4, RES_F32>, dim3(rows), dim3(256), 0, stream, (const bf16*)x, residual, w,
-               (bf16*)out, d, eps, init);
+               (bf16*)out, d, eps, init, w2, (bf16*)out2);
 }
 
 // x, out: `dtype`; residual: `res_dtype` (float beside bfloat16 activations keeps the stream
 // unrounded), or null.  init != 0: the residual is written, not read (the stream's first value).
-// x may be null when there is a residual.
-FMX_EXPORT int fmx_add_rmsnorm(const void* x, void* residual, const float* w, void* out, int rows, int d, float eps,
-                               int dtype, int res_dtype, int init, cudaStream_t stream) {
+// x may be null when there is a residual.  w2 and out2 (both or neither): a second weight of the same normed sum, in the same pass.
+FMX_EXPORT int fmx_add_rmsnorm_pair(const void* x, void* residual, const float* w, void* out, const float* w2, void* out2, int rows,
+                                    int d, float eps, int dtype, int res_dtype, int init, cudaStream_t stream) {
   if (rows == 0) return 0;
   if (rows < 0 || d <= 0) return fmx_fail("fmx_add_rmsnorm: bad sizes rows=%d d=%d", rows, d);
+  if ((w2 == nullptr) != (out2 == nullptr)) return fmx_fail("fmx_add_rmsnorm: a second weight and a second output come together");
   if (x == nullptr && (residual == nullptr || init)) return fmx_fail("fmx_add_rmsnorm: nothing to normalise");
   if (residual != nullptr && res_dtype != dtype && !(dtype == FMX_BF16 && res_dtype == FMX_F32))
     return fmx_fail("fmx_add_rmsnorm: a residual of type %d beside activations of type %d", res_dtype, dtype);
   const bool res_f32 = residual != nullptr && res_dtype == FMX_F32;
   if (dtype == FMX_F32)
     fmx_launch(add_rmsnorm_kernel<float, float, 256>, dim3(rows), dim3(256), 0, stream, (const float*)x, (float*)residual, w,
-               (float*)out, d, eps, init);
+               (float*)out, d, eps, init, w2, (float*)out2);
   else if (dtype == FMX_BF16) {
-    const bool vec = d % 8 == 0 && d <= 256 * 8 * 4 && aligned16(x) && aligned16(out) && aligned16(w) &&
+    const bool vec = d % 8 == 0 && d <= 256 * 8 * 4 && aligned16(x) && aligned16(out) && aligned16(w) && aligned16(w2) && aligned16(out2) &&
                      (!residual || aligned16(residual));
     if (vec && res_f32)
-      launch_add_rmsnorm_vec<true>(x, residual, w, out, rows, d, eps, init, stream);
+      launch_add_rmsnorm_vec<true>(x, residual, w, out, rows, d, eps, init, w2, out2, stream);
     else if (vec)
-      launch_add_rmsnorm_vec<false>(x, residual, w, out, rows, d, eps, init, stream);
+      launch_add_rmsnorm_vec<false>(x, residual, w, out, rows, d, eps, init, w2, out2, stream);
     else if (res_f32)
       fmx_launch(add_rmsnorm_kernel<bf16, float, 256>, dim3(rows), dim3(256), 0, stream, (const bf16*)x, (float*)residual, w,
-                 (bf16*)out, d, eps, init);
+                 (bf16*)out, d, eps, init, w2, (bf16*)out2);
     else
       fmx_launch(add_rmsnorm_kernel<bf16, bf16, 256>, dim3(rows), dim3(256), 0, stream, (const bf16*)x, (bf16*)residual, w,
-                 (bf16*)out, d, eps, init);
+                 (bf16*)out, d, eps, init, w2, (bf16*)out2);
   } else
     return fmx_fail("fmx_add_rmsnorm: unknown dtype %d", dtype);
   FMX_LAUNCH_CHECK();
   return 0;
+}
+
+FMX_EXPORT int fmx_add_rmsnorm(const void* x, void* residual, const float* w, void* out, int rows, int d, float eps,
+                               int dtype, int res_dtype, int init, cudaStream_t stream) {
+  return fmx_add_rmsnorm_pair(x, residual, w, out, nullptr, nullptr, rows, d, eps, dtype, res_dtype, init, stream);
 }
 
 // out[t, i] = act(gate_i) * up_i in 32-bit, act = silu (g / (1 + exp(-g)), KIND 2) or the tanh form of gelu
@@ -373,7 +390,7 @@ FMX_EXPORT int fmx_fill_rows(const float* vec, void* out, int rows, int cols, lo
 }
 
 // Elementwise activations of a feed-forward's hidden layer, over rows that may be slices of wider buffers.
-// kind 0: relu(x)^2; 1: gelu, tanh form: 0.5 x (1 + tanh(sqrt(2/pi) (x + 0.044715 x^3))); 2: silu.
+// kind 0: relu(x)^2; 1: gelu, tanh form: 0.5 x (1 + tanh(sqrt(2/pi) (x + 0.044715 x^3))); 2: silu; 3: gelu, exact form.
 namespace {
 template <typename T>
 __global__ void activation_kernel(const T* x, long long x_stride, T* out, long long out_stride, long long rows, int cols,
@@ -385,11 +402,7 @@ __global__ void activation_kernel(const T* x, long long x_stride, T* out, long l
     const long long r = idx / cols;
     const int c = (int)(idx - r * cols);
     const float v = to_f(x[r * x_stride + c]);
-    float y;
-    if (kind == 0) { const float p = fmaxf(v, 0.f); y = p * p; }
-    else if (kind == 1) y = 0.5f * v * (1.0f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
-    else y = v / (1.0f + expf(-v));
-    out[r * out_stride + c] = from_f<T>(y);
+    out[r * out_stride + c] = from_f<T>(act_f(kind, v));
   }
 }
 }  // namespace
@@ -397,7 +410,7 @@ __global__ void activation_kernel(const T* x, long long x_stride, T* out, long l
 FMX_EXPORT int fmx_activation(const void* x, long long x_stride, void* out, long long out_stride, int rows, int cols,
                               int kind, int dtype, cudaStream_t stream) {
   if (rows == 0 || cols == 0) return 0;
-  if (rows < 0 || cols < 0 || kind < 0 || kind > 2) return fmx_fail("fmx_activation: bad arguments rows=%d cols=%d kind=%d", rows, cols, kind);
+  if (rows < 0 || cols < 0 || kind < 0 || kind >= FMX_ACTS) return fmx_fail("fmx_activation: bad arguments rows=%d cols=%d kind=%d", rows, cols, kind);
   const long long n = (long long)rows * cols, cap = (long long)fmx_num_sms() * 16;
   const int block = 256;
   const int grid = (int)((n + block - 1) / block < cap ? (n + block - 1) / block : cap);

@@ -1,6 +1,6 @@
 // A routed feed-forward's own kernels: the router's choice and the experts' activation.
 //
-// moe_route: one warp per token.  Scores s = softmax(z) over all E experts (32-bit).  With groups (E / groups
+// moe_route: one warp per token.  Scores s = softmax(z) over all E experts (32-bit), or sigmoid(z) each.  With groups (E / groups
 // neighbouring experts each), a group scores as its best member and only the `keep` best groups may be chosen from.
 // The `top` best allowed experts are chosen (the lower index on a tie); the token's weights are their scores as they
 // are, not renormalised.  Out: a dense row of weights [E], zero where an expert is not chosen, and the chosen
@@ -12,6 +12,7 @@
 // shared one); with limit < 0 the expert's form is silu(g) u instead.  A column whose expert the token did not choose is zero, so that one product with all the experts'
 // down matrices side by side gives the weighted sum.
 #include <math.h>
+#include "activations.cuh"
 #include "common.cuh"
 
 namespace {
@@ -29,7 +30,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const float* z, long long z_stride, int T, int E, int top, int groups, int keep, float* weights,
                  int* chosen, const float* __restrict__ choice_bias, float weight_scale,
-                 const float* __restrict__ logit_bias, int renorm) {
+                 const float* __restrict__ logit_bias, int renorm, int sigmoid) {
   extern __shared__ float smem[];               // per warp: E scores, E marks (as floats), `groups` group scores
   pdl_wait();
   pdl_trigger();
@@ -46,12 +47,12 @@ moe_route_kernel(const float* z, long long z_stride, int T, int E, int top, int 
   m = warp_max(m);
   float sum = 0.f;
   for (int e = lane; e < E; e += 32) {
-    const float p = expf(logit(e) - m);
+    const float p = sigmoid ? sigmoid_f(logit(e)) : expf(logit(e) - m);
     s[e] = p;
     sum += p;
   }
   sum = warp_sum(sum);
-  const float inv = renorm ? 1.0f : 1.0f / sum;  // renorm: the chosen experts' exponentials are divided by their own sum
+  const float inv = renorm || sigmoid ? 1.0f : 1.0f / sum;  // renorm: the chosen experts' exponentials are divided by their own sum
   for (int e = lane; e < E; e += 32) {
     s[e] *= inv;
     ok[e] = 1.f;
@@ -110,9 +111,7 @@ moe_route_kernel(const float* z, long long z_stride, int T, int E, int top, int 
 // limit >= 0: g' sigmoid(1.702 g') (u' + 1), clamped; limit < 0: silu(g) u.
 __device__ __forceinline__ float expert_act(float g, float u, float limit) {
   if (limit < 0.f) return g / (1.0f + expf(-g)) * u;
-  g = fminf(g, limit);
-  u = fminf(fmaxf(u, -limit), limit);
-  return (g / (1.0f + expf(-1.702f * g))) * (u + 1.0f);
+  return clamped_gate(g, u, limit);
 }
 
 template <typename T>
@@ -171,11 +170,12 @@ __global__ void moe_expert_act_vec_kernel(const bf16* gu, long long gu_stride, c
 
 // Experts without a gate, side by side: u[t] holds F = E * ff (+ a shared expert's) hidden values; y = w * act(u) with w
 // the token's weight for the column's expert, zero where it did not choose it.  The shared columns at the end weigh
-// sigmoid(shared_gate[t]) where a gate is given, else 1.  act: 0 relu^2, 1 gelu (tanh form), 2 silu.
+// sigmoid(shared_gate[t]) where a gate is given, else 1.  act: see activations.cuh.  pre: the experts' weights multiply the hidden
+// values in front of the activation (an expert's input is weighed, not its output); the shared columns' stays behind it.
 template <typename T>
 __global__ void moe_plain_act_kernel(const T* u, long long u_stride, const float* weights, const float* shared_gate,
                                      long long sg_stride, T* out, long long out_stride, long long rows, int E, int ff, int F,
-                                     int act) {
+                                     int act, int pre) {
   pdl_wait();
   pdl_trigger();
   const long long n = rows * F;
@@ -189,11 +189,7 @@ __global__ void moe_plain_act_kernel(const T* u, long long u_stride, const float
     float y = 0.f;
     if (w != 0.f) {
       const float x = to_f(u[r * u_stride + c]);
-      float a;
-      if (act == 0) { const float p = fmaxf(x, 0.f); a = p * p; }
-      else if (act == 1) a = 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
-      else a = x / (1.0f + expf(-x));
-      y = w * a;
+      y = pre && e < E ? act_f(act, w * x) : w * act_f(act, x);
     }
     out[r * out_stride + c] = from_f<T>(y);
   }
@@ -202,14 +198,14 @@ __global__ void moe_plain_act_kernel(const T* u, long long u_stride, const float
 
 // choice_bias ([E], may be null): added to the scores for the choice only; weight_scale multiplies the chosen scores;
 // logit_bias ([E], may be null): added to the logits; renorm (without groups): a token's weights are the softmax over its
-// chosen experts' logits alone.
+// chosen experts' logits alone; sigmoid (without renorm): scores are sigmoid(z), not the softmax.
 FMX_EXPORT int fmx_moe_route_ex(const float* z, long long z_stride, int T, int E, int top, int groups, int keep, float* weights,
                                 int* chosen, const float* choice_bias, float weight_scale, const float* logit_bias, int renorm,
-                                cudaStream_t stream);
+                                int sigmoid, cudaStream_t stream);
 FMX_EXPORT int fmx_moe_route_biased(const float* z, long long z_stride, int T, int E, int top, int groups, int keep,
                                     float* weights, int* chosen, const float* choice_bias, float weight_scale,
                                     cudaStream_t stream) {
-  return fmx_moe_route_ex(z, z_stride, T, E, top, groups, keep, weights, chosen, choice_bias, weight_scale, nullptr, 0, stream);
+  return fmx_moe_route_ex(z, z_stride, T, E, top, groups, keep, weights, chosen, choice_bias, weight_scale, nullptr, 0, 0, stream);
 }
 FMX_EXPORT int fmx_moe_route(const float* z, long long z_stride, int T, int E, int top, int groups, int keep, float* weights,
                              int* chosen, cudaStream_t stream) {
@@ -218,15 +214,16 @@ FMX_EXPORT int fmx_moe_route(const float* z, long long z_stride, int T, int E, i
 
 FMX_EXPORT int fmx_moe_route_ex(const float* z, long long z_stride, int T, int E, int top, int groups, int keep, float* weights,
                                 int* chosen, const float* choice_bias, float weight_scale, const float* logit_bias, int renorm,
-                                cudaStream_t stream) {
+                                int sigmoid, cudaStream_t stream) {
   if (T == 0) return 0;
+  if (renorm && sigmoid) return fmx_fail("fmx_moe_route: sigmoid scores are not renormalised");
   if (renorm && groups > 1 && keep < groups) return fmx_fail("fmx_moe_route: weights over the chosen logits alone come without groups");
   if (T < 0 || E <= 0 || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || z_stride < E)
     return fmx_fail("fmx_moe_route: bad sizes T=%d E=%d top=%d groups=%d keep=%d", T, E, top, groups, keep);
   const size_t smem = (size_t)ROUTE_WARPS * (2 * (size_t)E + groups) * sizeof(float);
   if (smem > 48 * 1024) return fmx_fail("fmx_moe_route: %d experts are more than the kernel's shared memory holds", E);
   fmx_launch(moe_route_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, stream, z, z_stride, T, E,
-             top, groups, keep, weights, chosen, choice_bias, weight_scale, logit_bias, renorm);
+             top, groups, keep, weights, chosen, choice_bias, weight_scale, logit_bias, renorm, sigmoid);
   FMX_LAUNCH_CHECK();
   return 0;
 }
@@ -264,7 +261,7 @@ namespace {
 // moe_plain_act for bfloat16 rows in 16-byte pieces (eight columns of one expert: ff and the experts' columns are multiples of 8).
 __global__ void moe_plain_act_vec_kernel(const bf16* u, long long u_stride, const float* weights, const float* shared_gate,
                                          long long sg_stride, bf16* out, long long out_stride, long long rows, int E, int ff,
-                                         int F, int act) {
+                                         int F, int act, int pre) {
   pdl_wait();
   pdl_trigger();
   const int f8 = F / 8;
@@ -284,13 +281,8 @@ __global__ void moe_plain_act_vec_kernel(const bf16* u, long long u_stride, cons
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const float2 x = __bfloat1622float2(up[i]);
-        float a0, a1;
-        if (act == 0) { const float p0 = fmaxf(x.x, 0.f), p1 = fmaxf(x.y, 0.f); a0 = p0 * p0; a1 = p1 * p1; }
-        else if (act == 1) {
-          a0 = 0.5f * x.x * (1.0f + tanhf(0.7978845608028654f * (x.x + 0.044715f * x.x * x.x * x.x)));
-          a1 = 0.5f * x.y * (1.0f + tanhf(0.7978845608028654f * (x.y + 0.044715f * x.y * x.y * x.y)));
-        } else { a0 = x.x / (1.0f + expf(-x.x)); a1 = x.y / (1.0f + expf(-x.y)); }
-        op[i] = __floats2bfloat162_rn(w * a0, w * a1);
+        if (pre && e < E) op[i] = __floats2bfloat162_rn(act_f(act, w * x.x), act_f(act, w * x.y));
+        else op[i] = __floats2bfloat162_rn(w * act_f(act, x.x), w * act_f(act, x.y));
       }
     }
     *reinterpret_cast<uint4*>(out + r * out_stride + c) = o;
@@ -300,9 +292,9 @@ __global__ void moe_plain_act_vec_kernel(const bf16* u, long long u_stride, cons
 
 FMX_EXPORT int fmx_moe_plain_act(const void* u, long long u_stride, const float* weights, const float* shared_gate,
                                  long long sg_stride, void* out, long long out_stride, int rows, int E, int ff, int F, int act,
-                                 int dtype, cudaStream_t stream) {
+                                 int pre, int dtype, cudaStream_t stream) {
   if (rows == 0 || F == 0) return 0;
-  if (rows < 0 || E < 0 || ff <= 0 || F < E * ff || u_stride < F || out_stride < F || act < 0 || act > 2)
+  if (rows < 0 || E < 0 || ff <= 0 || F < E * ff || u_stride < F || out_stride < F || act < 0 || act >= FMX_ACTS)
     return fmx_fail("fmx_moe_plain_act: bad sizes rows=%d E=%d ff=%d F=%d act=%d", rows, E, ff, F, act);
   const bool vec = dtype == FMX_BF16 && F % 8 == 0 && ff % 8 == 0 && (E * ff) % 8 == 0 && u_stride % 8 == 0 && out_stride % 8 == 0 &&
                    ((uintptr_t)u & 15) == 0 && ((uintptr_t)out & 15) == 0;
@@ -311,13 +303,13 @@ FMX_EXPORT int fmx_moe_plain_act(const void* u, long long u_stride, const float*
   const int grid = (int)((n + block - 1) / block < cap ? (n + block - 1) / block : cap);
   if (vec)
     fmx_launch(moe_plain_act_vec_kernel, dim3(grid), dim3(block), 0, stream, (const bf16*)u, u_stride, weights, shared_gate, sg_stride,
-               (bf16*)out, out_stride, (long long)rows, E, ff, F, act);
+               (bf16*)out, out_stride, (long long)rows, E, ff, F, act, pre);
   else if (dtype == FMX_F32)
     fmx_launch(moe_plain_act_kernel<float>, dim3(grid), dim3(block), 0, stream, (const float*)u, u_stride, weights, shared_gate,
-               sg_stride, (float*)out, out_stride, (long long)rows, E, ff, F, act);
+               sg_stride, (float*)out, out_stride, (long long)rows, E, ff, F, act, pre);
   else if (dtype == FMX_BF16)
     fmx_launch(moe_plain_act_kernel<bf16>, dim3(grid), dim3(block), 0, stream, (const bf16*)u, u_stride, weights, shared_gate,
-               sg_stride, (bf16*)out, out_stride, (long long)rows, E, ff, F, act);
+               sg_stride, (bf16*)out, out_stride, (long long)rows, E, ff, F, act, pre);
   else
     return fmx_fail("fmx_moe_plain_act: unknown dtype %d", dtype);
   FMX_LAUNCH_CHECK();

@@ -22,7 +22,8 @@ qk_prepare_kernel(const TI* qkv, long long row_stride, const int* positions, con
                   const long long* slot_mapping, float* q_out, T* kv, int nh, int nkv, int hd, int vd, int rot,
                   int interleaved, float norm_eps, int page_size, long long num_pages, int* status,
                   const float* __restrict__ bias, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
-                  int norm_first, float amplitude, float v_scale) {
+                  int norm_first, float amplitude, float v_scale, const TI* v_first, long long v_first_stride,
+                  const float* __restrict__ v_share) {
   extern __shared__ float smem[];               // [rot/2] sines, [rot/2] cosines, then a head per warp
   pdl_wait();
   pdl_trigger();
@@ -118,9 +119,12 @@ qk_prepare_kernel(const TI* qkv, long long row_stride, const int* positions, con
   const TI* vsrc = row + (long long)(nh + nkv) * hd;
   const float* vbias = bias != nullptr ? bias + (long long)(nh + nkv) * hd : nullptr;
   T* vdst = kv + page * page_elems + (long long)nkv * page_size * hd;
+  const float share = v_share != nullptr ? v_share[0] : 0.f;
   for (int it = threadIdx.x; it < nkv * vd; it += blockDim.x) {
     const int g = it / vd, e = it - g * vd;
-    vdst[((long long)g * page_size + off) * vd + e] = from_f<T>((to_f(vsrc[it]) + (vbias != nullptr ? vbias[it] : 0.f)) * v_scale);
+    float v = (to_f(vsrc[it]) + (vbias != nullptr ? vbias[it] : 0.f)) * v_scale;
+    if (v_first != nullptr) v = (1.0f - share) * v + share * to_f(v_first[(long long)t * v_first_stride + it]);
+    vdst[((long long)g * page_size + off) * vd + e] = from_f<T>(v);
   }
 }
 
@@ -224,13 +228,17 @@ qk_prepare_whole_kernel(const TI* qkv, long long row_stride, const int* position
 // nothing is stored (a layer that reads another's cache then passes nkv = 0 as well).  in_dtype: the
 // type of qkv; dtype: the cache's.  bias (the whole row's, 32-bit), q_weight, k_weight may be null.  amplitude: what cosines
 // and sines are multiplied by (1: a plain rotation); v_scale: what the values are multiplied by, in 32-bit, on their way
-// into the cache.
-FMX_EXPORT int fmx_qk_prepare_ex(const void* qkv, long long row_stride, const int* positions, const float* inv_freq,
+// into the cache.  v_first (of the type of qkv, rows of v_first_stride; may be null) and v_share: the values become (1 - s) v + s v_first
+// with s = *v_share, in 32-bit.
+FMX_EXPORT int fmx_qk_prepare_mix(const void* qkv, long long row_stride, const int* positions, const float* inv_freq,
                                  const long long* slot_mapping, float* q_out, void* kv, int T, int nh, int nkv, int hd,
                                  int vd, int rot, int interleaved, float norm_eps, int page_size, long long num_pages,
                                  int in_dtype, int dtype, const float* bias, const float* q_weight, const float* k_weight,
-                                 int norm_first, float amplitude, float v_scale, int* status, cudaStream_t stream) {
+                                 int norm_first, float amplitude, float v_scale, const void* v_first, long long v_first_stride,
+                                  const float* v_share, int* status, cudaStream_t stream) {
   if (T == 0) return 0;
+  if ((v_first == nullptr) != (v_share == nullptr) || (v_first != nullptr && v_first_stride < (long long)nkv * vd))
+    return fmx_fail("fmx_qk_prepare: values to mix in come with their share and in rows of all heads");
   if (T < 0 || nh < 0 || nkv < 0 || hd <= 0 || vd <= 0 || hd > 256 || rot < 0 || rot > hd || (rot & 1) || page_size <= 0)
     return fmx_fail("fmx_qk_prepare: bad sizes T=%d nh=%d nkv=%d hd=%d vd=%d rot=%d", T, nh, nkv, hd, vd, rot);
   if (rot > 0 && inv_freq == nullptr) return fmx_fail("fmx_qk_prepare: rot=%d needs a frequency table", rot);
@@ -242,7 +250,7 @@ FMX_EXPORT int fmx_qk_prepare_ex(const void* qkv, long long row_stride, const in
 #define FMX_QKP(TI, TKV)                                                                                                  \
   fmx_launch(qk_prepare_kernel<TI, TKV>, dim3(T, head_blocks), dim3(QKP_WARPS * 32), smem, stream, (const TI*)qkv, row_stride, positions, \
              inv_freq, slot_mapping, q_out, (TKV*)kv, nh, nkv, hd, vd, rot, interleaved, norm_eps, page_size, num_pages,  \
-             status, bias, q_weight, k_weight, norm_first, amplitude, v_scale)
+             status, bias, q_weight, k_weight, norm_first, amplitude, v_scale, (const TI*)v_first, v_first_stride, v_share)
   if (in_dtype == FMX_F32 && dtype == FMX_F32)
     FMX_QKP(float, float);
   else if (in_dtype == FMX_BF16 && dtype == FMX_BF16)
@@ -254,6 +262,16 @@ FMX_EXPORT int fmx_qk_prepare_ex(const void* qkv, long long row_stride, const in
 #undef FMX_QKP
   FMX_LAUNCH_CHECK();
   return 0;
+}
+
+FMX_EXPORT int fmx_qk_prepare_ex(const void* qkv, long long row_stride, const int* positions, const float* inv_freq,
+                                 const long long* slot_mapping, float* q_out, void* kv, int T, int nh, int nkv, int hd,
+                                 int vd, int rot, int interleaved, float norm_eps, int page_size, long long num_pages,
+                                 int in_dtype, int dtype, const float* bias, const float* q_weight, const float* k_weight,
+                                 int norm_first, float amplitude, float v_scale, int* status, cudaStream_t stream) {
+  return fmx_qk_prepare_mix(qkv, row_stride, positions, inv_freq, slot_mapping, q_out, kv, T, nh, nkv, hd, vd, rot, interleaved,
+                            norm_eps, page_size, num_pages, in_dtype, dtype, bias, q_weight, k_weight, norm_first, amplitude,
+                            v_scale, nullptr, 0, nullptr, status, stream);
 }
 
 FMX_EXPORT int fmx_qk_prepare(const void* qkv, long long row_stride, const int* positions, const float* inv_freq,

@@ -27,6 +27,7 @@
 // something that never comes, with no copy in flight, and the expiry path runs.  Only the test
 // library `tc_expiry` is built that way; the product library never is.
 #include <cuda.h>
+#include "activations.cuh"
 #include "common.cuh"
 #include "tcgen05.cuh"
 
@@ -37,8 +38,9 @@ constexpr int THREADS = 192;
 
 // RELU2: max(x, 0)^2.  EXPERT: a routed expert's gated activation, w g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit),
 // u' = clamp(u, -limit, limit) and w the row's weight (limit < 0: w silu(g) u), over gate/up blocks like SILU_MUL.  F32: the product as 32-bit floats.
-// GELU_MUL: SILU_MUL with the tanh form of gelu on the gate.
-enum Epilogue { EPI_PLAIN = 0, EPI_SILU_MUL = 1, EPI_RESIDUAL = 2, EPI_RELU2 = 3, EPI_EXPERT = 4, EPI_F32 = 5, EPI_GELU_MUL = 6 };
+// GELU_MUL: SILU_MUL with the tanh form of gelu on the gate.  ACT: an expert without a gate: w act(x), or act(w x) (`pre`), w the row's
+// weight, and times sigmoid of a gate per row where one is given.
+enum Epilogue { EPI_PLAIN = 0, EPI_SILU_MUL = 1, EPI_RESIDUAL = 2, EPI_RELU2 = 3, EPI_EXPERT = 4, EPI_F32 = 5, EPI_GELU_MUL = 6, EPI_ACT = 7 };
 
 // A grouped product: the rows of A are (token, expert) pairs sorted expert by expert, each expert's rows starting on a
 // multiple of 128, and tile row m multiplies with the matrix of expert tile_expert[m], which lies expert_rows rows further
@@ -51,6 +53,9 @@ struct Grouped {
   const float* row_weight;
   int expert_rows;
   float limit;
+  int act, pre;
+  const float* row_gate;
+  long long row_gate_stride;
 };
 
 template <int BN> struct Cfg {
@@ -217,7 +222,12 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
       const int out_n0 = n_tile * OUT_COLS;
       const int n_out = GATED ? N / 2 : N;
       const bool row_in_use = row < M && (gr.row_token == nullptr || gr.row_token[row] >= 0);
-      const float row_w = (EPI == EPI_EXPERT && row_in_use) ? (gr.row_weight != nullptr ? gr.row_weight[row] : 1.0f) : 0.f;
+      float row_w = ((EPI == EPI_EXPERT || EPI == EPI_ACT) && row_in_use) ? (gr.row_weight != nullptr ? gr.row_weight[row] : 1.0f) : 0.f;
+      float in_w = 1.0f;                           // ACT: what multiplies the product in front of its activation, row_w what does behind
+      if (EPI == EPI_ACT) {
+        if (gr.pre) { in_w = row_w; row_w = 1.0f; }
+        if (gr.row_gate != nullptr && row_in_use) row_w *= sigmoid_f(gr.row_gate[(long long)row * gr.row_gate_stride]);
+      }
 #pragma unroll 1
       for (int c = 0; c < OUT_COLS; c += 16) {
         uint32_t v[16], u[16];
@@ -239,11 +249,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
               if (gr.limit < 0.f) {                  // silu(g) u, without clamps
                 f[i] = row_w * silu(f[i]) * __uint_as_float(u[i]);
               } else {
-                const float g = fminf(f[i], gr.limit);
-                const float w = fminf(fmaxf(__uint_as_float(u[i]), -gr.limit), gr.limit);
-                f[i] = row_w * (g / (1.0f + expf(-1.702f * g))) * (w + 1.0f);
+                f[i] = row_w * clamped_gate(f[i], __uint_as_float(u[i]), gr.limit);
               }
             }
+            if (EPI == EPI_ACT) f[i] = row_w * act_f(gr.act, in_w * f[i]);
             if (EPI == EPI_RELU2) {
               // as the unfused path rounds: the product to bfloat16 first, then the square of its positive part
               const float p = fmaxf(__bfloat162float(__float2bfloat16_rn(f[i])), 0.f);
@@ -330,7 +339,7 @@ FMX_EXPORT int fmx_expert_tcgen05(const void* A, long long lda, const void* W, l
   if (K % 8 || lda % 8 || ldw % 8 || ((uintptr_t)A & 15) || ((uintptr_t)W & 15))
     return fmx_fail("fmx_expert_tcgen05: rows must start on 16-byte boundaries (K=%d lda=%lld ldw=%lld)", K, lda, ldw);
   if (sms <= 0) sms = fmx_num_sms();
-  const Grouped gr{nullptr, nullptr, nullptr, nullptr, 0, limit};
+  const Grouped gr{nullptr, nullptr, nullptr, nullptr, 0, limit, 0, 0, nullptr, 0};
   return run<256, EPI_EXPERT>(A, lda, W, ldw, C, ldc, nullptr, 0, M, N, K, sms, status, stream, gr, 0);
 }
 
@@ -351,10 +360,40 @@ FMX_EXPORT int fmx_grouped_tcgen05(const void* A, long long lda, const void* W, 
   if (used_rows == nullptr || tile_expert == nullptr || row_token == nullptr || (gated && row_weight == nullptr))
     return fmx_fail("fmx_grouped_tcgen05: the sorted pairs' arrays are missing");
   if (sms <= 0) sms = fmx_num_sms();
-  const Grouped gr{used_rows, tile_expert, row_token, row_weight, N, limit};
+  const Grouped gr{used_rows, tile_expert, row_token, row_weight, N, limit, 0, 0, nullptr, 0};
   if (gated)
     return run<256, EPI_EXPERT>(A, lda, W, ldw, C, ldc, nullptr, 0, max_rows, N, K, sms, status, stream, gr, (long long)experts * N);
   return run<256, EPI_F32>(A, lda, W, ldw, C, ldc, nullptr, 0, max_rows, N, K, sms, status, stream, gr, (long long)experts * N);
+}
+
+// The grouped product of experts without a gate: as fmx_grouped_tcgen05, an expert's N = ff rows, C bfloat16 [max_rows, ff] =
+// w act(x W^T), or act(w x W^T) with pre.
+FMX_EXPORT int fmx_grouped_act_tcgen05(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc, int max_rows,
+                                       int N, int K, int experts, const int* used_rows, const int* tile_expert, const int* row_token,
+                                       const float* row_weight, int act, int pre, int sms, int* status, cudaStream_t stream) {
+  if (max_rows == 0 || N == 0) return 0;
+  if (max_rows < 0 || max_rows % BM || N <= 0 || K <= 0 || experts <= 0 || act < 0 || act >= FMX_ACTS)
+    return fmx_fail("fmx_grouped_act_tcgen05: bad sizes rows=%d N=%d K=%d experts=%d act=%d", max_rows, N, K, experts, act);
+  if (K % 8 || lda % 8 || ldw % 8 || ((uintptr_t)A & 15) || ((uintptr_t)W & 15))
+    return fmx_fail("fmx_grouped_act_tcgen05: rows must start on 16-byte boundaries (K=%d lda=%lld ldw=%lld)", K, lda, ldw);
+  if (used_rows == nullptr || tile_expert == nullptr || row_token == nullptr || row_weight == nullptr)
+    return fmx_fail("fmx_grouped_act_tcgen05: the sorted pairs' arrays are missing");
+  if (sms <= 0) sms = fmx_num_sms();
+  const Grouped gr{used_rows, tile_expert, row_token, row_weight, N, 0.f, act, pre, nullptr, 0};
+  return run<256, EPI_ACT>(A, lda, W, ldw, C, ldc, nullptr, 0, max_rows, N, K, sms, status, stream, gr, (long long)experts * N);
+}
+
+// One expert without a gate for every row: C bfloat16 [M, N] = act(A W^T), times sigmoid(row_gate[row * row_gate_stride]) where given.
+FMX_EXPORT int fmx_act_tcgen05(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc, int M, int N,
+                               int K, int act, const float* row_gate, long long row_gate_stride, int sms, int* status,
+                               cudaStream_t stream) {
+  if (M == 0 || N == 0) return 0;
+  if (M < 0 || N <= 0 || K <= 0 || act < 0 || act >= FMX_ACTS) return fmx_fail("fmx_act_tcgen05: bad sizes M=%d N=%d K=%d act=%d", M, N, K, act);
+  if (K % 8 || lda % 8 || ldw % 8 || ((uintptr_t)A & 15) || ((uintptr_t)W & 15))
+    return fmx_fail("fmx_act_tcgen05: rows must start on 16-byte boundaries (K=%d lda=%lld ldw=%lld)", K, lda, ldw);
+  if (sms <= 0) sms = fmx_num_sms();
+  const Grouped gr{nullptr, nullptr, nullptr, nullptr, 0, 0.f, act, 0, row_gate, row_gate_stride};
+  return run<256, EPI_ACT>(A, lda, W, ldw, C, ldc, nullptr, 0, M, N, K, sms, status, stream, gr, 0);
 }
 
 // The tile width (of 128, 192, 256) whose tiles fill the SMs' rounds best; wider wins ties.

@@ -24,7 +24,7 @@ from .batch import StepEntry
 from .loading import load_model
 from .step import StepFunction
 
-MAX_LIVE = 8          # request slots; traces keep up to four live, a step may name one more while another ends
+MAX_LIVE = 4          # request slots: the most requests that a trace keeps live at any time
 
 
 def pool_pages(max_tokens: int, page_size: int) -> int:
@@ -82,9 +82,10 @@ def main(argv=None) -> int:
     ap.add_argument("--max-tokens", type=int, required=True,
                     help="most tokens live requests hold at any time (each rounded up to 64)")
     ap.add_argument("--page-size", type=int, default=16, help="tokens per cache page")
+    ap.add_argument("--max-live", type=int, default=MAX_LIVE, help="most requests that are live at any time")
     args = ap.parse_args(argv)
     os.makedirs(args.out, exist_ok=True)
-    rp = Replayer(args.model, args.dtype, args.max_tokens, args.page_size)
+    rp = Replayer(args.model, args.dtype, args.max_tokens, args.page_size, max_live=args.max_live)
     for line in sys.stdin:
         line = line.strip()
         if not line:

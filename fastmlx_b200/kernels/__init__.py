@@ -75,14 +75,15 @@ def embedding(ids: torch.Tensor, table: torch.Tensor, status, out_dtype=None) ->
     return gather_rows(table, ids, status, BAD_TOKEN)
 
 
-def add_rmsnorm(x, residual, weight: torch.Tensor, eps: float, stream_dtype=None, out_dtype=None):
+def add_rmsnorm(x, residual, weight: torch.Tensor, eps: float, stream_dtype=None, out_dtype=None, weight2=None):
     """-> (norm(residual + x) * weight, residual + x); the sum replaces `residual` in place.
     Without a residual, x is the stream's first value: it is returned as the stream, as it is or,
     when `stream_dtype` is float32 beside bfloat16 activations, as a 32-bit copy that the later
     sums then never round.  x may be None when there is a residual (the stream itself is
-    normalised; `out_dtype` then names the activations' type)."""
-    _need_cuda(x, residual, weight)
-    assert weight.dtype == torch.float32
+    normalised; `out_dtype` then names the activations' type).  `weight2`: a second weight of the same normed sum, in the
+    same pass: -> (norm * weight, norm * weight2, sum)."""
+    _need_cuda(x, residual, weight, weight2)
+    assert weight.dtype == torch.float32 and (weight2 is None or weight2.dtype == torch.float32)
     ref = x if x is not None else residual
     assert ref is not None and ref.dim() == 2 and ref.is_contiguous()
     act = x.dtype if x is not None else (out_dtype or residual.dtype)
@@ -92,6 +93,12 @@ def add_rmsnorm(x, residual, weight: torch.Tensor, eps: float, stream_dtype=None
         init = 1
     assert residual is None or (residual.shape == ref.shape and residual.is_contiguous())
     out = torch.empty(ref.shape, dtype=act, device=ref.device)
+    if weight2 is not None:
+        out2 = torch.empty(ref.shape, dtype=act, device=ref.device)
+        call("common", "fmx_add_rmsnorm_pair", _ptr(x), _ptr(residual), weight.data_ptr(), out.data_ptr(), weight2.data_ptr(),
+             out2.data_ptr(), ref.shape[0], ref.shape[1], float(eps), _dt(out), _dt(residual) if residual is not None else _dt(out),
+             init, _stream())
+        return out, out2, (residual if residual is not None else x)
     call("common", "fmx_add_rmsnorm", _ptr(x), _ptr(residual), weight.data_ptr(), out.data_ptr(), ref.shape[0], ref.shape[1],
          float(eps), _dt(out), _dt(residual) if residual is not None else _dt(out), init, _stream())
     return out, (residual if residual is not None else x)
@@ -175,6 +182,7 @@ TC_MIN_ROWS = 128
 GATE_UP_BLOCK = 128              # gate/up rows of a fused weight alternate in blocks of this many
 EPI_PLAIN, EPI_SILU_MUL, EPI_RESIDUAL, EPI_RELU2 = 0, 1, 2, 3
 EPI_GELU_MUL = 6                 # the gated epilogue with the tanh form of gelu on the gate
+GEMV_GATE_CLAMPED = 2 << 20      # likewise: the clamped form
 GEMV_GATE_GELU = 1 << 20         # added to a gated whole-K product's block size: gelu on the gate instead of silu
 
 
@@ -191,25 +199,32 @@ def can_gemv(x, w) -> bool:
 
 
 def gemv(x, w, bias=None, out_dtype=torch.bfloat16, residual=None, block: int = 0, out=None, wide=None, warps=None,
-         act: str | None = None):
+         act: str | None = None, limit: float = 0.0, row_gate=None):
     """x[M <= 16, K] @ w[N, K]^T, one block per `wide` (8, 16, 32) output features and the whole of K:
     nothing is summed across blocks.  residual [M, n_out] is added to the product (out may be
     the residual itself).  block > 0: w's rows alternate in blocks of `block` gate rows and
-    their up rows, and the result is silu(gate) * up, [M, N/2] (with act="gelu_tanh": gelu(gate) * up).  act (relu2,
-    gelu_tanh, silu) without blocks: the activation of the product (and bias), in the same pass; `out` may be a slice
-    of a wider buffer."""
+    their up rows, and the result is silu(gate) * up, [M, N/2] (with act="gelu_tanh": gelu(gate) * up; "clamped": g' sigmoid(1.702 g')
+    (u' + 1), clamped by `limit`).  act (relu2, gelu_tanh, silu, gelu) without blocks: the activation of the product (and
+    bias), in the same pass, multiplied by sigmoid(row_gate[m, 0]) (32-bit) where one is given; `out` may be a slice of a wider
+    buffer."""
     M, K = x.shape
     N = w.shape[0]
     n_out = N // 2 if block else N
     if act is not None and block:
-        assert block > 0 and act in ("silu", "gelu_tanh") and out_dtype == torch.bfloat16
-        block = int(block) + (GEMV_GATE_GELU if act == "gelu_tanh" else 0)
+        assert block > 0 and act in ("silu", "gelu_tanh", "clamped") and out_dtype == torch.bfloat16
+        block = int(block) + {"silu": 0, "gelu_tanh": GEMV_GATE_GELU, "clamped": GEMV_GATE_CLAMPED}[act]
     elif act is not None:
         assert out_dtype == torch.bfloat16
         block = -1 - ACTIVATIONS[act]
     if out is None:
         out = torch.empty((M, n_out), dtype=out_dtype, device=x.device)
     # wide / warps left open: the library plans them (`fmx_gemv_plan_width`, `fmx_gemv_plan_warps`)
+    if limit or row_gate is not None or act == "clamped":
+        assert row_gate is None or (row_gate.dtype == torch.float32 and row_gate.shape[0] == M)
+        call("bf16", "fmx_gemv_ex", x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), _ptr(bias), _ptr(residual),
+             residual.stride(0) if residual is not None else 0, out.data_ptr(), out.stride(0), M, N, K, _dt(out), int(block),
+             int(wide or 0), int(warps or 0), float(limit), _ptr(row_gate), row_gate.stride(0) if row_gate is not None else 0, _stream())
+        return out
     call("bf16", "fmx_gemv", x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), _ptr(bias), _ptr(residual),
          residual.stride(0) if residual is not None else 0, out.data_ptr(), out.stride(0), M, N, K, _dt(out), int(block),
          int(wide or 0), int(warps or 0), _stream())
@@ -340,7 +355,7 @@ def paged_attention_simple(qkv, kv, ctx, group, nh, nkv, hd, scale, window) -> t
 
 def qk_prepare(qkv, positions, inv_freq, rotary_dim, traditional, norm_eps, slot_mapping, kv, nh, nkv, hd, vd,
                status, bias=None, q_weight=None, k_weight=None, norm_first: bool = False, whole: bool = False,
-               values_from_keys: bool = False, amplitude: float = 1.0, v_scale: float = 1.0) -> torch.Tensor:
+               values_from_keys: bool = False, amplitude: float = 1.0, v_scale: float = 1.0, v_first=None, v_share=None) -> torch.Tensor:
     """Queries and keys of qkv[T, nh*hd + nkv*hd + nkv*vd] made ready for attention: rotated over their
     first `rotary_dim` dimensions, then (norm_eps not None) each head divided by its root mean square;
     keys and values are stored at slot_mapping in pages that hold [nkv, page, hd] keys and then
@@ -350,7 +365,8 @@ def qk_prepare(qkv, positions, inv_freq, rotary_dim, traditional, norm_eps, slot
     before the rotation instead of after it.  `whole` (with `norm_first`): q and k are each divided by the root mean
     square of their whole projection, all heads at once, and the weights are that wide ([nh*hd], [nkv*hd]);
     `values_from_keys`: qkv holds q | k only, and a token's values are its keys as projected (vd = hd).  `amplitude`
-    multiplies the rotation's cosines and sines, `v_scale` the values on their way into the cache, both in 32-bit."""
+    multiplies the rotation's cosines and sines, `v_scale` the values on their way into the cache, both in 32-bit.
+    `v_first` ([T, nkv*vd] of qkv's type, rows may be a slice) and `v_share` (32-bit [1]): the values become (1 - s) v + s v_first."""
     _need_cuda(qkv, positions, inv_freq, slot_mapping, kv, bias, q_weight, k_weight)
     assert qkv.dim() == 2 and qkv.stride(1) == 1 and positions.dtype == torch.int32
     T = qkv.shape[0]
@@ -363,6 +379,15 @@ def qk_prepare(qkv, positions, inv_freq, rotary_dim, traditional, norm_eps, slot
         num_pages, page_size = 0, 1
     for v in (bias, q_weight, k_weight):
         assert v is None or (v.dtype == torch.float32 and v.is_contiguous())
+    if v_first is not None:
+        assert not whole and not values_from_keys and v_first.dtype == qkv.dtype and v_first.shape == (T, nkv * vd)
+        assert v_first.stride(1) == 1 and v_share.dtype == torch.float32 and v_share.numel() == 1
+        call("common", "fmx_qk_prepare_mix", qkv.data_ptr(), qkv.stride(0), positions.data_ptr(), _ptr(inv_freq),
+             _ptr(slot_mapping), q.data_ptr(), _ptr(kv), T, nh, nkv if kv is not None else 0, hd, vd, int(rotary_dim),
+             int(bool(traditional)), -1.0 if norm_eps is None else float(norm_eps), page_size, num_pages, _dt(qkv),
+             _dt(kv) if kv is not None else _dt(qkv), _ptr(bias), _ptr(q_weight), _ptr(k_weight), int(bool(norm_first)),
+             float(amplitude), float(v_scale), v_first.data_ptr(), v_first.stride(0), v_share.data_ptr(), _ptr(status), _stream())
+        return q
     if whole or values_from_keys:
         assert norm_first or norm_eps is None, "the norm over the whole projection comes before the rotation"
         call("common", "fmx_qk_prepare_whole", qkv.data_ptr(), qkv.stride(0), positions.data_ptr(), _ptr(inv_freq),
@@ -829,16 +854,65 @@ def channel_scan(qkv, g, beta, ctx, state, H, G, D, Dv, lanes: int = 0, cpt: int
     return out
 
 
-def head_norm_gate(o, gate, weight, eps, H, Dv, out_dtype, act: str = "sigmoid", out=None) -> torch.Tensor:
-    """o[T, H*Dv] (32-bit) per head divided by its root mean square, times weight[Dv], times sigmoid(gate) (act="silu":
-    silu(gate)); gate (of its own type) and out may be slices of wider buffers."""
+def head_norm_gate(o, gate, weight, eps, H, Dv, out_dtype, act: str = "sigmoid", out=None, divisor=None) -> torch.Tensor:
+    """o[T, H*Dv] (32-bit) per head divided by its root mean square, times weight (Dv values for all heads, or H*Dv), times
+    sigmoid(gate) (act="silu": silu(gate)); gate (of its own type) and out may be slices of wider buffers.  `divisor` = (nq [T, H],
+    gates [T, H, 4]), 32-bit: o is first divided by max(|nq|, gates[.., 2]) + 1e-6."""
     T = o.shape[0]
     if out is None:
         out = torch.empty((T, H * Dv), dtype=out_dtype, device=o.device)
     assert act in ("sigmoid", "silu") and o.is_contiguous() and gate.stride(1) == 1 and out.stride(1) == 1
     assert gate.shape == (T, H * Dv) and out.shape == (T, H * Dv) and weight.dtype == torch.float32
-    call("chan", "fmx_head_norm_gate", o.data_ptr(), gate.data_ptr(), gate.stride(0), _dt(gate), weight.data_ptr(), out.data_ptr(),
-         out.stride(0), _dt(out), T, H, Dv, float(eps), int(act == "silu"), _stream())
+    assert weight.numel() in (Dv, H * Dv) and weight.is_contiguous()
+    nq, gates = divisor if divisor is not None else (None, None)
+    assert divisor is None or (nq.is_contiguous() and gates.is_contiguous() and nq.dtype == gates.dtype == torch.float32)
+    call("common", "fmx_head_norm_gate", o.data_ptr(), gate.data_ptr(), gate.stride(0), _dt(gate), weight.data_ptr(), out.data_ptr(),
+         out.stride(0), _dt(out), T, H, Dv, float(eps), int(act == "silu"), Dv if weight.numel() == H * Dv else 0, _ptr(nq), _ptr(gates),
+         _stream())
+    return out
+
+
+# ----------------------------------------------------------------------------- the matrix memory with exponential gates
+def mlstm_gates(z, bias, cap: float, ctx, state, m_off: int, H: int) -> torch.Tensor:
+    """The capped log gates of z[T, input gates (H) | forget gates (H)] (32-bit, rows may be a slice) with bias[2 H], run over every
+    request's tokens: -> [T, H, 4] in 32-bit, (exp(f + m - m'), exp(i - m'), exp(-m'), 0) with m' = max(f + m, i) the running
+    maximum, which is read from and left in the requests' slots at m_off."""
+    _need_cuda(z, bias)
+    assert z.dtype == torch.float32 and z.stride(1) == 1 and z.shape[1] == 2 * H and bias.dtype == torch.float32 and bias.numel() == 2 * H
+    gates = torch.empty((z.shape[0], H, 4), dtype=torch.float32, device=z.device)
+    call("mlstm", "fmx_mlstm_gates", z.data_ptr(), z.stride(0), bias.data_ptr(), float(cap), ctx.row_start.data_ptr(),
+         ctx.row_slot.data_ptr(), state.data_ptr(), state.stride(0), int(m_off), gates.data_ptr(), ctx.R, H, state.shape[0], _stream())
+    return gates
+
+
+def mlstm_scan(proj, gates, ctx, state, H: int, D: int, Dv: int, lanes: int = 0, cpt: int = 0):
+    """The matrix memory over every request's tokens of the step, in order, from and into the requests' slots (S^T per head with n as
+    its last row, [H, Dv + 1, D], at the head of a slot): S <- keep S + put k v^T, n <- keep n + put k.  proj[T, q (H*D) | k (H*D) |
+    v (H*Dv) ...], gates as `mlstm_gates` left them.  -> (S^T q [T, H*Dv], n . q [T, H]) in 32-bit, q times D^-1/2, not divided
+    yet.  `lanes` (8, 16, 32) and `cpt` (1, 2, 4; 0: the library's choice): lanes that share a column, and columns that they hold."""
+    T = proj.shape[0]
+    assert proj.stride(1) == 1 and gates.is_contiguous() and gates.shape == (T, H, 4)
+    out = torch.empty((T, H * Dv), dtype=torch.float32, device=proj.device)
+    nq = torch.empty((T, H), dtype=torch.float32, device=proj.device)
+    call("mlstm", "fmx_mlstm_scan", proj.data_ptr(), proj.stride(0), gates.data_ptr(), ctx.row_start.data_ptr(), ctx.row_slot.data_ptr(),
+         state.data_ptr(), state.stride(0), out.data_ptr(), nq.data_ptr(), ctx.R, H, D, Dv, state.shape[0], _dt(proj), int(lanes), int(cpt),
+         _stream())
+    return out, nq
+
+
+def mlstm_step(proj, z, bias, cap: float, ctx, state, H: int, D: int, Dv: int, weight, eps: float, out_dtype, out=None) -> torch.Tensor:
+    """Rows of one token each, in one kernel: gates, recurrence, division, each head over its root mean square, times weight[H*Dv],
+    times sigmoid of the output gate.  proj[T, q | k | v | output gate ...]; z, bias, state as above (m behind the heads' states).
+    -> [T, H*Dv] in `out_dtype`; `out` may be a slice of a wider buffer."""
+    _need_cuda(proj, z)
+    T = proj.shape[0]
+    if out is None:
+        out = torch.empty((T, H * Dv), dtype=out_dtype, device=proj.device)
+    assert proj.stride(1) == 1 and z.dtype == torch.float32 and z.stride(1) == 1 and out.stride(1) == 1 and out.shape == (T, H * Dv)
+    assert weight.dtype == torch.float32 and weight.numel() == H * Dv and bias.dtype == torch.float32
+    call("mlstm", "fmx_mlstm_step", proj.data_ptr(), proj.stride(0), _dt(proj), z.data_ptr(), z.stride(0), bias.data_ptr(), float(cap),
+         ctx.row_start.data_ptr(), ctx.row_slot.data_ptr(), state.data_ptr(), state.stride(0), H * (Dv + 1) * D, weight.data_ptr(), float(eps),
+         out.data_ptr(), out.stride(0), _dt(out), ctx.R, H, D, Dv, state.shape[0], _stream())
     return out
 
 
@@ -930,13 +1004,15 @@ def sigmoid_gate(o, gate, group: int = 1):
 
 
 def moe_route(logits, top: int, groups: int = 1, keep: int = 1, want_chosen: bool = False, experts: int | None = None,
-              correction=None, scale: float = 1.0, logit_bias=None, renorm: bool = False):
+              correction=None, scale: float = 1.0, logit_bias=None, renorm: bool = False, scores: str = "softmax"):
     """Router logits [T, E] (32-bit) -> weights [T, E] (32-bit): the softmax score where an expert is among the token's
     `top` best of the `keep` best groups (of `groups` groups of neighbours, each scored by its best member), else zero;
     not renormalised.  With `want_chosen` also the chosen indices, int32 [T, top].  `experts`: the row's first that many
     columns are the experts' logits (a row may hold other columns behind them).  `correction` (32-bit [E]): added to the
     scores for the choice only; `scale` multiplies the chosen experts' scores.  `logit_bias` (32-bit [E]): added to the
-    logits; `renorm`: the weights are the softmax over the chosen logits alone."""
+    logits; `renorm`: the weights are the softmax over the chosen logits alone; `scores="sigmoid"`: a score is the sigmoid of its
+    logit alone."""
+    assert scores in ("softmax", "sigmoid")
     _need_cuda(logits, correction, logit_bias)
     assert logit_bias is None or (logit_bias.dtype == torch.float32 and logit_bias.is_contiguous())
     assert logits.dim() == 2 and logits.dtype == torch.float32 and logits.stride(1) == 1
@@ -946,14 +1022,16 @@ def moe_route(logits, top: int, groups: int = 1, keep: int = 1, want_chosen: boo
     w = torch.empty((T, E), dtype=torch.float32, device=logits.device)
     chosen = torch.empty((T, top), dtype=torch.int32, device=logits.device) if want_chosen else None
     call("common", "fmx_moe_route_ex", logits.data_ptr(), logits.stride(0), T, E, int(top), int(groups), int(keep),
-         w.data_ptr(), _ptr(chosen), _ptr(correction), float(scale), _ptr(logit_bias), int(bool(renorm)), _stream())
+         w.data_ptr(), _ptr(chosen), _ptr(correction), float(scale), _ptr(logit_bias), int(bool(renorm)),
+         int(scores == "sigmoid"), _stream())
     return (w, chosen) if want_chosen else w
 
 
-def moe_plain_act(u, weights, E: int, ff: int, act: str, shared_gate=None, out=None):
+def moe_plain_act(u, weights, E: int, ff: int, act: str, shared_gate=None, out=None, weigh_input: bool = False):
     """The hidden layers of experts without a gate, side by side: u[T, F], F = E*ff + the shared expert's width;
     -> [T, F]: w * act(u) with w the token's weight for the column's expert, zero where it did not choose it; the shared
-    columns at the end weigh sigmoid(shared_gate[t]) (32-bit, one value per token; rows may be a slice) or 1."""
+    columns at the end weigh sigmoid(shared_gate[t]) (32-bit, one value per token; rows may be a slice) or 1.  `weigh_input`:
+    act(w * u) for the experts' columns."""
     _need_cuda(u, weights, shared_gate)
     assert u.dim() == 2 and u.stride(1) == 1 and weights.dtype == torch.float32 and weights.is_contiguous()
     T, F = u.shape
@@ -962,8 +1040,26 @@ def moe_plain_act(u, weights, E: int, ff: int, act: str, shared_gate=None, out=N
         out = torch.empty((T, F), dtype=u.dtype, device=u.device)
     call("common", "fmx_moe_plain_act", u.data_ptr(), u.stride(0), weights.data_ptr(), _ptr(shared_gate),
          shared_gate.stride(0) if shared_gate is not None else 0, out.data_ptr(), out.stride(0), T, int(E), int(ff), F,
-         ACTIVATIONS[act], _dt(u), _stream())
+         ACTIVATIONS[act], int(bool(weigh_input)), _dt(u), _stream())
     return out
+
+
+def plain_up(x, w, act: str, row_gate=None, out=None, status=None):
+    """An expert without a gate for every token: sigmoid(row_gate[t, 0]) * act(x w^T) (without a gate 1), in one kernel where its
+    size has one (whole-K product up to 16 rows, tcgen05 product from 128 rows that fill the GPU), else the library's product and
+    the activation kernel.  row_gate 32-bit [T, 1]; `out` may be a slice of a wider buffer.  -> [T, N]."""
+    T, N = x.shape[0], w.shape[0]
+    if out is None:
+        out = torch.empty((T, N), dtype=x.dtype, device=x.device)
+    if can_gemv(x, w):
+        return gemv(x, w, act=act, row_gate=row_gate, out=out)
+    if (_bf16_operands(x, w) and T >= TC_MIN_ROWS and out.stride(1) == 1 and tc_fills_the_gpu(T, N, num_sms(x.device))):
+        call("tc", "fmx_act_tcgen05", x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), T, N, x.shape[1],
+             ACTIVATIONS[act], _ptr(row_gate), row_gate.stride(0) if row_gate is not None else 0, num_sms(x.device),
+             _ptr(status if status is not None else _status_word(x.device)), _stream())
+        return out
+    none = torch.empty((T, 0), dtype=torch.float32, device=x.device)
+    return moe_plain_act(linear(x, w, None, x.dtype), none, 0, N, act, shared_gate=row_gate, out=out)
 
 
 def moe_expert_act(gu, weights, E: int, ff: int, limit: float, limit_shared: float = 0.0, out=None, block: int = 0):
@@ -993,12 +1089,14 @@ def can_expert_tc(x, w) -> bool:
             and tc_fills_the_gpu(x.shape[0], w.shape[0], num_sms(x.device)))
 
 
-def expert_gate_up_tc(x, w, limit: float, status=None) -> torch.Tensor:
+def expert_gate_up_tc(x, w, limit: float, status=None, out=None) -> torch.Tensor:
     """g' sigmoid(1.702 g') (u' + 1) of x w^T, g' = min(g, limit), u' = clamp(u, -limit, limit), for w [2 ff, K] in blocks of 128
     gate rows followed by their up rows: product and activation in one tcgen05 kernel.  -> bfloat16 [M, ff]."""
     M, K = x.shape
     N = w.shape[0]
-    out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
+    if out is None:
+        out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
+    assert out.dtype == torch.bfloat16 and out.stride(1) == 1 and out.shape == (M, N // 2)
     call("tc", "fmx_expert_tcgen05", x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, N, K,
          float(limit), num_sms(x.device), _ptr(status if status is not None else _status_word(x.device)), _stream())
     return out
@@ -1061,6 +1159,29 @@ def moe_grouped_gate_up(x, plan, gate_up, E: int, ff: int, limit: float, block: 
         w_up, stride = gate_up.data_ptr() + 2 * E * ff * K, ff * K
     call("bf16", "fmx_moe_grouped_gate_up", x.data_ptr(), x.stride(0), sorted_token.data_ptr(), sorted_w.data_ptr(),
          tile_expert.data_ptr(), gate_up.data_ptr(), w_up, K, stride, y.data_ptr(), tiles, ff, K, float(limit), int(block), T, _stream())
+    return y
+
+
+def moe_grouped_up(x, plan, up, E: int, ff: int, act: str, weigh_input: bool = False, status=None) -> torch.Tensor:
+    """`moe_grouped_gate_up` for experts without a gate: up [E ff, K] bfloat16, expert after expert; row r of the result is
+    w act(x w_up^T) of the row's token under the row's expert, w the pair's weight, or (`weigh_input`) act(w x w_up^T).
+    -> bfloat16 [tiles * MOE_TILE_ROWS, ff] (padding rows are not written)."""
+    sorted_token, sorted_w, _, tile_expert, tiles, used = plan
+    _need_cuda(x, up)
+    T, K = x.shape
+    assert x.dtype == torch.bfloat16 and up.dtype == torch.bfloat16 and up.is_contiguous() and x.stride(1) == 1 and up.shape == (E * ff, K)
+    rows = tiles * MOE_TILE_ROWS
+    y = torch.empty((rows, ff), dtype=torch.bfloat16, device=x.device)
+    if T >= MOE_TC_MIN_TOKENS and ff % 8 == 0:
+        xs = torch.empty((rows, K), dtype=torch.bfloat16, device=x.device)
+        call("bf16", "fmx_moe_gather", x.data_ptr(), x.stride(0), sorted_token.data_ptr(), used.data_ptr(), xs.data_ptr(), rows, K,
+             _stream())
+        call("tc", "fmx_grouped_act_tcgen05", xs.data_ptr(), K, up.data_ptr(), K, y.data_ptr(), ff, rows, ff, K, E, used.data_ptr(),
+             tile_expert.data_ptr(), sorted_token.data_ptr(), sorted_w.data_ptr(), ACTIVATIONS[act], int(bool(weigh_input)),
+             num_sms(x.device), _ptr(status if status is not None else _status_word(x.device)), _stream())
+        return y
+    call("bf16", "fmx_moe_grouped_up", x.data_ptr(), x.stride(0), sorted_token.data_ptr(), sorted_w.data_ptr(), tile_expert.data_ptr(),
+         up.data_ptr(), K, ff * K, y.data_ptr(), tiles, ff, K, ACTIVATIONS[act], int(bool(weigh_input)), T, _stream())
     return y
 
 
@@ -1134,7 +1255,7 @@ def head_linear(x, w, out_dtype, x_head_stride: int | None = None, out=None, out
     return out
 
 
-ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2}
+ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "gelu": 3}
 
 
 def activation(x, kind: str, out=None) -> torch.Tensor:

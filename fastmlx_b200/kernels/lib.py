@@ -62,10 +62,14 @@ _SIGNATURES = {
         "fmx_embed_scaled": [_P, _I, _P, _P, _I, _I, _L, _F, _P, _I, _P],
         "fmx_rmsnorm_pair_mean": [_P, _L, _P, _L, _I, _P, _P, _F, _P, _L, _I, _I, _I, _P],
         "fmx_moe_route_biased": [_P, _L, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P],
-        "fmx_moe_route_ex": [_P, _L, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P, _I, _P],
+        "fmx_moe_route_ex": [_P, _L, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P, _I, _I, _P],
         "fmx_layernorm_step": [_P, _L, _I, _P, _F, _F, _P, _P, _P, _F, _P, _L, _I, _I, _I, _P],
         "fmx_logit_cap": [_P, _L, _I, _I, _F, _F, _P],
-        "fmx_moe_plain_act": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _P],
+        "fmx_moe_plain_act": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P],
+        "fmx_add_rmsnorm_pair": [_P, _P, _P, _P, _P, _P, _I, _I, _F, _I, _I, _I, _P],
+        "fmx_qk_prepare_mix": [_P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _L, _I, _I, _P, _P, _P, _I, _F,
+                               _F, _P, _L, _P, _P, _P],
+        "fmx_head_norm_gate": [_P, _P, _L, _I, _P, _P, _L, _I, _I, _I, _I, _F, _I, _I, _P, _P, _P],
         "fmx_retention_prepare": [_P, _L, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _P],
         "fmx_retention_gate_norm": [_P, _P, _L, _I, _P, _L, _I, _I, _I, _I, _F, _P],
         "fmx_sigmoid_attention": [_P, _L, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _L, _F, _F, _I, _I, _I, _P, _P, _P],
@@ -73,6 +77,8 @@ _SIGNATURES = {
     },
     "bf16": {
         "fmx_gemv": [_P, _L, _P, _L, _P, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P],
+        "fmx_gemv_ex": [_P, _L, _P, _L, _P, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _I, _F, _P, _L, _P],
+        "fmx_moe_grouped_up": [_P, _L, _P, _P, _P, _P, _L, _L, _P, _I, _I, _I, _I, _I, _I, _P],
         "fmx_gemv_argmax": [_P, _L, _P, _L, _P, _P, _P, _I, _I, _I, _P],
         "fmx_moe_sort": [_P, _P, _I, _I, _I, _P, _P, _P, _P, _I, _P, _P],
         "fmx_moe_gather": [_P, _L, _P, _P, _P, _I, _I, _P],
@@ -82,6 +88,8 @@ _SIGNATURES = {
     },
     "tc": {
         "fmx_gemm_tcgen05": [_P, _L, _P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _P, _P],
+        "fmx_grouped_act_tcgen05": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _P, _I, _I, _I, _P, _P],
+        "fmx_act_tcgen05": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _P, _L, _I, _P, _P],
         "fmx_expert_tcgen05": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _F, _I, _P, _P],
         "fmx_grouped_tcgen05": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _P, _F, _I, _I, _P, _P],
     },
@@ -90,7 +98,11 @@ _SIGNATURES = {
                                       _I, _I, _I, _I, _I, _P, _P],
         "fmx_channel_gla_prepare": [_P, _L, _P, _L, _P, _P, _P, _I, _I, _I, _I, _F, _F, _I, _P],
         "fmx_channel_scan": [_P, _P, _P, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
-        "fmx_head_norm_gate": [_P, _P, _L, _I, _P, _P, _L, _I, _I, _I, _I, _F, _I, _P],
+    },
+    "mlstm": {
+        "fmx_mlstm_gates": [_P, _L, _P, _F, _P, _P, _P, _L, _L, _P, _I, _I, _I, _P],
+        "fmx_mlstm_scan": [_P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+        "fmx_mlstm_step": [_P, _L, _I, _P, _L, _P, _F, _P, _P, _P, _L, _L, _P, _F, _P, _L, _I, _I, _I, _I, _I, _I, _P],
     },
     "mixattn": {
         "fmx_mixattn": [_P, _L, _P, _P, _I, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _L, _F, _F, _I, _I, _P, _P, _I, _I, _P, _P],

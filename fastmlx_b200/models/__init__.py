@@ -5,3 +5,4 @@ from . import medirax  # noqa: F401
 from . import sorupel  # noqa: F401
 from . import kafepel  # noqa: F401
 from . import bonerax  # noqa: F401
+from . import gepadra  # noqa: F401

@@ -7,6 +7,7 @@ from .embedding import BigramEmbedding, Embedding, LMHead
 from .gla import GatedLinearAttention
 from .linear import BlockDiagonalLinear, JoinedLinear, Linear
 from .mlp import DenseMLP, SwiGLU
+from .mlstm import MatrixMemoryMixer
 from .model import Model
 from .latent import LatentAttention
 from .loop import LoopInput, LoopPass
@@ -21,4 +22,4 @@ __all__ = ["GQAAttention", "FeedForward", "Mixer", "Norm", "PagedKVSpec", "Part"
            "SwiGLU", "DenseMLP", "JoinedLinear", "ParallelBlock", "GatedDeltaMixer", "Model", "RMSNorm", "NoPositionEncoding", "RotaryEmbedding", "inverse_frequencies", "SandwichBlock", "LatentAttention", "LoopInput", "LoopPass", "RoutedExperts",
            "DynamicTanh", "Pending", "BigramEmbedding", "StateSpaceMixer", "PairMixer", "PlainRoutedExperts",
            "RetentionMixer", "MixerOnly", "FreeDim", "PostNormBlock", "ChannelDeltaMixer", "GatedLinearAttention", "BlockDiagonalLinear",
-           "LayerNorm"]
+           "LayerNorm", "MatrixMemoryMixer"]

@@ -39,7 +39,8 @@ class GQAAttention(Mixer):
     divided by the root mean square of the whole projection, all heads at once, and the weights have the
     projection's width.  `chunk` c > 0 (instead of a window): position i sees j <= i only where i // c == j // c,
     runs counted from position 0 of the request whatever the cut of its prompt; the cache gives earlier runs' pages
-    back.  `sink` s: the softmax's denominator has one more term exp(s) that has no value (s = 0 adds one).
+    back.  `sink` s: the softmax's denominator has one more term exp(s) that has no value (s = 0 adds one); a string
+    names a tensor of one learned s per head instead.
     `gate_per_head`: the gate has one value per head, not one per output element.
 
     And a form without a softmax.  `weights="sigmoid"`: a visible key weighs sigmoid(score + b_h) with one number per
@@ -50,6 +51,10 @@ class GQAAttention(Mixer):
     `value_scale`: the values are multiplied by it, in 32-bit, before they are stored, and with them the heads' outputs
     (`scale_output` sets it; a block that scales its mixers uses that).  A rotation whose cosines and sines have an
     amplitude (`pos.amplitude`) takes this route too.
+
+    `value_mix`: the layer is the "first" of those that mix their values, or a "later" one whose values become (1 - l) v +
+    l v_first, in 32-bit, before they are stored; v_first are the first one's values of the same token in the same
+    step (handed on in the step's scratch), l a scalar tensor `value_mix_name` (the first one has it too and does not use it).
     """
 
     supports_cuda_graph = True
@@ -62,8 +67,9 @@ class GQAAttention(Mixer):
                  weight_suffix: str = ".weight", bias_suffix: str = ".bias", qk_norm_weights=None,
                  qk_norm_first: bool = False, keep_first: int = 0, gate: str | None = None, late_bias: bool = False,
                  out_bias: bool | None = None, values_from_keys: bool = False, qk_norm_whole: bool = False,
-                 chunk: int = 0, sink: float | None = None, gate_per_head: bool = False, weights: str = "softmax",
-                 head_bias: str | None = None, head_mix: str | None = None, value_scale: float = 1.0):
+                 chunk: int = 0, sink: float | str | None = None, gate_per_head: bool = False, weights: str = "softmax",
+                 head_bias: str | None = None, head_mix: str | None = None, value_scale: float = 1.0,
+                 value_mix: str | None = None, value_mix_name: str = "vmix"):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are no multiple of {num_kv_heads} kv heads")
         self.nh, self.nkv, self.hd = int(num_heads), int(num_kv_heads), int(head_dim)
@@ -75,7 +81,15 @@ class GQAAttention(Mixer):
         self.gate_name = f"{name}.{gate}" if gate else None
         self.late_bias = bool(late_bias) and bool(bias)
         self.values_from_keys, self.qk_norm_whole = bool(values_from_keys), bool(qk_norm_whole)
-        self.chunk, self.sink, self.gate_per_head = int(chunk or 0), None if sink is None else float(sink), bool(gate_per_head)
+        self.chunk, self.gate_per_head = int(chunk or 0), bool(gate_per_head)
+        self.sink_name = f"{name}.{sink}" if isinstance(sink, str) else None
+        self.sink = None if sink is None or self.sink_name else float(sink)
+        if value_mix not in (None, "first", "later"):
+            raise ValueError(f"a layer is the first of those that mix values or a later one, not {value_mix!r}")
+        if value_mix and (share_kv or values_from_keys or (late_bias and bias)):
+            raise ValueError("mixed values come from a projection of their own with its bias inside the product")
+        self.value_mix, self.value_mix_name = value_mix, f"{name}.{value_mix_name}"
+        self.mix_share = None
         if weights not in ("softmax", "sigmoid"):
             raise ValueError(f"attention weights are a softmax or sigmoids, not {weights!r}")
         self.sigmoid = weights == "sigmoid"
@@ -99,7 +113,7 @@ class GQAAttention(Mixer):
             raise ValueError("a weight or an order for the q/k norm needs its eps")
         self.general = (self.softcap > 0 or self.qk_norm_eps is not None or self.vd != self.hd or self.keep_first > 0
                         or self.gate_name is not None or self.late_bias or self.values_from_keys or self.chunk > 0
-                        or self.sink is not None or self.sigmoid or pos.amplitude != 1.0)
+                        or sink is not None or self.sigmoid or pos.amplitude != 1.0 or value_mix is not None)
         self.scale = float(scale) if scale is not None else float(head_dim) ** -0.5
         self.window = int(window)
         self.share_kv = bool(share_kv)
@@ -135,6 +149,10 @@ class GQAAttention(Mixer):
             specs.append(WeightSpec(self.head_mix_name, (self.nh, self.nh), "head_mix"))
         if self.head_bias_name:
             specs.append(WeightSpec(self.head_bias_name, (self.nh,), "head_bias"))
+        if self.sink_name:
+            specs.append(WeightSpec(self.sink_name, (self.nh,), "bias"))
+        if self.value_mix:
+            specs.append(WeightSpec(self.value_mix_name, (), "share"))
         return specs
 
     def bind_own(self, tensors, rt: Runtime):
@@ -144,6 +162,10 @@ class GQAAttention(Mixer):
             self.q_weight, self.k_weight = (to_f32_vector(tensors[n], rt) for n in self.qk_norm_weights)
         if self.sink is not None:
             self.sinks = torch.full((self.nh,), self.sink, dtype=torch.float32, device=rt.device)
+        elif self.sink_name:
+            self.sinks = to_f32_vector(tensors[self.sink_name], rt)
+        if self.value_mix == "later":
+            self.mix_share = to_f32_vector(tensors[self.value_mix_name], rt).reshape(1)
         if self.sigmoid:
             self.head_mix = to_f32_vector(tensors[self.head_mix_name], rt) if self.head_mix_name else \
                 torch.eye(self.nh, dtype=torch.float32, device=rt.device)
@@ -186,6 +208,12 @@ class GQAAttention(Mixer):
         more = dict(whole=True, values_from_keys=self.values_from_keys) if self.qk_norm_whole or self.values_from_keys else {}
         if self.pos.amplitude != 1.0 or self.value_scale != 1.0:
             more.update(amplitude=self.pos.amplitude, v_scale=self.value_scale)
+        if self.value_mix:
+            v = qkv[:, (self.nh + self.nkv) * self.hd:self.qkv_features]
+            if self.value_mix == "first":
+                ctx.scratch["first values"] = v
+            else:
+                more.update(v_first=ctx.scratch["first values"], v_share=self.mix_share)
         wide = dict(vd=self.vd) if self.vd != self.hd else {}
         q = k.qk_prepare(qkv, ctx.positions, inv_freq, rot, trad, self.qk_norm_eps, g.slot_mapping if store else None,
                          cache.kv if store else None, self.nh, self.nkv, self.hd, self.vd, ctx.status,

@@ -59,20 +59,32 @@ class MixerOnly(PreNormBlock):
 
 
 class ParallelBlock(Part):
-    """h = norm(x); x <- x + (mixer(h) + ffn(h)): one norm, and both sublayers read its output.
+    """h = norm(x); x <- x + (mixer(h) + ffn(h)): one norm, and both sublayers read its output; or with `norm2`
+    x <- x + (mixer(norm(x)) + ffn(norm2(x))), two RMS norms of the same x in one pass.
 
     Mixer and feed-forward are built with `output=False`: their output projections are joined
     into one product over [mixer's heads | feed-forward's hidden layer], so that the two
     sublayers' outputs are added inside the product's 32-bit accumulators, and the block's
-    output is rounded once before the 32-bit residual sum takes it.  `ffn` may be None."""
+    output is rounded once before the 32-bit residual sum takes it.  `ffn` may be None.  A feed-forward of several output
+    matrices names them as `out_pieces`; one that multiplies with some of them itself (`kept_pieces`, known once it is bound)
+    hands on what it needs for that from `forward_inner` and adds its own outputs to the block's in `add_kept`."""
 
-    def __init__(self, mixer: Mixer, ffn: FeedForward | None, norm: Norm, width: int):
-        self.mixer, self.ffn, self.norm = mixer, ffn, norm
-        pieces = [mixer.out_piece] + ([ffn.out_piece] if ffn is not None else [])
+    def __init__(self, mixer: Mixer, ffn: FeedForward | None, norm: Norm, width: int, norm2: Norm | None = None):
+        self.mixer, self.ffn, self.norm, self.norm2 = mixer, ffn, norm, norm2
+        pieces = [mixer.out_piece]
+        if ffn is not None:
+            pieces += ffn.out_pieces if hasattr(ffn, "out_pieces") else [ffn.out_piece]
         self.out = JoinedLinear(width, pieces)
 
     def children(self):
-        return tuple(p for p in (self.norm, self.mixer, self.ffn, self.out) if p is not None)
+        return tuple(p for p in (self.norm, self.norm2, self.mixer, self.ffn, self.out) if p is not None)
+
+    def bind(self, tensors, rt):
+        self.rt = rt
+        for c in self.children():
+            if c is self.out:                     # the last one: the feed-forward is bound
+                c.leave_out(getattr(self.ffn, "kept_pieces", ()))
+            c.bind(tensors, rt)
 
     def cache_spec(self):
         return self.mixer.cache_spec()
@@ -86,13 +98,19 @@ class ParallelBlock(Part):
             bool(getattr(self.ffn, "supports_cuda_graph", True))
 
     def forward(self, delta, residual, ctx, cache):
-        h, residual = self.norm.forward(delta, residual)
+        if self.norm2 is not None:
+            h, h2, residual = self.norm.forward_pair(self.norm2, delta, residual)
+        else:
+            h, residual = self.norm.forward(delta, residual)
+            h2 = h
         joined = torch.empty((h.shape[0], self.out.in_features), dtype=self.rt.dtype, device=h.device)
         m = self.mixer.inner_features
         self.mixer.forward_inner(h, ctx, cache, out=joined[:, :m] if self.ffn is not None else joined)
-        if self.ffn is not None:
-            self.ffn.forward_inner(h, ctx, out=joined[:, m:])
-        return self.out.forward(joined), residual
+        if self.ffn is None:
+            return self.out.forward(joined), residual
+        kept = self.ffn.forward_inner(h2, ctx, out=joined[:, m:])
+        y = self.out.forward(joined)
+        return (self.ffn.add_kept(y, kept) if getattr(self.ffn, "kept_pieces", ()) else y), residual
 
 
 class SandwichBlock(Part):

@@ -171,34 +171,52 @@ class RoutedExperts(FeedForward):
 
 class PlainRoutedExperts(FeedForward):
     """y = sum over the token's chosen experts of w_e expert_e(x) (+ sigmoid(g . x) shared(x)), experts without a gate:
-    expert(x) = W_down act(W_up x), act the square of relu (or gelu_tanh, silu), no biases.
+    expert(x) = W_down act(W_up x), act the square of relu (or gelu in its exact form, gelu_tanh, silu), no biases.
 
-    Router: logits z = W_r x and scores s = softmax(z) over all experts, in 32-bit.  The `top` experts with the largest
-    s + correction are chosen (a vector of one number per expert that bears on the choice only; the lower index on a
-    tie); a chosen expert weighs w_e = s_e * scale, not renormalised.  A shared expert of the same form and a width of
-    its own runs for every token and is added times sigmoid(g . x), one number per token.
+    Router: logits z = W_r x and scores s in 32-bit, `scores="softmax"` (over all experts) or "sigmoid" (each logit alone).
+    The `top` experts with the largest s + correction are chosen (a vector of one number per expert that bears on the choice
+    only; the lower index on a tie); a chosen expert weighs w_e = s_e * scale, not renormalised.  `weigh="input"`: the
+    weight multiplies the expert's input instead of its output, y = sum of expert_e(w_e x); there are no biases, so it is
+    applied to the hidden values in front of the activation.  A shared expert of the same form and a width of its own
+    runs for every token and is added times sigmoid(g . x), one number per token.
 
-    All experts run side by side: the up matrices are stacked into one matrix and the down matrices laid side by side;
-    the activation kernel zeroes the columns of experts a token did not choose and multiplies the others by the token's
-    weight (the shared columns by the token's gate), and one product with the down matrices gives the weighted sum inside
-    the product's 32-bit accumulators.  The router's matrix and the shared gate's vector are stacked too, so that one
-    32-bit product gives a token's logits and its gate.  Nothing loops on the host and no token's result depends on what
-    else is in the batch, so a decode step can be captured.
+    Two ways to compute it, chosen once by size (`sparse`), neither of which loops on the host or makes a token's result
+    depend on what else is in the batch, so that a decode step can be captured:
+
+    * all experts side by side (small experts, and the 32-bit path): the up matrices are stacked into one matrix and the down
+      matrices laid side by side; the activation kernel zeroes the columns of experts a token did not choose and weighs the
+      others (the shared columns by the token's gate), and one product with the down matrices gives the sum inside the
+      product's 32-bit accumulators;
+    * grouped products (bfloat16, large experts): the (token, expert) pairs are sorted expert by expert on the device, a
+      tiled kernel multiplies each tile of pairs with its expert's up rows and applies weight and activation in its
+      epilogue, a second one multiplies with the expert's down matrix, and a last kernel adds a token's pair outputs to the
+      rest of the layer's output in 32-bit.  Only chosen experts' weights are read.
+
+    The router's matrix and the shared gate's vector are stacked, so that one 32-bit product gives a token's logits and its gate.
+    `output=False` leaves the down projections to the block, which joins them with the mixer's (`out_pieces`): with the
+    experts side by side all of them, with grouped products the shared expert's alone (`kept_pieces` are the others').
 
     Tensors, under `name`: router, correction; e<i>.up, e<i>.down; shared.up, shared.down, shared.sg."""
 
     supports_cuda_graph = True
+    SPARSE_MIN_BYTES = 8 << 20
 
     def __init__(self, width: int, experts: int, top: int, ff: int, name: str, scale: float = 1.0, shared_ff: int = 0,
                  activation: str = "relu2", correction: str | None = "correction", shared_gate: str | None = "sg",
                  weight_suffix: str = "", expert_prefix: str = "e", shared_name: str = "shared", router_name: str = "router",
-                 proj_names=("up", "down")):
-        if activation not in ("relu2", "gelu_tanh", "silu"):
+                 proj_names=("up", "down"), scores: str = "softmax", weigh: str = "output", output: bool = True,
+                 sparse: bool | None = None):
+        """`sparse`: grouped products (True), all experts side by side (False), or by size (None): grouped where the
+        experts' matrices together pass SPARSE_MIN_BYTES and more than twice as many experts exist as a token uses."""
+        if activation not in ("relu2", "gelu", "gelu_tanh", "silu"):
             raise ValueError(f"unknown activation {activation!r}")
+        if scores not in ("softmax", "sigmoid") or weigh not in ("output", "input"):
+            raise ValueError(f"unknown scores {scores!r} or place of the weights {weigh!r}")
         if not 0 < top <= experts:
             raise ValueError(f"top={top} of {experts} experts")
         self.width, self.E, self.top, self.ff, self.scale = int(width), int(experts), int(top), int(ff), float(scale)
         self.shared_ff, self.activation = int(shared_ff), activation
+        self.scores, self.weigh, self.output, self.want_sparse, self.sparse = scores, weigh, bool(output), sparse, False
         self.F = self.E * self.ff + self.shared_ff
         u, d = proj_names
         pre = [f"{name}.{expert_prefix}{i}" for i in range(self.E)] + ([f"{name}.{shared_name}"] if self.shared_ff else [])
@@ -208,13 +226,21 @@ class PlainRoutedExperts(FeedForward):
         self.router_name = f"{name}.{router_name}{weight_suffix}"
         self.correction_name = f"{name}.{correction}" if correction else None
         self.gate_name = f"{name}.{shared_name}.{shared_gate}{weight_suffix}" if self.shared_ff and shared_gate else None
+        self.out_pieces = [(n, w, None) for n, w in self.down_names]
+        self.kept_pieces = ()
+
+    @property
+    def inner_features(self) -> int:
+        """Columns of the hidden layer that go through the block's joined product."""
+        return self.shared_ff if self.sparse else self.F
 
     def own_weight_specs(self):
         specs = [WeightSpec(self.router_name, (self.E, self.width), "matrix")]
         if self.correction_name:
             specs.append(WeightSpec(self.correction_name, (self.E,), "bias"))
         specs += [WeightSpec(n, (w, self.width), "matrix") for n, w in self.up_names]
-        specs += [WeightSpec(n, (self.width, w), "matrix") for n, w in self.down_names]
+        if self.output:                                            # else the block's joined product declares them
+            specs += [WeightSpec(n, (self.width, w), "matrix") for n, w in self.down_names]
         if self.gate_name:
             specs.append(WeightSpec(self.gate_name, (1, self.width), "matrix"))
         return specs
@@ -231,16 +257,72 @@ class PlainRoutedExperts(FeedForward):
         downs = [to_compute(tensors[n], rt) for n, _ in self.down_names]
         if len({m.dtype for m in ups + downs}) > 1:
             ups, downs = [m.float() for m in ups], [m.float() for m in downs]
-        self.up = torch.cat(ups, 0).contiguous()                  # [F, width]
-        self.down = torch.cat(downs, 1).contiguous()              # [width, F]
+        can = (rt.dtype == torch.bfloat16 and all(m.dtype == torch.bfloat16 for m in ups + downs) and self.width % 8 == 0
+               and self.ff % 8 == 0 and rt.device.type == "cuda" and hasattr(rt.k, "moe_grouped_up"))
+        big = 2 * self.E * self.ff * self.width * 2 >= self.SPARSE_MIN_BYTES and self.E > 2 * self.top
+        self.sparse = can and (big if self.want_sparse is None else bool(self.want_sparse))
+        self.shared_up = self.shared_down = self.down = None
+        self.kept_pieces = ()
+        if self.sparse:
+            if self.shared_ff:
+                self.shared_up = ups.pop().contiguous()
+                shared_down = downs.pop()
+                self.shared_down = shared_down.contiguous() if self.output else None
+            self.kept_pieces = tuple(n for n, _ in self.down_names[:self.E])
+            self.down = torch.cat(downs, 0).contiguous()          # [E width, ff], one under the other
+        elif self.output:
+            self.down = torch.cat(downs, 1).contiguous()          # [width, F]
+        self.up = torch.cat(ups, 0).contiguous()                  # [F, width], or the routed experts' [E ff, width]
 
     def weight_bytes(self):
-        return sum(t.numel() * t.element_size() for t in (self.router, self.up, self.down))
+        return sum(t.numel() * t.element_size() for t in (self.router, self.up, self.down, self.shared_up, self.shared_down)
+                   if t is not None)
+
+    def active_weight_bytes(self, tokens: int) -> int:
+        """Bytes of weights a step of `tokens` tokens reads at most: all with the experts side by side; with grouped
+        products the router, the shared expert's and those of at most tokens * top experts."""
+        if not self.sparse:
+            return self.weight_bytes()
+        used = min(self.E, tokens * self.top)
+        rest = sum(t.numel() * t.element_size() for t in (self.router, self.shared_up, self.shared_down) if t is not None)
+        return rest + self.router.element_size() * 2 * used * self.ff * self.width
+
+    def route(self, x, want_chosen: bool = False):
+        """-> (weights [T, E], chosen [T, top] or None, the shared gate's values in front of its sigmoid [T, 1] or None)."""
+        k = self.rt.k
+        z = k.linear(x, self.router, None, torch.float32)
+        more = {} if self.scores == "softmax" else dict(scores=self.scores)
+        w = k.moe_route(z, self.top, experts=self.E, correction=self.correction, scale=self.scale, want_chosen=want_chosen, **more)
+        w, chosen = w if want_chosen else (w, None)
+        return w, chosen, z[:, self.E:] if self.gate_name else None
+
+    def forward_inner(self, x, ctx, out=None):
+        """Without grouped products: the hidden layers side by side after weight and activation, [T, F], into `out` where one
+        is given.  With them: the shared expert's into `out`; -> what `add_kept` takes."""
+        k = self.rt.k
+        status = ctx.status if ctx is not None else None
+        more = dict(weigh_input=True) if self.weigh == "input" else {}
+        if not self.sparse:
+            w, _, gate = self.route(x)
+            return k.moe_plain_act(k.linear(x, self.up, None, self.rt.dtype), w, self.E, self.ff, self.activation, shared_gate=gate,
+                                   out=out, **more)
+        w, chosen, gate = self.route(x, want_chosen=True)
+        plan = k.moe_sort(chosen, w)
+        y = k.moe_grouped_up(x, plan, self.up, self.E, self.ff, self.activation, weigh_input=self.weigh == "input", status=status)
+        pairs = k.moe_grouped_down(y, plan, self.down, self.E, self.ff, stacked=True, tokens=x.shape[0], status=status)
+        if self.shared_ff:
+            k.plain_up(x, self.shared_up, self.activation, gate, out=out, status=status)
+        return pairs, plan
+
+    def add_kept(self, y, kept):
+        """y [T, width] plus the token's pair outputs in the order of its choices, in 32-bit, rounded once."""
+        pairs, plan = kept
+        return self.rt.k.moe_combine(pairs, plan, y, plan[2].numel() // self.top, self.top, self.rt.dtype)
 
     def forward(self, x, ctx):
         k = self.rt.k
-        z = k.linear(x, self.router, None, torch.float32)
-        w = k.moe_route(z, self.top, experts=self.E, correction=self.correction, scale=self.scale)
-        hidden = k.linear(x, self.up, None, self.rt.dtype)
-        act = k.moe_plain_act(hidden, w, self.E, self.ff, self.activation, shared_gate=z[:, self.E:] if self.gate_name else None)
-        return k.linear(act, self.down, None, self.rt.dtype)
+        if not self.sparse:
+            return k.linear(self.forward_inner(x, ctx), self.down, None, self.rt.dtype)
+        out = torch.empty((x.shape[0], self.shared_ff), dtype=self.rt.dtype, device=x.device)
+        kept = self.forward_inner(x, ctx, out=out)
+        return self.add_kept(k.linear(out, self.shared_down, None, self.rt.dtype) if self.shared_ff else None, kept)

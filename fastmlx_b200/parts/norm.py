@@ -54,6 +54,13 @@ class RMSNorm(Norm):
             b.release(x)
         return out, stream
 
+    def forward_pair(self, other: "RMSNorm", x, residual):
+        """-> (norm(s) * w, norm(s) * w', s): this norm and `other` (of the same eps) of the same sum s, in one pass."""
+        if other.eps != self.eps or other.width != self.width:
+            raise ValueError("two norms in one pass share their width and eps")
+        return self.rt.k.add_rmsnorm(x, residual, self.weight, self.eps, stream_dtype=torch.float32, out_dtype=self.rt.dtype,
+                                     weight2=other.weight)
+
     def fold(self):
         """(weight, eps) for a kernel that normalises its input rows itself."""
         return (self.weight, self.eps)

@@ -24,7 +24,7 @@ def embedding(ids, table, status, out_dtype=None):
     return out.to(out_dtype) if out_dtype is not None else out
 
 
-def add_rmsnorm(x, residual, weight, eps, stream_dtype=None, out_dtype=None):
+def add_rmsnorm(x, residual, weight, eps, stream_dtype=None, out_dtype=None, weight2=None):
     act = x.dtype if x is not None else (out_dtype or residual.dtype)
     if residual is not None:
         h = residual.to(F64) if x is None else (x.to(F64) + residual.to(F64))
@@ -34,8 +34,10 @@ def add_rmsnorm(x, residual, weight, eps, stream_dtype=None, out_dtype=None):
     else:
         residual = x
     h = residual.to(F64)
-    out = h * torch.rsqrt((h * h).mean(-1, keepdim=True) + eps) * weight.to(F64)
-    return out.to(act), residual
+    n = h * torch.rsqrt((h * h).mean(-1, keepdim=True) + eps)
+    if weight2 is not None:
+        return (n * weight.to(F64)).to(act), (n * weight2.to(F64)).to(act), residual
+    return (n * weight.to(F64)).to(act), residual
 
 
 def silu_mul(gate_up, block=None):
@@ -191,7 +193,7 @@ def _rotate(heads, positions, inv_freq, rotary_dim, traditional):
 
 def qk_prepare(qkv, positions, inv_freq, rotary_dim, traditional, norm_eps, slot_mapping, kv, nh, nkv, hd, vd, status,
                bias=None, q_weight=None, k_weight=None, norm_first=False, whole=False, values_from_keys=False, amplitude=1.0,
-               v_scale=1.0):
+               v_scale=1.0, v_first=None, v_share=None):
     T = qkv.shape[0]
     n_qk = (nh + nkv) * hd
     row = qkv[:, :n_qk + (0 if values_from_keys else nkv * vd)].to(F64)
@@ -199,6 +201,9 @@ def qk_prepare(qkv, positions, inv_freq, rotary_dim, traditional, norm_eps, slot
         row = row + bias.to(F64)
     if values_from_keys:                       # a token's values are its keys as they were projected
         row = torch.cat([row, row[:, nh * hd:n_qk]], 1)
+    if v_first is not None:                    # the values mixed with those of another layer
+        lam = v_share.to(F64)
+        row = torch.cat([row[:, :n_qk], (1 - lam) * row[:, n_qk:] + lam * v_first.to(F64)], 1)
     heads = row[:, :n_qk].reshape(T, nh + nkv, hd)
     w = torch.ones(nh + nkv, hd, dtype=F64)
     if q_weight is not None:
@@ -338,10 +343,10 @@ def sigmoid_gate(o, gate, group=1):
 
 
 def moe_route(logits, top, groups=1, keep=1, want_chosen=False, experts=None, correction=None, scale=1.0, logit_bias=None,
-              renorm=False):
+              renorm=False, scores="softmax"):
     T, E = logits.shape[0], int(experts if experts is not None else logits.shape[1])
     z = logits[:, :E].to(torch.float32) + (logit_bias if logit_bias is not None else 0.0)
-    s = torch.softmax(z, -1)
+    s = torch.softmax(z, -1) if scores == "softmax" else torch.sigmoid(z)
     pick = s if correction is None else s + correction.to(torch.float32)
     w = torch.zeros(T, E, dtype=torch.float32)
     chosen = torch.full((T, top), -1, dtype=torch.int32)
@@ -361,10 +366,15 @@ def moe_route(logits, top, groups=1, keep=1, want_chosen=False, experts=None, co
     return (w, chosen) if want_chosen else w
 
 
-def moe_plain_act(u, weights, E, ff, act, shared_gate=None, out=None):
+def moe_plain_act(u, weights, E, ff, act, shared_gate=None, out=None, weigh_input=False):
     T, F = u.shape
     x = u.to(F64)
-    if act == "relu2":
+    if weigh_input:                            # the weights in front of the activation (the shared columns' gate stays behind it)
+        x = torch.cat([x[:, :E * ff] * weights.to(F64).repeat_interleave(ff, dim=1), x[:, E * ff:]], 1)
+        weights = torch.ones_like(weights)
+    if act == "gelu":
+        a = 0.5 * x * (1.0 + torch.erf(x * 0.5 ** 0.5))
+    elif act == "relu2":
         a = torch.relu(x) ** 2
     elif act == "gelu_tanh":
         a = 0.5 * x * (1.0 + torch.tanh(0.7978845608028654 * (x + 0.044715 * x ** 3)))
@@ -679,10 +689,14 @@ def channel_scan(qkv, g, beta, ctx, state, H, G, D, Dv):
     return out
 
 
-def head_norm_gate(o, gate, weight, eps, H, Dv, out_dtype, act="sigmoid", out=None):
+def head_norm_gate(o, gate, weight, eps, H, Dv, out_dtype, act="sigmoid", out=None, divisor=None):
     T = o.shape[0]
     v = o.to(F64).reshape(T, H, Dv)
-    v = (v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps) * weight.to(F64)).reshape(T, H * Dv)
+    if divisor is not None:                    # (n . q, gates): the normaliser, not below a floor
+        nq, gates = divisor
+        v = v / (torch.maximum(nq.to(F64).abs(), gates[:, :, 2].to(F64)) + 1e-6)[:, :, None]
+    w = weight.to(F64).reshape(-1, Dv)         # one row for all heads, or one per head
+    v = (v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps) * w).reshape(T, H * Dv)
     z = gate.to(F64)
     res = (v * (torch.sigmoid(z) if act == "sigmoid" else _silu(z))).to(out_dtype)
     if out is not None:
@@ -717,3 +731,55 @@ def logit_cap(x, scale, cap):
     v = x.to(F64) * scale
     x.copy_((cap * torch.tanh(v / cap) if cap and cap > 0 else v).to(x.dtype))
     return x
+
+
+# ----------------------------------------------------------------------------- the matrix memory with exponential gates
+def mlstm_gates(z, bias, cap, ctx, state, m_off, H):
+    """z[T, input gates (H) | forget gates (H)] -> [T, H, 4]: what the state is kept by, what the new key and value are put in by,
+    exp(-m), nothing; the running maxima in the slots move on."""
+    T = z.shape[0]
+    out = torch.zeros(T, H, 4, dtype=torch.float32)
+    g = cap * torch.tanh((z.to(F64) + bias.to(F64)) / cap)
+    i, f = g[:, :H], -_softplus(-g[:, H:])
+    for r in range(ctx.R):
+        slot = int(ctx.row_slot[r])
+        a, e = int(ctx.row_start[r]), int(ctx.row_start[r + 1])
+        if slot < 0 or e <= a:
+            continue
+        m = state[slot, m_off:m_off + H].to(F64)
+        for t in range(a, e):
+            new = torch.maximum(f[t] + m, i[t])
+            out[t, :, 0], out[t, :, 1], out[t, :, 2] = torch.exp(f[t] + m - new), torch.exp(i[t] - new), torch.exp(-new)
+            m = new
+        state[slot, m_off:m_off + H] = m.to(torch.float32)
+    return out
+
+
+def mlstm_scan(proj, gates, ctx, state, H, D, Dv):
+    """-> (S^T q [T, H*Dv], n . q [T, H]) in 32-bit, from and into the slots ([H, Dv + 1, D], n the last row of a head)."""
+    T, n = proj.shape[0], H * (Dv + 1) * D
+    out, nq = torch.zeros(T, H * Dv, dtype=torch.float32), torch.zeros(T, H, dtype=torch.float32)
+    x = proj.to(F64)
+    for r in range(ctx.R):
+        slot = int(ctx.row_slot[r])
+        a, e = int(ctx.row_start[r]), int(ctx.row_start[r + 1])
+        if slot < 0 or e <= a:
+            continue
+        S = state[slot, :n].to(F64).reshape(H, Dv + 1, D)
+        for t in range(a, e):
+            q, k = x[t, :H * D].reshape(H, D) * D ** -0.5, x[t, H * D:2 * H * D].reshape(H, D)
+            v = torch.cat([x[t, 2 * H * D:2 * H * D + H * Dv].reshape(H, Dv), torch.ones(H, 1, dtype=F64)], 1)
+            keep, put = gates[t, :, 0].to(F64), gates[t, :, 1].to(F64)
+            S = keep[:, None, None] * S + (put[:, None] * v)[:, :, None] * k[:, None, :]
+            o = (S * q[:, None, :]).sum(-1)
+            out[t], nq[t] = o[:, :Dv].reshape(-1).to(torch.float32), o[:, Dv].to(torch.float32)
+        state[slot, :n] = S.reshape(-1).to(torch.float32)
+    return out, nq
+
+
+def mlstm_step(proj, z, bias, cap, ctx, state, H, D, Dv, weight, eps, out_dtype, out=None):
+    """Rows of one token each: gates, recurrence, norm and output gate (proj holds q | k | v | output gate)."""
+    gates = mlstm_gates(z, bias, cap, ctx, state, H * (Dv + 1) * D, H)
+    o, nq = mlstm_scan(proj, gates, ctx, state, H, D, Dv)
+    n = 2 * H * D + H * Dv
+    return head_norm_gate(o, proj[:, n:n + H * Dv], weight, eps, H, Dv, out_dtype, out=out, divisor=(nq, gates))

@@ -79,14 +79,18 @@ mlstm_gates_kernel(const float* z, long long z_stride, const float* __restrict__
   if (t0 < n && t1 == n) *mp = m;                  // (every thread has read the old one: the barrier above)
 }
 
-// Four neighbouring values of which `have` exist; `vec`: their start is aligned for one access.
+// Four neighbouring values of which `have` exist (the others are zero); `vec`, the same for all threads: their starts are aligned
+// for one access and `have` is four or more, or none.  Selects and not branches: the lanes stay together.
 template <typename T> __device__ __forceinline__ float4 some4(const T* p, int have, bool vec) {
-  if (vec && have >= 4) return load4(p);
   float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-  if (have > 0) x.x = to_f(p[0]);
-  if (have > 1) x.y = to_f(p[1]);
-  if (have > 2) x.z = to_f(p[2]);
-  if (have > 3) x.w = to_f(p[3]);
+  if (vec) {
+    if (have >= 4) x = load4(p);
+  } else {
+    x.x = have > 0 ? to_f(p[0]) : 0.f;
+    x.y = have > 1 ? to_f(p[1]) : 0.f;
+    x.z = have > 2 ? to_f(p[2]) : 0.f;
+    x.w = have > 3 ? to_f(p[3]) : 0.f;
+  }
   return x;
 }
 
@@ -139,22 +143,18 @@ mlstm_scan_kernel(const T* proj, long long stride, const float4* gates, const in
     for (int it = 0; it < NIT; ++it) {
       const int item = threadIdx.x + it * 128;
       const int s = item / CH, e = 4 * (item - s * CH);
-      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (s < cnt) {                               // (a run's missing tokens: k = q = v = 0)
-        const T* row = proj + (long long)(first + t0 + s) * stride;
-        if (e < DP) x = some4(row + koff + e, D - e, vec_in);
-        else if (e < 2 * DP) x = some4(row + qoff + e - DP, D - (e - DP), vec_in);
-        else {
-          const int c = c0 + e - 2 * DP;
-          x = some4(row + voff + c, Dv - c, vec_in);
-          if (c <= Dv && Dv < c + 4) {             // n's column has the value 1
-            if (c == Dv) x.x = 1.f;
-            else if (c + 1 == Dv) x.y = 1.f;
-            else if (c + 2 == Dv) x.z = 1.f;
-            else x.w = 1.f;
-          }
-        }
-      }
+      // one source per piece of four: k, q or the values (a run's missing tokens have none: k = q = v = 0)
+      const T* row = proj + (long long)(first + t0 + min(s, cnt - 1)) * stride;
+      const bool is_k = e < DP, is_q = !is_k && e < 2 * DP;
+      const int d = is_k ? e : is_q ? e - DP : c0 + e - 2 * DP;
+      const T* src = row + (is_k ? koff : is_q ? qoff : voff) + d;
+      const int have = s < cnt ? (is_k || is_q ? D : Dv) - d : 0;
+      float4 x = some4(src, have, vec_in);
+      const int one = is_k || is_q || s >= cnt ? -1 : Dv - d;          // n's column has the value 1
+      x.x = one == 0 ? 1.f : x.x;
+      x.y = one == 1 ? 1.f : x.y;
+      x.z = one == 2 ? 1.f : x.z;
+      x.w = one == 3 ? 1.f : x.w;
       ahead[it] = x;
     }
     if (threadIdx.x < TB) {
@@ -173,9 +173,10 @@ mlstm_scan_kernel(const T* proj, long long stride, const float4* gates, const in
     for (int it = 0; it < NIT; ++it) {
       const int item = threadIdx.x + it * 128;
       const int s = item / CH, e = 4 * (item - s * CH);
-      if (s < TB) *reinterpret_cast<float4*>(buf + s * ROWF + e) = ahead[it];
+      if (TB * CH % 128 == 0 || s < TB) *reinterpret_cast<float4*>(buf + s * ROWF + e) = ahead[it];
     }
     if (threadIdx.x < TB) *reinterpret_cast<float2*>(buf + threadIdx.x * ROWF + 2 * DP + COLS) = ahead_gate;
+    __syncwarp();
     __syncthreads();
     if (run + 1 < n_runs) fetch_run(run + 1);
     const int cnt = min(TB, n - run * TB);
@@ -212,6 +213,7 @@ mlstm_scan_kernel(const T* proj, long long stride, const float4* gates, const in
           o[j * CPT + c] = pair_sum(a) + pair_sum(b);
         }
       }
+      __syncwarp();
       const float mine = reduce_scatter<NV, L>(o, sub) * q_scale;
       const int at = sub * NV / L, j = at / CPT, col = col0 + at % CPT;
       if (sub % (L / NV) == 0 && s + j < cnt && col <= Dv) {
@@ -324,6 +326,7 @@ mlstm_step_kernel(const TP* proj, long long stride, const float* z, long long z_
       }
     }
     if (j0 - grp + U * GROUPS <= Dv) load_rows(j0 + U * GROUPS);
+    __syncwarp();
 #pragma unroll
     for (int u = 0; u < U; ++u) {
 #pragma unroll

@@ -67,7 +67,8 @@ def one_layer(mixer, width=48, vocab=61, mlp=None, eps=1e-6):
 def lively_tensors(config, seed, dtype=torch.bfloat16, settled=False):
     """Weights at which every mechanism counts: matrices that keep activations of order one, forget gates spread over what
     keeps a state for a few tokens and for hundreds, sinks, shares of a mix and norm weights away from zero and one.
-    `settled`: routers whose rows differ much in length, so that rounding seldom changes a choice."""
+    `settled`: every token's embedding names its experts, layer by layer, on dimensions of their own that the routers read, so
+    that rounding seldom changes a choice."""
     from fastmlx_b200 import registry
     cfg, model = registry.build_model(config)
     g = torch.Generator().manual_seed(seed)
@@ -81,7 +82,7 @@ def lively_tensors(config, seed, dtype=torch.bfloat16, settled=False):
         elif spec.name.endswith(".sink"):
             t = t * 1.5
         elif spec.name.endswith(".router"):
-            t = t * (3.0 if settled else 1.5) / shape_in(spec)
+            t = t * (0.1 if settled else 1.5) / shape_in(spec)
         elif spec.kind == "matrix":
             t = t / shape_in(spec)
         elif spec.kind == "embedding":
@@ -92,8 +93,20 @@ def lively_tensors(config, seed, dtype=torch.bfloat16, settled=False):
             t = t * 0.2
         elif spec.kind == "norm":
             t = 1.0 + 0.2 * t
-        out[spec.name] = t.to(dtype)
-    return out
+        out[spec.name] = t
+    if settled:
+        at, vocab = 0, config["vocab"]
+        for i, spec in enumerate(config["layers"]):
+            if not spec["mlp"] or spec["mlp"]["kind"] != "moe":
+                continue
+            E, top = spec["mlp"]["router"]["experts"], spec["mlp"]["router"]["top"]
+            for e in range(E):
+                out[f"l{i}.mlp.router"][e, at + e] = 3.0
+            chosen = torch.zeros(vocab, E)
+            chosen.scatter_(1, torch.rand(vocab, E, generator=g).argsort(1)[:, :top], 1.0)
+            out["embed"][:, at:at + E] = (2 * chosen - 1) * (2.0 + 1.3 * torch.rand(vocab, E, generator=g))
+            at += E
+    return {n: t.to(dtype) for n, t in out.items()}
 
 
 def shape_in(spec):

@@ -35,7 +35,9 @@ one) whose active parameters equal the Llama layer's; `sorupel`, `kafepel` and `
 those sizes: sigmoid attention with mixed heads beside a retention in every layer, gated feed-forwards alternating with a
 mixture of 8 squared-relu experts and a gated shared one; a Bonerax model: gated linear attention, a delta rule with a decay
 per key channel, and windowed attention beside such a delta rule, gated feed-forwards alternating with a mixture of 16
-gated experts, 4 per token).
+gated experts, 4 per token); `gepadra` likewise (a Gepadra model: windowed attention that keeps the first tokens, with sinks and
+mixed values, beside a matrix memory with exponential gates; clamped gated feed-forwards alternating with a mixture of 16
+gelu experts, 2 per token, and a shared one).
 
 Every timed step reads well over 126 MB (weights alone are 2.5 GB), so no input stays in L2
 between iterations.  tamnd/fastmlx publishes no number to compare with, and cannot run here
@@ -485,6 +487,23 @@ def bonerax_like(shape: dict, layers: int, window: int = 1024) -> dict:
             "norm": {"eps": 1e-6}, "layers": out}
 
 
+def gepadra_like(shape: dict, layers: int, window: int = 1024) -> dict:
+    """A Gepadra configuration with a Llama shape's width, heads and vocabulary: layers in the pattern attention (sliding
+    window beside 8 kept tokens, half of each head rotated, mixed values), matrix memory, matrix memory, attention;
+    feed-forwards are a clamped gated one of the Llama layer's size, and in every second layer 16 gelu experts of half its
+    hidden size, 2 per token, with a shared one of half of it (the parameters a token uses are the same)."""
+    d, nh, nkv, hd = shape["hidden_size"], shape["num_attention_heads"], shape["num_key_value_heads"], shape["head_dim"]
+    ff = shape["intermediate_size"]
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 2}, "expert": {"ff": ff // 2}, "shared": {"ff": ff // 2}}
+    att = {"heads": nh, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": window, "keep_first": 8},
+           "rot": {"dims": hd // 2, "base": 500000.0}, "v_mix": True}
+    mem = {"heads": nh, "dim": hd, "vdim": hd, "gate_cap": 15.0}
+    return {"architecture": "Gepadra", "vocab": shape["vocab_size"], "width": d, "norm": {"eps": 1e-6},
+            "layers": [{"type": "mlstm" if i % 4 in (1, 2) else "attention", "mixer": mem if i % 4 in (1, 2) else att,
+                        "mlp": moe if i % 2 else dense} for i in range(layers)]}
+
+
 def step_weight_bytes(model, tokens: int) -> int:
     """Bytes of weights a step of `tokens` tokens must read: every run of the schedule reads its layer (a looped layer
     once per pass); a routed feed-forward with grouped products reads the experts its tokens chose, at most."""
@@ -551,7 +570,8 @@ def compare_designs(shapes, layers: int, context: int, steps: int, warmup: int, 
         name, shape = SHAPES[key]
         make = {"llama": lambda: dict(shape, num_hidden_layers=layers), "medirax": lambda: medirax_like(shape, layers),
                 "gekavik": lambda: gekavik_like(shape, layers), "sorupel": lambda: sorupel_like(shape, layers),
-                "kafepel": lambda: kafepel_like(shape, layers), "bonerax": lambda: bonerax_like(shape, layers)}
+                "kafepel": lambda: kafepel_like(shape, layers), "bonerax": lambda: bonerax_like(shape, layers),
+                "gepadra": lambda: gepadra_like(shape, layers)}
         out[key] = {"layers": layers, "context": context}
         for design in which:
             out[key][design] = design_numbers(make[design](), shape["vocab_size"], pk, context, steps, warmup)
@@ -577,7 +597,7 @@ def main() -> int:
                     "layers of equal size are measured side by side; prints that comparison alone")
     ap.add_argument("--design-layers", type=int, default=8, help="layers of each model of the --designs comparison")
     ap.add_argument("--design-set", default="llama,medirax", help="which designs the --designs comparison measures "
-                    "(comma-separated, of llama, medirax, gekavik, sorupel, kafepel, bonerax)")
+                    "(comma-separated, of llama, medirax, gekavik, sorupel, kafepel, bonerax, gepadra)")
     ap.add_argument("--only-steps", type=int, default=0,
                     help="for a profiler's launch list: fill the batch, run this many decode steps and stop (no timing, no JSON line); "
                     "with --designs: a 2,048-token prompt step and the decode steps of the first design named, at the first size named")
@@ -603,14 +623,15 @@ def main() -> int:
     if args.designs:
         keys = [k for k in args.designs.split(",") if k]
         which = [w for w in args.design_set.split(",") if w]
-        if any(w not in ("llama", "medirax", "gekavik", "sorupel", "kafepel", "bonerax") for w in which):
-            print(f"bench.py: --design-set takes llama, medirax, gekavik, sorupel, kafepel, bonerax (got {args.design_set!r})")
+        if any(w not in ("llama", "medirax", "gekavik", "sorupel", "kafepel", "bonerax", "gepadra") for w in which):
+            print(f"bench.py: --design-set takes llama, medirax, gekavik, sorupel, kafepel, bonerax, gepadra (got {args.design_set!r})")
             return 2
         if args.only_steps > 0:
             shape = SHAPES[keys[0]][1]
             make = {"llama": lambda: dict(shape, num_hidden_layers=args.design_layers), "medirax": lambda: medirax_like(shape, args.design_layers),
                     "gekavik": lambda: gekavik_like(shape, args.design_layers), "sorupel": lambda: sorupel_like(shape, args.design_layers),
-                    "kafepel": lambda: kafepel_like(shape, args.design_layers), "bonerax": lambda: bonerax_like(shape, args.design_layers)}
+                    "kafepel": lambda: kafepel_like(shape, args.design_layers), "bonerax": lambda: bonerax_like(shape, args.design_layers),
+                    "gepadra": lambda: gepadra_like(shape, args.design_layers)}
             design_steps(make[which[0]](), shape["vocab_size"], args.batch, min(args.context, 4096), args.only_steps, warmup,
                          not args.no_cuda_graphs)
             print(f"ran a {PREFILL_TOKENS}-token prompt step and {args.only_steps} decode steps of batch {args.batch} of {which[0]} at the {keys[0]} sizes")

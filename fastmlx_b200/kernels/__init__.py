@@ -875,25 +875,43 @@ def head_norm_gate(o, gate, weight, eps, H, Dv, out_dtype, act: str = "sigmoid",
 # ----------------------------------------------------------------------------- the matrix memory with exponential gates
 def mlstm_gates(z, bias, cap: float, ctx, state, m_off: int, H: int) -> torch.Tensor:
     """The capped log gates of z[T, input gates (H) | forget gates (H)] (32-bit, rows may be a slice) with bias[2 H], run over every
-    request's tokens: -> [T, H, 4] in 32-bit, (exp(f + m - m'), exp(i - m'), exp(-m'), 0) with m' = max(f + m, i) the running
+    request's tokens: -> [T, H, 4] in 32-bit, (exp(f + m - m'), exp(i - m'), exp(-m'), f + m - m') with m' = max(f + m, i) the running
     maximum, which is read from and left in the requests' slots at m_off."""
     _need_cuda(z, bias)
     assert z.dtype == torch.float32 and z.stride(1) == 1 and z.shape[1] == 2 * H and bias.dtype == torch.float32 and bias.numel() == 2 * H
     gates = torch.empty((z.shape[0], H, 4), dtype=torch.float32, device=z.device)
     call("mlstm", "fmx_mlstm_gates", z.data_ptr(), z.stride(0), bias.data_ptr(), float(cap), ctx.row_start.data_ptr(),
-         ctx.row_slot.data_ptr(), state.data_ptr(), state.stride(0), int(m_off), gates.data_ptr(), ctx.R, H, state.shape[0], _stream())
+         ctx.row_slot.data_ptr(), state.data_ptr(), state.stride(0), int(m_off), gates.data_ptr(), ctx.R, H, state.shape[0],
+         int(ctx.max_q_len), _stream())
     return gates
 
 
-def mlstm_scan(proj, gates, ctx, state, H: int, D: int, Dv: int, lanes: int = 0, cpt: int = 0):
+MEMORY_CHUNK_MIN = 24        # steps whose longest row brings at least this many tokens walk the matrix memory in runs of 64 tokens
+
+
+def can_mlstm_chunks(proj, state, D: int, Dv: int) -> bool:
+    """Do the matrix products over runs of tokens take this recurrence?  bfloat16 projections in 16-byte rows, keys of 32, 64, 96
+    or 128 values, values in eights."""
+    return (proj.dtype == torch.bfloat16 and D in (32, 64, 96, 128) and Dv % 8 == 0 and proj.stride(0) % 8 == 0 and proj.stride(1) == 1
+            and proj.data_ptr() % 16 == 0 and state.stride(0) % 2 == 0 and state.data_ptr() % 8 == 0)
+
+
+def mlstm_scan(proj, gates, ctx, state, H: int, D: int, Dv: int, lanes: int = 0, cpt: int = 0, chunks: bool | None = None, columns: int = 0):
     """The matrix memory over every request's tokens of the step, in order, from and into the requests' slots (S^T per head with n as
     its last row, [H, Dv + 1, D], at the head of a slot): S <- keep S + put k v^T, n <- keep n + put k.  proj[T, q (H*D) | k (H*D) |
     v (H*Dv) ...], gates as `mlstm_gates` left them.  -> (S^T q [T, H*Dv], n . q [T, H]) in 32-bit, q times D^-1/2, not divided
-    yet.  `lanes` (8, 16, 32) and `cpt` (1, 2, 4; 0: the library's choice): lanes that share a column, and columns that they hold."""
+    yet.  `chunks`: in runs of 64 tokens as matrix products (True; `columns` of S per block, 0: the library's choice), token by
+    token (False), or by type and size (None).  `lanes` (8, 16, 32) and `cpt` (1, 2, 4; 0: the library's choice), token by token:
+    lanes that share a column, and columns that they hold."""
     T = proj.shape[0]
     assert proj.stride(1) == 1 and gates.is_contiguous() and gates.shape == (T, H, 4)
     out = torch.empty((T, H * Dv), dtype=torch.float32, device=proj.device)
     nq = torch.empty((T, H), dtype=torch.float32, device=proj.device)
+    if chunks or (chunks is None and not lanes and not cpt and ctx.max_q_len >= MEMORY_CHUNK_MIN and can_mlstm_chunks(proj, state, D, Dv)):
+        call("mlstm", "fmx_mlstm_chunks", proj.data_ptr(), proj.stride(0), gates.data_ptr(), ctx.row_start.data_ptr(),
+             ctx.row_slot.data_ptr(), state.data_ptr(), state.stride(0), out.data_ptr(), nq.data_ptr(), ctx.R, H, D, Dv, state.shape[0],
+             int(columns), _stream())
+        return out, nq
     call("mlstm", "fmx_mlstm_scan", proj.data_ptr(), proj.stride(0), gates.data_ptr(), ctx.row_start.data_ptr(), ctx.row_slot.data_ptr(),
          state.data_ptr(), state.stride(0), out.data_ptr(), nq.data_ptr(), ctx.R, H, D, Dv, state.shape[0], _dt(proj), int(lanes), int(cpt),
          _stream())

@@ -100,7 +100,8 @@ _SIGNATURES = {
         "fmx_channel_scan": [_P, _P, _P, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     },
     "mlstm": {
-        "fmx_mlstm_gates": [_P, _L, _P, _F, _P, _P, _P, _L, _L, _P, _I, _I, _I, _P],
+        "fmx_mlstm_gates": [_P, _L, _P, _F, _P, _P, _P, _L, _L, _P, _I, _I, _I, _I, _P],
+        "fmx_mlstm_chunks": [_P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I, _P],
         "fmx_mlstm_scan": [_P, _L, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
         "fmx_mlstm_step": [_P, _L, _I, _P, _L, _P, _F, _P, _P, _P, _L, _L, _P, _F, _P, _L, _I, _I, _I, _I, _I, _I, _P],
     },

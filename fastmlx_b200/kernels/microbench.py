@@ -8,6 +8,8 @@ launches), for tuning and for profiler captures on a small case.
     python -m fastmlx_b200.kernels.microbench --kernel sample --batch 8 --N 128256
     python -m fastmlx_b200.kernels.microbench --kernel recurrence --batch 1 --qlen 2048 --nh 64 --hd 64 --state 128
     python -m fastmlx_b200.kernels.microbench --kernel channel --batch 1 --qlen 2048 --nh 32 --hd 64 --state 64
+    python -m fastmlx_b200.kernels.microbench --kernel memory --batch 1 --qlen 2048 --nh 32 --hd 64 --state 64
+    python -m fastmlx_b200.kernels.microbench --kernel experts --M 2048 --N 4096 --K 2048
     python -m fastmlx_b200.kernels.microbench --kernel attn_masked --batch 64 --qlen 1 --ctx 4096 --hd 64
     python -m fastmlx_b200.kernels.microbench --kernel attn_mixed --batch 64 --qlen 1 --ctx 4096 --hd 64
 """
@@ -182,6 +184,77 @@ def _channel(a) -> int:
     return 0
 
 
+def _memory(a) -> int:
+    """The matrix memory with exponential gates: --nh heads of --hd values over --state rows of state; --batch requests of --qlen
+    tokens each.  Portions: gates, the recurrence with every number of columns per group of lanes, division and norm; single
+    tokens (--qlen 1) also the one kernel that does all of it; and two norms of rows of --K in one pass.  Per kernel:
+    microseconds (events, L2 flushed) and the bytes it must move over that time."""
+    H, P, N, B, q = a.nh, a.hd, a.state, a.batch, a.qlen
+    T, inner, n = B * q, a.nh * a.hd, 2 * a.nh * a.state + a.nh * a.hd
+    ctx = _rows_ctx(B, q)
+    flush = _flush()
+    gen = lambda *s: torch.randn(*s, device=DEV)
+    proj, z, bias = gen(T, n + inner).bfloat16(), gen(T, 2 * H), gen(2 * H)
+    m_off = H * (P + 1) * N
+    state = gen(B, -(-(m_off + H) // 4) * 4) * 0.1
+    w = torch.rand(inner, device=DEV) + 0.5
+    gates = k.mlstm_gates(z, bias, 15.0, ctx, state, m_off, H)
+    o, nq = k.mlstm_scan(proj, gates, ctx, state, H, N, P)
+    x, res, w1, w2 = gen(T, a.K).bfloat16(), gen(T, a.K), torch.rand(a.K, device=DEV), torch.rand(a.K, device=DEV)
+    moved = 2 * B * m_off * 4
+    rows = [("gates", lambda: k.mlstm_gates(z, bias, 15.0, ctx, state, m_off, H), T * H * (8 + 16))]
+    for ln, cpt in ((0, 0),) + tuple((ln, c) for ln in ((8, 16) if N <= 64 else (16,) if N <= 128 else (32,)) for c in (1, 2, 4) if 4 * c <= ln):
+        rows.append((f"scan lanes={ln} cpt={cpt}", lambda ln=ln, cpt=cpt: k.mlstm_scan(proj, gates, ctx, state, H, N, P, ln, cpt, chunks=False),
+                     moved + T * (n * 2 + H * 8 + (inner + H) * 4)))
+    if q > 1:
+        rows += [(f"chunks columns={c}", lambda c=c: k.mlstm_scan(proj, gates, ctx, state, H, N, P, chunks=True, columns=c), rows[-1][2])
+                 for c in ((0, 32, 16) if N in (64, 128) else (0,))]
+    rows.append(("head_norm_gate", lambda: k.head_norm_gate(o, proj[:, n:], w, 1e-6, H, P, torch.bfloat16, divisor=(nq, gates)), T * inner * (4 + 2 + 2)))
+    if q == 1:
+        rows.append(("step", lambda: k.mlstm_step(proj, z, bias, 15.0, ctx, state, H, N, P, w, 1e-6, torch.bfloat16),
+                     moved + T * ((n + inner) * 2 + inner * 2)))
+    rows.append((f"two norms width={a.K}", lambda: k.add_rmsnorm(x, res, w1, 1e-6, torch.float32, torch.bfloat16, weight2=w2), T * a.K * (2 + 4 + 4 + 2 + 2)))
+    for name, fn, nbytes in rows:
+        if not name.startswith(a.only):
+            continue
+        us = _time_events(fn, a.replays, flush)
+        print(f"memory {name} B={B} qlen={q} heads={H} vdim={P} state={N}: {us:.1f} us, {nbytes / 1e6:.1f} MB, {nbytes / us / 1e3:.0f} GB/s")
+    print("status", ctx.status.tolist())
+    return 0
+
+
+def _experts(a) -> int:
+    """Grouped products of 16 experts of hidden size --N over inputs of --K for --M tokens, 2 experts each: experts without a gate
+    beside gated ones (whose up product is twice as wide), the down product, and a shared expert without a gate.  Per kernel:
+    microseconds (events, L2 flushed), TFLOP/s, and the weights' bytes (of at most 2 M experts) over that time."""
+    T, ff, K, E, top = a.M, a.N, a.K, 16, 2
+    flush = _flush()
+    k.set_status_word(torch.device(DEV), torch.zeros(4, dtype=torch.int32, device=DEV))
+    gen = lambda *s: torch.randn(*s, device=DEV).bfloat16()
+    x, up, gu, down, shared = gen(T, K), gen(E * ff, K) * 0.02, gen(2 * E * ff, K) * 0.02, gen(E * K, ff) * 0.02, gen(ff, K) * 0.02
+    w, chosen = k.moe_route(torch.randn(T, E, device=DEV), top, want_chosen=True, scores="sigmoid")
+    plan, gate = k.moe_sort(chosen, w), torch.randn(T, 1, device=DEV)
+    y = k.moe_grouped_up(x, plan, up, E, ff, "gelu", weigh_input=True)
+    pairs = k.moe_grouped_down(y, plan, down, E, ff, stacked=True, tokens=T)
+    rest = gen(T, K)
+    used = min(E, top * T)
+    block = k.MOE_BLOCK if ff % k.MOE_BLOCK == 0 else 0
+    rows = [("route", lambda: k.moe_route(torch.empty(T, E, device=DEV), top, want_chosen=True, scores="sigmoid"), 0, T * E * 8),
+            ("sort", lambda: k.moe_sort(chosen, w), 0, T * top * 4),
+            ("grouped up, gelu", lambda: k.moe_grouped_up(x, plan, up, E, ff, "gelu", weigh_input=True), 2.0 * T * top * ff * K, used * ff * K * 2),
+            ("grouped gate/up, clamped", lambda: k.moe_grouped_gate_up(x, plan, gu, E, ff, 7.0, block), 4.0 * T * top * ff * K, used * 2 * ff * K * 2),
+            ("grouped down", lambda: k.moe_grouped_down(y, plan, down, E, ff, stacked=True, tokens=T), 2.0 * T * top * ff * K, used * ff * K * 2),
+            ("combine", lambda: k.moe_combine(pairs, plan, rest, T, top, torch.bfloat16), 0, T * K * (4 * top + 4)),
+            ("shared up, gelu and gate", lambda: k.plain_up(x, shared, "gelu", gate), 2.0 * T * ff * K, ff * K * 2),
+            ("library's product of that size", lambda: torch.mm(x, shared.t()), 2.0 * T * ff * K, ff * K * 2)]
+    for name, fn, flops, nbytes in rows:
+        if not name.startswith(a.only):
+            continue
+        us = _time_events(fn, a.replays, flush)
+        print(f"experts {name} tokens={T} ff={ff} width={K}: {us:.1f} us, {flops / us / 1e6:.0f} TFLOP/s, {nbytes / us / 1e3:.0f} GB/s of weights")
+    return 0
+
+
 def _attn_masked(a) -> int:
     """The tiled two-term attention kernel over bfloat16 pages with a sliding window (keys and values apart) and with
     runs of positions, one more term in the denominator and values that are read from a second plane, at equal sizes;
@@ -270,7 +343,7 @@ def _attn_mixed(a) -> int:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
-    ap.add_argument("--kernel", required=True, choices=["attn_decode", "attn_prefill", "gemv", "gemm", "sample", "recurrence", "channel", "attn_masked", "attn_mixed"])
+    ap.add_argument("--kernel", required=True, choices=["attn_decode", "attn_prefill", "gemv", "gemm", "sample", "recurrence", "channel", "memory", "experts", "attn_masked", "attn_mixed"])
     ap.add_argument("--simple", action="store_true", help="attn_mixed: time the kernel of one warp per token, head and value head too")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--ctx", type=int, default=8192, help="tokens already in the cache")
@@ -297,6 +370,10 @@ def main(argv=None) -> int:
         return _recurrence(a)
     if a.kernel == "channel":
         return _channel(a)
+    if a.kernel == "memory":
+        return _memory(a)
+    if a.kernel == "experts":
+        return _experts(a)
     if a.kernel == "attn_masked":
         return _attn_masked(a)
     if a.kernel == "attn_mixed":

@@ -736,7 +736,7 @@ def logit_cap(x, scale, cap):
 # ----------------------------------------------------------------------------- the matrix memory with exponential gates
 def mlstm_gates(z, bias, cap, ctx, state, m_off, H):
     """z[T, input gates (H) | forget gates (H)] -> [T, H, 4]: what the state is kept by, what the new key and value are put in by,
-    exp(-m), nothing; the running maxima in the slots move on."""
+    exp(-m), the logarithm of the first; the running maxima in the slots move on."""
     T = z.shape[0]
     out = torch.zeros(T, H, 4, dtype=torch.float32)
     g = cap * torch.tanh((z.to(F64) + bias.to(F64)) / cap)
@@ -750,6 +750,7 @@ def mlstm_gates(z, bias, cap, ctx, state, m_off, H):
         for t in range(a, e):
             new = torch.maximum(f[t] + m, i[t])
             out[t, :, 0], out[t, :, 1], out[t, :, 2] = torch.exp(f[t] + m - new), torch.exp(i[t] - new), torch.exp(-new)
+            out[t, :, 3] = f[t] + m - new
             m = new
         state[slot, m_off:m_off + H] = m.to(torch.float32)
     return out

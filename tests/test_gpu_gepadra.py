@@ -393,7 +393,7 @@ def test_gates_kernel(lens, H, cap):
     s2 = st.cuda()
     want = plain_ops.mlstm_gates(z[:, :2 * H], bias, cap, c, st, 8, H)
     got = k.mlstm_gates(z.cuda()[:, :2 * H], bias.cuda(), cap, dev, s2, 8, H)
-    assert (got.cpu()[:, :, :2] - want[:, :, :2]).abs().max() < 1e-5 and (got.cpu() / want)[:, :, 2].sub(1).abs().max() < 2e-5
+    assert (got.cpu()[:, :, [0, 1, 3]] - want[:, :, [0, 1, 3]]).abs().max() < 2e-5 and (got.cpu() / want)[:, :, 2].sub(1).abs().max() < 2e-5
     assert (s2.cpu() - st).abs().max() < 2e-5
     dev.row_slot[0] = -1
     before = s2.clone()
@@ -438,6 +438,37 @@ def test_memory_kernels(H, D, Dv, lens):
         k.mlstm_scan(proj.cuda(), gates.cuda(), dev, s2, H, D, Dv)
         k.mlstm_step(proj.cuda()[:, :n], z.cuda(), bias.cuda(), 5.0, dev, s2, H, D, Dv, w.cuda(), 1e-6, torch.bfloat16) if max(lens) == 1 else None
         assert torch.equal(s2[c.row_slot[0]].cpu(), st[c.row_slot[0]]) and int(dev.status[0]) == 0
+
+
+@pytest.mark.parametrize("H,D,Dv", [(3, 64, 64), (2, 32, 40), (2, 96, 24), (2, 128, 128), (1, 128, 8), (2, 64, 72)])
+@pytest.mark.parametrize("lens", [[1, 64, 63], [65, 1, 200, 2], [300], [129, 1]], ids=str)
+@pytest.mark.parametrize("gates", ["spread", "sharp"])
+def test_memory_in_runs_as_matrix_products(H, D, Dv, lens, gates):
+    """Runs of 64 tokens, whole and broken off, from slots that hold a state; gates near one, and gates that close and open so
+    that a run's weights span the whole range of an exponential.  Against the walk token by token."""
+    from fastmlx_b200 import kernels as k
+    g = torch.Generator().manual_seed(D + sum(lens))
+    T, slots = sum(lens), [2, 0, 3, 1][:len(lens)]
+    c, dev = _ctx(lens, slots)
+    proj = torch.randn(T, 2 * H * D + H * Dv + 8, generator=g).bfloat16()
+    m_off = H * (Dv + 1) * D
+    st = torch.randn(5, -(-(m_off + H) // 4) * 4, generator=g) * 0.5
+    z = torch.randn(T, 2 * H, generator=g) * (2 if gates == "spread" else 20) + torch.tensor([0.0] * H + [3.0 if gates == "spread" else 8.0] * H)
+    gt = plain_ops.mlstm_gates(z, torch.zeros(2 * H), 15.0, c, st.clone(), m_off, H)
+    s1 = st.clone()
+    o1, nq1 = plain_ops.mlstm_scan(proj, gt, c, s1, H, D, Dv)
+    assert k.can_mlstm_chunks(proj.cuda(), st.cuda(), D, Dv)
+    for columns in (0, 32, 16) if D in (64, 128) else (0, 32):
+        s2 = st.cuda()
+        o2, nq2 = k.mlstm_scan(proj.cuda(), gt.cuda(), dev, s2, H, D, Dv, chunks=True, columns=columns)
+        err = (o1 - o2.cpu()).reshape(T, H, Dv).abs().amax(-1) / o1.reshape(T, H, Dv).abs().amax(-1).clamp(min=0.05 * float(o1.abs().max()))
+        assert err.max() < 1e-4, (columns, float(err.max()), int(err.argmax()))
+        assert (nq1 - nq2.cpu()).abs().max() < 1e-5 * nq1.abs().max().clamp(min=1)
+        assert (s1 - s2.cpu()).abs().max() < 3e-5 * s1.abs().max()
+    dev.row_slot[0] = -1
+    s2 = st.cuda()
+    k.mlstm_scan(proj.cuda(), gt.cuda(), dev, s2, H, D, Dv, chunks=True)
+    assert torch.equal(s2[c.row_slot[0]].cpu(), st[c.row_slot[0]])
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])

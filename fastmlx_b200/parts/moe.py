@@ -251,7 +251,9 @@ class PlainRoutedExperts(FeedForward):
             rows.append(to_compute(tensors[self.gate_name], rt).reshape(1, self.width))
         if len({r.dtype for r in rows}) > 1:
             rows = [r.float() for r in rows]
-        self.router = torch.cat(rows, 0).contiguous()             # [E (+1), width]: the experts' logits, then the shared gate's
+        pad = -sum(r.shape[0] for r in rows) % 8                  # rows of zeros, so that a token's row of logits fills whole 16-byte pieces
+        rows.append(torch.zeros((pad, self.width), dtype=rows[0].dtype, device=rows[0].device))
+        self.router = torch.cat(rows, 0).contiguous()             # [E (+1) (+ zeros), width]: the experts' logits, then the shared gate's
         self.correction = to_f32_vector(tensors[self.correction_name], rt) if self.correction_name else None
         ups = [to_compute(tensors[n], rt) for n, _ in self.up_names]
         downs = [to_compute(tensors[n], rt) for n, _ in self.down_names]
@@ -294,7 +296,7 @@ class PlainRoutedExperts(FeedForward):
         more = {} if self.scores == "softmax" else dict(scores=self.scores)
         w = k.moe_route(z, self.top, experts=self.E, correction=self.correction, scale=self.scale, want_chosen=want_chosen, **more)
         w, chosen = w if want_chosen else (w, None)
-        return w, chosen, z[:, self.E:] if self.gate_name else None
+        return w, chosen, z[:, self.E:self.E + 1] if self.gate_name else None
 
     def forward_inner(self, x, ctx, out=None):
         """Without grouped products: the hidden layers side by side after weight and activation, [T, F], into `out` where one

@@ -122,6 +122,20 @@ def test_replay(models, name, dtype, cut):
         assert len(prompts) > rp.manager.max_requests, "too many slots for one to be used again"
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("seed", range(6))
+def test_replay_of_drawn_configurations(tmp_path, seed, dtype):
+    cfg = tg.drawn(100 + seed)
+    d = tg.make_model_dir(tmp_path, cfg, seed, tg.lively_tensors(cfg, seed, settled=dtype == "bfloat16"))
+    W = tiny.load_plain_weights(d)
+    prompts = {f"r{i}": tiny.rand_tokens(n, cfg["vocab"], 40 * seed + i) for i, n in enumerate([97, 3, 150, 41])}
+    both = {r: _unsure(cfg, W, t) for r, t in prompts.items()}
+    for cut in ("whole", "mixed"):
+        steps = CUTS[cut](prompts)
+        outs, _ = _run(d, dtype, steps, 384, 16)
+        _compare(steps, outs, prompts, {r: b[0] for r, b in both.items()}, TOL[dtype], {r: b[1] for r, b in both.items()} if dtype == "bfloat16" else None)
+
+
 @pytest.mark.parametrize("name", ["G1", "G4"])
 def test_cuts_agree_in_32_bit(models, name):
     """The logits at a place do not depend on the cut, the batch, the pages or the slot beyond the order of 32-bit

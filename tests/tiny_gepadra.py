@@ -60,6 +60,35 @@ DENSE = config(89, 64, [layer(memory(2, 16, 24, 7.0), dense(96, 1.1)), layer(att
                         layer(memory(4, 16, 32, 3.0)), layer(attention(6, 3, 16, 16, 0.25, (30, 17), (8, 40.0), True), dense(64, 0.7))])
 
 
+def drawn(seed):
+    """A configuration drawn from a seed: any order of layers, sizes that the tiled kernels take and sizes that they do not."""
+    import random
+    r = random.Random(seed)
+    kv, vdim = r.choice([1, 2, 3]), r.choice([16, 24, 32, 48])
+
+    def att(mix):
+        g, dv = (kv, vdim) if mix else (r.choice([1, 2]), r.choice([8, 16, 20, 64]))
+        dim = r.choice([16, 32, 48, 20, 64])
+        mask = (r.choice([1, 13, 16, 40, 64]), r.choice([0, 1, 4, 16, 19, 50])) if r.random() < 0.8 else None
+        rot = (r.choice([2, 8, dim]), r.choice([20.0, 1000.0, 1e6])) if r.random() < 0.8 else None
+        return attention(g * r.choice([1, 2, 4]), g, dim, dv, r.uniform(0.5, 1.5) * dim ** -0.5, mask, rot, mix)
+
+    def mem():
+        return memory(r.choice([1, 2, 3, 6]), r.choice([8, 12, 32, 64, 96, 128, 10]), r.choice([8, 16, 24, 32, 64, 7]), r.uniform(1.0, 16.0))
+
+    def mlp():
+        kind = r.random()
+        if kind < 0.2:
+            return None
+        if kind < 0.5:
+            return dense(r.choice([48, 128, 256, 72]), r.uniform(0.3, 4.0))
+        experts = r.choice([1, 4, 8, 12])
+        return moe(experts, r.randint(1, experts), r.choice([16, 24, 64, 30]), r.choice([None, 32, 40, 128]))
+
+    layers = [layer(att(r.random() < 0.7) if r.random() < 0.5 else mem(), mlp()) for _ in range(r.randint(2, 6))]
+    return config(r.choice([61, 128, 200]), r.choice([64, 96, 128, 72]), layers, eps=r.choice([1e-6, 1e-5, 1e-4]))
+
+
 def one_layer(mixer, width=48, vocab=61, mlp=None, eps=1e-6):
     return config(vocab, width, [layer(mixer, mlp)], eps=eps)
 

@@ -257,8 +257,8 @@ def _experts(a) -> int:
 
 def _attn_masked(a) -> int:
     """The tiled two-term attention kernel over bfloat16 pages with a sliding window (keys and values apart) and with
-    runs of positions, one more term in the denominator and values that are read from a second plane, at equal sizes;
-    then over pages of keys that are the values too (a latent of --hd values per token), with a learned term or none."""
+    runs of positions, one more term in the denominator and values that are read from a second plane, at equal sizes; with a
+    window beside kept first tokens and a learned term; then over pages of keys that are the values too (a latent of --hd values per token), with a learned term or none."""
     B, q, c, nh, nkv, hd, ps, span = a.batch, a.qlen, a.ctx if a.ctx != 8192 or a.qlen == 1 else 0, a.nh, a.nkv, a.hd, a.page, a.span
     ctx = _rows_ctx(B, q, c)
     per = -(-(c + q) // ps)
@@ -274,6 +274,8 @@ def _attn_masked(a) -> int:
     cases = [("window", lambda: k.paged_attention_wide(qq, kv, ctx, grp, nh, nkv, hd, hd ** -0.5, 30.0, span), seen, kvb(span + q)),
              ("runs of positions, one more term", lambda: k.paged_attention_wide(qq, kv, ctx, grp, nh, nkv, hd, hd ** -0.5, 30.0, 0, chunk=span, sinks=sinks0),
               seen_c, kvb((c + q - 1) % span + 1 if q == 1 else span))]
+    cases.append(("window, kept tokens, a learned term", lambda: k.paged_attention_wide(qq, kv, ctx, grp, nh, nkv, hd, hd ** -0.5, 0.0, span,
+                                                                                        keep_first=8, sinks=sinks), seen, kvb(span + q)))
     if hd <= 128:                                   # values twice as wide as keys: another library of the same kernel
         kv2 = torch.randn(B * per + 8, nkv * ps * 3 * hd, device=DEV).bfloat16()
         cases.append(("window, values twice as wide", lambda: k.paged_attention_wide(qq, kv2, ctx, grp, nh, nkv, hd, hd ** -0.5, 0.0, span, vd=2 * hd),

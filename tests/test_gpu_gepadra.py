@@ -656,7 +656,7 @@ def test_replay_with_grouped_experts(models, monkeypatch, cut):
     _compare(steps, outs, prompts, ref, TOL["bfloat16"], skip)
 
 
-@pytest.mark.parametrize("hd,vd,nh,nkv", [(64, 32, 8, 2), (32, 48, 4, 1), (64, 64, 16, 1), (96, 32, 3, 3), (16, 16, 24, 1), (128, 128, 6, 2)])
+@pytest.mark.parametrize("hd,vd,nh,nkv", [(64, 32, 8, 2), (32, 48, 4, 1), (64, 64, 16, 1), (80, 48, 3, 3), (16, 16, 24, 1), (128, 128, 6, 2)])
 @pytest.mark.parametrize("window,keep", [(0, 0), (45, 0), (45, 20), (16, 33)])
 def test_tiled_attention_with_sinks_kept_tokens_and_values_of_another_width(hd, vd, nh, nkv, window, keep):
     from fastmlx_b200 import kernels as k

@@ -56,6 +56,7 @@ struct Grouped {
   int act, pre;
   const float* row_gate;
   long long row_gate_stride;
+  int expert_cols;               // the experts' matrices side by side instead: expert e's K columns start e * expert_cols columns in
 };
 
 template <int BN> struct Cfg {
@@ -132,8 +133,12 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     bool ok = true;
     for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x) {
       const int m0 = (t % tiles_m) * BM;
-      int n0 = (t / tiles_m) * BN;
-      if (gr.tile_expert != nullptr) n0 += max(0, gr.tile_expert[m0 / BM]) * gr.expert_rows;      // this tile's expert's rows of W
+      int n0 = (t / tiles_m) * BN, k0 = 0;
+      if (gr.tile_expert != nullptr) {             // this tile's expert's rows, or columns, of W
+        const int e = max(0, gr.tile_expert[m0 / BM]);
+        n0 += e * gr.expert_rows;
+        k0 = e * gr.expert_cols;                   // (behind an expert's columns A is zero: what W holds there does not count)
+      }
       for (int kb = 0; kb < k_blocks; ++kb) {
 #ifdef FMX_SKIP_LAST_STAGE
         if (kb == k_blocks - 1 && t + (int)gridDim.x >= n_tiles) break;      // the test build: never bring the last block
@@ -143,7 +148,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
         unsigned char* sa = smem + (size_t)stage * cfg::STAGE_BYTES;
         mbar_expect_tx(fb, cfg::STAGE_BYTES);
         tma_load_2d(smem_u32(sa), &map_a, kb * BK, m0, fb);
-        tma_load_2d(smem_u32(sa + cfg::A_BYTES), &map_w, kb * BK, n0, fb);
+        tma_load_2d(smem_u32(sa + cfg::A_BYTES), &map_w, k0 + kb * BK, n0, fb);
         ++issued;
         if (++stage == cfg::STAGES) { stage = 0; phase ^= 1; }
       }
@@ -309,10 +314,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 
 template <int BN, int EPI>
 int run(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc, const void* residual,
-        long long ldr, int M, int N, int K, int sms, int* status, cudaStream_t stream, Grouped gr = Grouped{}, long long w_rows = 0) {
+        long long ldr, int M, int N, int K, int sms, int* status, cudaStream_t stream, Grouped gr = Grouped{}, long long w_rows = 0, int w_cols = 0) {
   using cfg = Cfg<BN>;
   CUtensorMap map_a, map_w;
-  if (make_map_k128(&map_a, A, M, K, lda, BM) || make_map_k128(&map_w, W, w_rows > 0 ? w_rows : N, K, ldw, BN)) return 1;
+  if (make_map_k128(&map_a, A, M, K, lda, BM) || make_map_k128(&map_w, W, w_rows > 0 ? w_rows : N, w_cols > 0 ? w_cols : K, ldw, BN)) return 1;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_kernel<BN, EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -339,7 +344,7 @@ FMX_EXPORT int fmx_expert_tcgen05(const void* A, long long lda, const void* W, l
   if (K % 8 || lda % 8 || ldw % 8 || ((uintptr_t)A & 15) || ((uintptr_t)W & 15))
     return fmx_fail("fmx_expert_tcgen05: rows must start on 16-byte boundaries (K=%d lda=%lld ldw=%lld)", K, lda, ldw);
   if (sms <= 0) sms = fmx_num_sms();
-  const Grouped gr{nullptr, nullptr, nullptr, nullptr, 0, limit, 0, 0, nullptr, 0};
+  const Grouped gr{nullptr, nullptr, nullptr, nullptr, 0, limit, 0, 0, nullptr, 0, 0};
   return run<256, EPI_EXPERT>(A, lda, W, ldw, C, ldc, nullptr, 0, M, N, K, sms, status, stream, gr, 0);
 }
 
@@ -360,7 +365,7 @@ FMX_EXPORT int fmx_grouped_tcgen05(const void* A, long long lda, const void* W, 
   if (used_rows == nullptr || tile_expert == nullptr || row_token == nullptr || (gated && row_weight == nullptr))
     return fmx_fail("fmx_grouped_tcgen05: the sorted pairs' arrays are missing");
   if (sms <= 0) sms = fmx_num_sms();
-  const Grouped gr{used_rows, tile_expert, row_token, row_weight, N, limit, 0, 0, nullptr, 0};
+  const Grouped gr{used_rows, tile_expert, row_token, row_weight, N, limit, 0, 0, nullptr, 0, 0};
   if (gated)
     return run<256, EPI_EXPERT>(A, lda, W, ldw, C, ldc, nullptr, 0, max_rows, N, K, sms, status, stream, gr, (long long)experts * N);
   return run<256, EPI_F32>(A, lda, W, ldw, C, ldc, nullptr, 0, max_rows, N, K, sms, status, stream, gr, (long long)experts * N);
@@ -379,8 +384,25 @@ FMX_EXPORT int fmx_grouped_act_tcgen05(const void* A, long long lda, const void*
   if (used_rows == nullptr || tile_expert == nullptr || row_token == nullptr || row_weight == nullptr)
     return fmx_fail("fmx_grouped_act_tcgen05: the sorted pairs' arrays are missing");
   if (sms <= 0) sms = fmx_num_sms();
-  const Grouped gr{used_rows, tile_expert, row_token, row_weight, N, 0.f, act, pre, nullptr, 0};
+  const Grouped gr{used_rows, tile_expert, row_token, row_weight, N, 0.f, act, pre, nullptr, 0, 0};
   return run<256, EPI_ACT>(A, lda, W, ldw, C, ldc, nullptr, 0, max_rows, N, K, sms, status, stream, gr, (long long)experts * N);
+}
+
+// The down product of grouped pairs over the experts' matrices side by side: W [N, experts * K] with rows of ldw, expert e's K columns
+// start e * K columns in (K a multiple of 8, so that they start on 16 bytes); C 32-bit [max_rows, N].
+FMX_EXPORT int fmx_grouped_down_tcgen05(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc, int max_rows,
+                                        int N, int K, int experts, const int* used_rows, const int* tile_expert, const int* row_token,
+                                        int sms, int* status, cudaStream_t stream) {
+  if (max_rows == 0 || N == 0) return 0;
+  if (max_rows < 0 || max_rows % BM || N <= 0 || K <= 0 || experts <= 0 || (long long)experts * K > ldw)
+    return fmx_fail("fmx_grouped_down_tcgen05: bad sizes rows=%d N=%d K=%d experts=%d", max_rows, N, K, experts);
+  if (K % 8 || lda % 8 || ldw % 8 || ((uintptr_t)A & 15) || ((uintptr_t)W & 15))
+    return fmx_fail("fmx_grouped_down_tcgen05: rows must start on 16-byte boundaries (K=%d lda=%lld ldw=%lld)", K, lda, ldw);
+  if (used_rows == nullptr || tile_expert == nullptr || row_token == nullptr)
+    return fmx_fail("fmx_grouped_down_tcgen05: the sorted pairs' arrays are missing");
+  if (sms <= 0) sms = fmx_num_sms();
+  const Grouped gr{used_rows, tile_expert, row_token, nullptr, 0, 0.f, 0, 0, nullptr, 0, K};
+  return run<256, EPI_F32>(A, lda, W, ldw, C, ldc, nullptr, 0, max_rows, N, K, sms, status, stream, gr, N, experts * K);
 }
 
 // One expert without a gate for every row: C bfloat16 [M, N] = act(A W^T), times sigmoid(row_gate[row * row_gate_stride]) where given.
@@ -392,7 +414,7 @@ FMX_EXPORT int fmx_act_tcgen05(const void* A, long long lda, const void* W, long
   if (K % 8 || lda % 8 || ldw % 8 || ((uintptr_t)A & 15) || ((uintptr_t)W & 15))
     return fmx_fail("fmx_act_tcgen05: rows must start on 16-byte boundaries (K=%d lda=%lld ldw=%lld)", K, lda, ldw);
   if (sms <= 0) sms = fmx_num_sms();
-  const Grouped gr{nullptr, nullptr, nullptr, nullptr, 0, 0.f, act, 0, row_gate, row_gate_stride};
+  const Grouped gr{nullptr, nullptr, nullptr, nullptr, 0, 0.f, act, 0, row_gate, row_gate_stride, 0};
   return run<256, EPI_ACT>(A, lda, W, ldw, C, ldc, nullptr, 0, M, N, K, sms, status, stream, gr, 0);
 }
 

@@ -1204,11 +1204,11 @@ def moe_grouped_up(x, plan, up, E: int, ff: int, act: str, weigh_input: bool = F
 
 
 def moe_grouped_down(y, plan, down, E: int, ff: int, stacked: bool = False, tokens: int = 0, status=None) -> torch.Tensor:
-    """The pairs' outputs.  down bfloat16: [d, E ff], the experts' down matrices side by side, or with `stacked`
-    [E d, ff], one under the other.  -> 32-bit [tiles * MOE_TILE_ROWS, d] (padding rows are not written).  `tokens`:
-    the step's tokens (stacked matrices and MOE_TC_MIN_TOKENS of them: the tcgen05 kernel)."""
+    """The pairs' outputs.  down bfloat16: [d, E ff], the experts' down matrices side by side (rows may be a slice of wider
+    ones), or with `stacked` [E d, ff], one under the other.  -> 32-bit [tiles * MOE_TILE_ROWS, d] (padding rows are not written).  `tokens`:
+    the step's tokens (from MOE_TC_MIN_TOKENS on the tcgen05 kernel)."""
     sorted_token, _, _, tile_expert, tiles, used = plan
-    assert down.dtype == torch.bfloat16 and down.is_contiguous() and y.is_contiguous()
+    assert down.dtype == torch.bfloat16 and down.stride(1) == 1 and (down.is_contiguous() or not stacked) and y.is_contiguous()
     d = down.shape[0] // E if stacked else down.shape[0]
     assert down.shape == ((E * d, ff) if stacked else (d, E * ff))
     rows = tiles * MOE_TILE_ROWS
@@ -1218,7 +1218,12 @@ def moe_grouped_down(y, plan, down, E: int, ff: int, stacked: bool = False, toke
              used.data_ptr(), tile_expert.data_ptr(), sorted_token.data_ptr(), None, 0.0, 0, num_sms(y.device),
              _ptr(status if status is not None else _status_word(y.device)), _stream())
         return out
-    ldw, stride = (ff, d * ff) if stacked else (E * ff, ff)
+    if not stacked and tokens >= MOE_TC_MIN_TOKENS and ff % 8 == 0 and down.stride(0) % 8 == 0 and down.data_ptr() % 16 == 0:
+        call("tc", "fmx_grouped_down_tcgen05", y.data_ptr(), ff, down.data_ptr(), down.stride(0), out.data_ptr(), d, rows, d, ff, E,
+             used.data_ptr(), tile_expert.data_ptr(), sorted_token.data_ptr(), num_sms(y.device),
+             _ptr(status if status is not None else _status_word(y.device)), _stream())
+        return out
+    ldw, stride = (ff, d * ff) if stacked else (down.stride(0), ff)
     call("bf16", "fmx_moe_grouped_down", y.data_ptr(), sorted_token.data_ptr(), tile_expert.data_ptr(), down.data_ptr(), ldw, stride,
          out.data_ptr(), tiles, d, ff, int(tokens), _stream())
     return out

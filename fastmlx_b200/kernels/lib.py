@@ -89,6 +89,7 @@ _SIGNATURES = {
     "tc": {
         "fmx_gemm_tcgen05": [_P, _L, _P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _P, _P],
         "fmx_grouped_act_tcgen05": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _P, _I, _I, _I, _P, _P],
+        "fmx_grouped_down_tcgen05": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P],
         "fmx_act_tcgen05": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _P, _L, _I, _P, _P],
         "fmx_expert_tcgen05": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _F, _I, _P, _P],
         "fmx_grouped_tcgen05": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _P, _F, _I, _I, _P, _P],

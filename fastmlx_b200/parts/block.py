@@ -66,25 +66,27 @@ class ParallelBlock(Part):
     into one product over [mixer's heads | feed-forward's hidden layer], so that the two
     sublayers' outputs are added inside the product's 32-bit accumulators, and the block's
     output is rounded once before the 32-bit residual sum takes it.  `ffn` may be None.  A feed-forward of several output
-    matrices names them as `out_pieces`; one that multiplies with some of them itself (`kept_pieces`, known once it is bound)
-    hands on what it needs for that from `forward_inner` and adds its own outputs to the block's in `add_kept`."""
+    matrices names them as `out_pieces`; they stand in front of the mixer's.  It may multiply with the first of them itself in
+    steps that it chooses by their size: `skips(tokens)` says how many leading columns the joined product then leaves out,
+    `forward_inner` hands on what `add_kept` adds to the block's output, and `bind_joined` shows it the joined matrix."""
 
     def __init__(self, mixer: Mixer, ffn: FeedForward | None, norm: Norm, width: int, norm2: Norm | None = None):
         self.mixer, self.ffn, self.norm, self.norm2 = mixer, ffn, norm, norm2
+        self.several = hasattr(ffn, "out_pieces")
         pieces = [mixer.out_piece]
-        if ffn is not None:
-            pieces += ffn.out_pieces if hasattr(ffn, "out_pieces") else [ffn.out_piece]
+        if self.several:
+            pieces = list(ffn.out_pieces) + pieces
+        elif ffn is not None:
+            pieces.append(ffn.out_piece)
         self.out = JoinedLinear(width, pieces)
 
     def children(self):
         return tuple(p for p in (self.norm, self.norm2, self.mixer, self.ffn, self.out) if p is not None)
 
     def bind(self, tensors, rt):
-        self.rt = rt
-        for c in self.children():
-            if c is self.out:                     # the last one: the feed-forward is bound
-                c.leave_out(getattr(self.ffn, "kept_pieces", ()))
-            c.bind(tensors, rt)
+        super().bind(tensors, rt)
+        if self.several:
+            self.ffn.bind_joined(self.out.weight)
 
     def cache_spec(self):
         return self.mixer.cache_spec()
@@ -103,14 +105,19 @@ class ParallelBlock(Part):
         else:
             h, residual = self.norm.forward(delta, residual)
             h2 = h
-        joined = torch.empty((h.shape[0], self.out.in_features), dtype=self.rt.dtype, device=h.device)
+        skip = self.ffn.skips(h.shape[0]) if self.several else 0
+        joined = torch.empty((h.shape[0], self.out.in_features - skip), dtype=self.rt.dtype, device=h.device)
         m = self.mixer.inner_features
+        if self.several:
+            f = joined.shape[1] - m
+            self.mixer.forward_inner(h, ctx, cache, out=joined[:, f:])
+            kept = self.ffn.forward_inner(h2, ctx, out=joined[:, :f])
+            y = self.out.forward(joined, skip=skip)
+            return (self.ffn.add_kept(y, kept) if skip else y), residual
         self.mixer.forward_inner(h, ctx, cache, out=joined[:, :m] if self.ffn is not None else joined)
-        if self.ffn is None:
-            return self.out.forward(joined), residual
-        kept = self.ffn.forward_inner(h2, ctx, out=joined[:, m:])
-        y = self.out.forward(joined)
-        return (self.ffn.add_kept(y, kept) if getattr(self.ffn, "kept_pieces", ()) else y), residual
+        if self.ffn is not None:
+            self.ffn.forward_inner(h2, ctx, out=joined[:, m:])
+        return self.out.forward(joined), residual
 
 
 class SandwichBlock(Part):

@@ -79,26 +79,18 @@ class JoinedLinear(Part):
     def __init__(self, out_features: int, pieces, bias_scales=None):
         self.out_features = int(out_features)
         self.bias_scales = [1.0] * len(pieces) if bias_scales is None else [float(s) for s in bias_scales]
-        self.all_pieces = [(w, int(k), b) for w, k, b in pieces]
-        self.weight = None
-        self.bias = None
-        self.leave_out(())
-
-    def leave_out(self, names) -> None:
-        """The pieces whose weight tensors are named here do not join the product (their part multiplies with them in
-        another way); said before the product is bound."""
-        keep = [i for i, (w, _, _) in enumerate(self.all_pieces) if w not in set(names)]
-        self.pieces = [self.all_pieces[i] for i in keep]
-        self.scales = [self.bias_scales[i] for i in keep]
+        self.pieces = [(w, int(k), b) for w, k, b in pieces]
         self.offsets, at = [], 0
         for _, k, _ in self.pieces:
             self.offsets.append(at)
             at += k
         self.in_features = at
+        self.weight = None
+        self.bias = None
 
     def own_weight_specs(self):
-        specs = [WeightSpec(w, (self.out_features, k), "matrix") for w, k, _ in self.all_pieces]
-        specs += [WeightSpec(b, (self.out_features,), "bias") for _, _, b in self.all_pieces if b is not None]
+        specs = [WeightSpec(w, (self.out_features, k), "matrix") for w, k, _ in self.pieces]
+        specs += [WeightSpec(b, (self.out_features,), "bias") for _, _, b in self.pieces if b is not None]
         return specs
 
     def bind_own(self, tensors, rt: Runtime):
@@ -107,7 +99,7 @@ class JoinedLinear(Part):
             ws = [w.float() for w in ws]
         self.weight = ws[0].contiguous() if len(ws) == 1 else torch.cat(ws, dim=1).contiguous()
         bs = [to_f32_vector(tensors[b], rt) * s if s != 1.0 else to_f32_vector(tensors[b], rt)
-              for (_, _, b), s in zip(self.pieces, self.scales) if b is not None]
+              for (_, _, b), s in zip(self.pieces, self.bias_scales) if b is not None]
         self.bias = None
         if bs:
             total = bs[0]
@@ -118,8 +110,10 @@ class JoinedLinear(Part):
     def weight_bytes(self):
         return self.weight.numel() * self.weight.element_size()
 
-    def forward(self, x, out_dtype=None):
-        return self.rt.k.linear(x, self.weight, self.bias, out_dtype or self.rt.dtype)
+    def forward(self, x, out_dtype=None, skip: int = 0):
+        """`skip`: x holds no inputs for the first that many columns, which the product leaves out."""
+        w = self.weight[:, skip:] if skip else self.weight
+        return self.rt.k.linear(x, w, self.bias, out_dtype or self.rt.dtype)
 
 
 class BlockDiagonalLinear(Part):

@@ -180,34 +180,38 @@ class PlainRoutedExperts(FeedForward):
     applied to the hidden values in front of the activation.  A shared expert of the same form and a width of its own
     runs for every token and is added times sigmoid(g . x), one number per token.
 
-    Two ways to compute it, chosen once by size (`sparse`), neither of which loops on the host or makes a token's result
-    depend on what else is in the batch, so that a decode step can be captured:
+    Two ways to compute it, over the same matrices, neither of which loops on the host or makes a token's result depend on what
+    else is in the batch; a step's number of tokens alone chooses (`grouped`), so that a decode step can be captured:
 
-    * all experts side by side (small experts, and the 32-bit path): the up matrices are stacked into one matrix and the down
-      matrices laid side by side; the activation kernel zeroes the columns of experts a token did not choose and weighs the
-      others (the shared columns by the token's gate), and one product with the down matrices gives the sum inside the
-      product's 32-bit accumulators;
+    * all experts side by side (small experts, the 32-bit path, and steps of few tokens that would use most of the experts
+      anyway): the up matrices are stacked into one matrix and the down matrices laid side by side; the activation kernel
+      zeroes the columns of experts a token did not choose and weighs the others (the shared columns by the token's gate), and
+      one product with the down matrices gives the sum inside the product's 32-bit accumulators;
     * grouped products (bfloat16, large experts): the (token, expert) pairs are sorted expert by expert on the device, a
       tiled kernel multiplies each tile of pairs with its expert's up rows and applies weight and activation in its
-      epilogue, a second one multiplies with the expert's down matrix, and a last kernel adds a token's pair outputs to the
-      rest of the layer's output in 32-bit.  Only chosen experts' weights are read.
+      epilogue, a second one multiplies with the expert's columns of the down matrix, and a last kernel adds a token's pair
+      outputs to the rest of the layer's output in 32-bit.  Only chosen experts' weights are read.
 
     The router's matrix and the shared gate's vector are stacked, so that one 32-bit product gives a token's logits and its gate.
-    `output=False` leaves the down projections to the block, which joins them with the mixer's (`out_pieces`): with the
-    experts side by side all of them, with grouped products the shared expert's alone (`kept_pieces` are the others').
+    `output=False` leaves the down projections to the block, which joins them with the mixer's (`out_pieces`, in front of it);
+    where the products are grouped the joined one takes the shared expert's columns and the mixer's alone (`skips`).
 
     Tensors, under `name`: router, correction; e<i>.up, e<i>.down; shared.up, shared.down, shared.sg."""
 
     supports_cuda_graph = True
     SPARSE_MIN_BYTES = 8 << 20
+    # Side by side the whole-K and the library's products stream every expert at about 5 TB/s; grouped, few tokens per expert, the
+    # used ones at about 2.3: fewer tokens than fill the tensor-memory kernel are grouped where they use less than this share.
+    GROUPED_SHARE = 0.45
 
     def __init__(self, width: int, experts: int, top: int, ff: int, name: str, scale: float = 1.0, shared_ff: int = 0,
                  activation: str = "relu2", correction: str | None = "correction", shared_gate: str | None = "sg",
                  weight_suffix: str = "", expert_prefix: str = "e", shared_name: str = "shared", router_name: str = "router",
                  proj_names=("up", "down"), scores: str = "softmax", weigh: str = "output", output: bool = True,
                  sparse: bool | None = None):
-        """`sparse`: grouped products (True), all experts side by side (False), or by size (None): grouped where the
-        experts' matrices together pass SPARSE_MIN_BYTES and more than twice as many experts exist as a token uses."""
+        """`sparse`: grouped products in steps that gain by them (True), all experts side by side always (False), or by size
+        (None): as True where the experts' matrices together pass SPARSE_MIN_BYTES and more than twice as many experts exist as
+        a token uses."""
         if activation not in ("relu2", "gelu", "gelu_tanh", "silu"):
             raise ValueError(f"unknown activation {activation!r}")
         if scores not in ("softmax", "sigmoid") or weigh not in ("output", "input"):
@@ -227,12 +231,7 @@ class PlainRoutedExperts(FeedForward):
         self.correction_name = f"{name}.{correction}" if correction else None
         self.gate_name = f"{name}.{shared_name}.{shared_gate}{weight_suffix}" if self.shared_ff and shared_gate else None
         self.out_pieces = [(n, w, None) for n, w in self.down_names]
-        self.kept_pieces = ()
-
-    @property
-    def inner_features(self) -> int:
-        """Columns of the hidden layer that go through the block's joined product."""
-        return self.shared_ff if self.sparse else self.F
+        self.inner_features = self.F
 
     def own_weight_specs(self):
         specs = [WeightSpec(self.router_name, (self.E, self.width), "matrix")]
@@ -260,34 +259,39 @@ class PlainRoutedExperts(FeedForward):
         if len({m.dtype for m in ups + downs}) > 1:
             ups, downs = [m.float() for m in ups], [m.float() for m in downs]
         can = (rt.dtype == torch.bfloat16 and all(m.dtype == torch.bfloat16 for m in ups + downs) and self.width % 8 == 0
-               and self.ff % 8 == 0 and rt.device.type == "cuda" and hasattr(rt.k, "moe_grouped_up"))
+               and self.ff % 8 == 0 and self.shared_ff % 8 == 0 and rt.device.type == "cuda" and hasattr(rt.k, "moe_grouped_up"))
         big = 2 * self.E * self.ff * self.width * 2 >= self.SPARSE_MIN_BYTES and self.E > 2 * self.top
         self.sparse = can and (big if self.want_sparse is None else bool(self.want_sparse))
-        self.shared_up = self.shared_down = self.down = None
-        self.kept_pieces = ()
-        if self.sparse:
-            if self.shared_ff:
-                self.shared_up = ups.pop().contiguous()
-                shared_down = downs.pop()
-                self.shared_down = shared_down.contiguous() if self.output else None
-            self.kept_pieces = tuple(n for n, _ in self.down_names[:self.E])
-            self.down = torch.cat(downs, 0).contiguous()          # [E width, ff], one under the other
-        elif self.output:
-            self.down = torch.cat(downs, 1).contiguous()          # [width, F]
-        self.up = torch.cat(ups, 0).contiguous()                  # [F, width], or the routed experts' [E ff, width]
+        self.up = torch.cat(ups, 0).contiguous()                  # [F, width]: the routed experts' rows, then the shared one's
+        self.down = torch.cat(downs, 1).contiguous() if self.output else None         # [width, F]
+
+    def bind_joined(self, weight):
+        """The block's joined matrix, whose first F columns are this part's down matrices."""
+        self.down = weight[:, :self.F]
+        if weight.stride(0) % 8 or weight.data_ptr() % 16:
+            self.sparse = False                                   # the grouped kernels read rows of 16-byte pieces
+
+    def used(self, tokens: int) -> float:
+        """The share of the experts that so many tokens use, if every choice is as likely as any other."""
+        return 1.0 - (1.0 - self.top / self.E) ** tokens
+
+    def grouped(self, tokens: int) -> bool:
+        return self.sparse and (tokens >= self.rt.k.MOE_TC_MIN_TOKENS or self.used(tokens) < self.GROUPED_SHARE)
+
+    def skips(self, tokens: int) -> int:
+        return self.E * self.ff if self.grouped(tokens) else 0
 
     def weight_bytes(self):
-        return sum(t.numel() * t.element_size() for t in (self.router, self.up, self.down, self.shared_up, self.shared_down)
-                   if t is not None)
+        """Without the down matrices where the block holds them."""
+        return sum(t.numel() * t.element_size() for t in (self.router, self.up, self.down if self.output else None) if t is not None)
 
     def active_weight_bytes(self, tokens: int) -> int:
-        """Bytes of weights a step of `tokens` tokens reads at most: all with the experts side by side; with grouped
-        products the router, the shared expert's and those of at most tokens * top experts."""
-        if not self.sparse:
+        """`weight_bytes` less what a step of `tokens` tokens does not read: nothing with the experts side by side; with grouped
+        products both matrices (wherever they are held) of all but at most tokens * top routed experts."""
+        if not self.grouped(tokens):
             return self.weight_bytes()
-        used = min(self.E, tokens * self.top)
-        rest = sum(t.numel() * t.element_size() for t in (self.router, self.shared_up, self.shared_down) if t is not None)
-        return rest + self.router.element_size() * 2 * used * self.ff * self.width
+        unused = self.E - min(self.E, tokens * self.top)
+        return self.weight_bytes() - self.router.element_size() * 2 * unused * self.ff * self.width
 
     def route(self, x, want_chosen: bool = False):
         """-> (weights [T, E], chosen [T, top] or None, the shared gate's values in front of its sigmoid [T, 1] or None)."""
@@ -304,16 +308,17 @@ class PlainRoutedExperts(FeedForward):
         k = self.rt.k
         status = ctx.status if ctx is not None else None
         more = dict(weigh_input=True) if self.weigh == "input" else {}
-        if not self.sparse:
+        if not self.grouped(x.shape[0]):
             w, _, gate = self.route(x)
             return k.moe_plain_act(k.linear(x, self.up, None, self.rt.dtype), w, self.E, self.ff, self.activation, shared_gate=gate,
                                    out=out, **more)
         w, chosen, gate = self.route(x, want_chosen=True)
         plan = k.moe_sort(chosen, w)
-        y = k.moe_grouped_up(x, plan, self.up, self.E, self.ff, self.activation, weigh_input=self.weigh == "input", status=status)
-        pairs = k.moe_grouped_down(y, plan, self.down, self.E, self.ff, stacked=True, tokens=x.shape[0], status=status)
+        n = self.E * self.ff
+        y = k.moe_grouped_up(x, plan, self.up[:n], self.E, self.ff, self.activation, weigh_input=self.weigh == "input", status=status)
+        pairs = k.moe_grouped_down(y, plan, self.down[:, :n], self.E, self.ff, tokens=x.shape[0], status=status)
         if self.shared_ff:
-            k.plain_up(x, self.shared_up, self.activation, gate, out=out, status=status)
+            k.plain_up(x, self.up[n:], self.activation, gate, out=out, status=status)
         return pairs, plan
 
     def add_kept(self, y, kept):
@@ -323,8 +328,8 @@ class PlainRoutedExperts(FeedForward):
 
     def forward(self, x, ctx):
         k = self.rt.k
-        if not self.sparse:
+        if not self.grouped(x.shape[0]):
             return k.linear(self.forward_inner(x, ctx), self.down, None, self.rt.dtype)
         out = torch.empty((x.shape[0], self.shared_ff), dtype=self.rt.dtype, device=x.device)
         kept = self.forward_inner(x, ctx, out=out)
-        return self.add_kept(k.linear(out, self.shared_down, None, self.rt.dtype) if self.shared_ff else None, kept)
+        return self.add_kept(k.linear(out, self.down[:, self.E * self.ff:], None, self.rt.dtype) if self.shared_ff else None, kept)

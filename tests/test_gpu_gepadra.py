@@ -607,7 +607,7 @@ def test_clamped_gated_feed_forward(T, ff):
 @pytest.mark.parametrize("T", [1, 3, 40, 100, 300])
 @pytest.mark.parametrize("ff,shared", [(128, 256), (72, 40), (264, 0)])
 @pytest.mark.parametrize("weigh", ["input", "output"])
-def test_grouped_experts_without_a_gate(T, ff, shared, weigh):
+def test_grouped_experts_without_a_gate(monkeypatch, T, ff, shared, weigh):
     """Only the chosen experts run, sorted pairs on the tensor cores (the tcgen05 kernel from 128 tokens on), against the same
     experts side by side; with the output product the part's own and the block's."""
     from fastmlx_b200 import kernels as k
@@ -618,6 +618,7 @@ def test_grouped_experts_without_a_gate(T, ff, shared, weigh):
     x = torch.randn(T, width, generator=g).bfloat16().cuda()
     rt = Runtime(torch.device("cuda"), torch.bfloat16, k)
     opts = dict(shared_ff=shared, activation="gelu", correction=None, scores="sigmoid", weigh=weigh)
+    monkeypatch.setattr(PlainRoutedExperts, "GROUPED_SHARE", 1.1)           # however many experts the tokens use
     outs, tensors = [], None
     for sparse, output in ((False, True), (True, True), (True, False), (False, False)):
         part = PlainRoutedExperts(width, E, top, ff, "m", sparse=sparse, output=output, **opts)
@@ -625,30 +626,30 @@ def test_grouped_experts_without_a_gate(T, ff, shared, weigh):
             gw = torch.Generator().manual_seed(5)
             tensors = {s.name: (torch.randn(s.shape, generator=gw) * 2 / s.shape[-1] ** 0.5).bfloat16() for s in part.weight_specs()}
         part.bind(tensors, rt)
-        assert part.sparse == sparse and len(part.kept_pieces) == (E if sparse else 0)
+        assert part.sparse == sparse and part.skips(T) == (E * ff if sparse else 0)
         if output:
             y = part.forward(x, None)
         else:
-            joined = JoinedLinear(width, part.out_pieces)
-            joined.leave_out(part.kept_pieces)
-            h = torch.empty(T, part.inner_features, dtype=torch.bfloat16, device="cuda")
-            kept = part.forward_inner(x, None, out=h)
-            if joined.pieces:
-                joined.bind(tensors, rt)
-                y = joined.forward(h)
-            else:
-                y = torch.zeros(T, width, dtype=torch.bfloat16, device="cuda")
-            y = part.add_kept(y, kept) if sparse else y
+            joined = JoinedLinear(width, part.out_pieces + [("mixer", 24, None)])
+            joined.bind(dict(tensors, mixer=torch.zeros(width, 24).bfloat16()), rt)
+            part.bind_joined(joined.weight)
+            skip = part.skips(T)
+            h = torch.ones(T, joined.in_features - skip, dtype=torch.bfloat16, device="cuda")
+            kept = part.forward_inner(x, None, out=h[:, :h.shape[1] - 24])
+            y = joined.forward(h, skip=skip)
+            y = part.add_kept(y, kept) if skip else y
         outs.append(y.double().cpu())
     for o in outs[1:]:
         assert (o - outs[0]).abs().max() < 2e-2 * outs[0].abs().max()
 
 
+@pytest.mark.parametrize("share", [1.1, 0.45], ids=["always", "by-size"])
 @pytest.mark.parametrize("cut", ["whole", "portions", "mixed", "ones"])
-def test_replay_with_grouped_experts(models, monkeypatch, cut):
+def test_replay_with_grouped_experts(models, monkeypatch, cut, share):
     """The same model with its experts' products grouped: pair outputs are added to the joined product's."""
     from fastmlx_b200.parts import PlainRoutedExperts
     monkeypatch.setattr(PlainRoutedExperts, "SPARSE_MIN_BYTES", 0)
+    monkeypatch.setattr(PlainRoutedExperts, "GROUPED_SHARE", share)
     d, W, prompts, ref, skip = models["G3", "bfloat16"]
     steps = CUTS[cut](prompts)
     outs, rp = _run(d, "bfloat16", steps, CASES["G3"]["max_tokens"], CASES["G3"]["page"])
